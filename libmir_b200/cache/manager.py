@@ -3,11 +3,12 @@
 Host-side bookkeeping only; the device memory the ids refer to is in cache/storage.py, so the manager
 can be tested without a GPU.
 
-Groups.  Schedule entries (layer runs) with the same needs share a group: (kv_heads, head_dim, window)
+Groups.  Schedule entries (layer runs) with the same needs share a group: (kv_heads, head_dim, window, chunk)
 for paged keys/values.  Each group has its own PagePool and each request has one block table per
 group; one page id addresses the same slot range in every entry of the group, as libmir's block id
 addresses every layer (runtime/src/kv/write.rs:7-10).  A group without a window keeps every token; a
-group with a window gives pages back as soon as no later query can see them.
+group with a window, or whose queries see their own run of `chunk` positions only, gives pages back as soon as no
+later query can see them.
 
 Lengths.  `length` is the number of tokens whose keys are in the cache.  A step first `grow`s the
 request to length + count (pages for the new tokens, all groups or none), runs, then `commit`s the new
@@ -46,6 +47,25 @@ class GroupInfo:
     @property
     def window(self) -> Optional[int]:
         return self.requirement.window
+
+    @property
+    def chunk(self) -> Optional[int]:
+        return self.requirement.chunk
+
+    @property
+    def releases(self) -> bool:
+        """Whether a live request's pages are given back as it goes on (a window, or runs of positions)."""
+        return self.requirement.releases
+
+    def dead_keys(self, length: int) -> int:
+        """How many of a request's first keys no later query sees once `length` tokens are cached: a query at position
+        p >= length sees keys above p - window, and keys of its own run of `chunk` positions only."""
+        dead = 0
+        if self.window is not None:
+            dead = length - self.window + 1
+        if self.chunk is not None:
+            dead = max(dead, length // self.chunk * self.chunk)
+        return max(0, dead)
 
     @property
     def keep_first(self) -> int:
@@ -104,7 +124,7 @@ class CacheManager:
             if item.source != item.entry and split_requirement(item.requirement)[0] is not None:
                 self.entry_group[item.entry] = self.entry_group[item.source]
                 self.entry_local[item.entry] = self.entry_local[item.source]
-        capable = len(self.groups) == 1 and self.groups[0].window is None and not self.state_entries
+        capable = len(self.groups) == 1 and not self.groups[0].releases and not self.state_entries
         self.prefix: Optional[PrefixIndex] = PrefixIndex() if prefix_cache and capable else None
         self._model_key = model_key.encode()
         self.prefix_hit_tokens = 0                     # tokens that admitted requests found cached
@@ -164,9 +184,10 @@ class CacheManager:
     def peak_pages(self, length: int, group: GroupInfo, portion: int) -> int:
         """Most pages of `group` that a request of `length` tokens holds at once when it is fed in
         portions of at most `portion` tokens."""
-        if group.window is None:
+        if not group.releases:
             return self._blocks_for(length)
-        span = min(length, group.window + portion)
+        seen = min(reach for reach in (group.window, group.chunk) if reach is not None)
+        span = min(length, seen + portion)
         kept = self._blocks_for(min(length, group.keep_first))
         return min(self._blocks_for(length), span // self.page_size + 2 + kept)
 
@@ -239,11 +260,9 @@ class CacheManager:
                         pool.mark_cached(table[block])
         sequence.length = new_length
         for index, group in enumerate(self.groups):
-            if group.window is None:
+            if not group.releases:
                 continue
-            # a later query at position p >= new_length sees keys j > p - window >= new_length - window
-            dead_keys = new_length - group.window + 1       # keys < dead_keys are never read again
-            dead_blocks = max(0, dead_keys // self.page_size)
+            dead_blocks = group.dead_keys(new_length) // self.page_size      # the keys in them are never read again
             table = sequence.tables[index]
             # blocks that hold one of the first `keep_first` tokens are never given back
             first = max(sequence.first_live[index], self._blocks_for(group.keep_first))
@@ -278,7 +297,7 @@ class CacheManager:
             "page_size": self.page_size,
             "live_requests": len(self.live),
             "free_slots": len(self._free_slots),
-            "groups": [{"window": g.window, "kv_heads": g.requirement.kv_heads, "head_dim": g.requirement.head_dim,
+            "groups": [{"window": g.window, "chunk": g.chunk, "kv_heads": g.requirement.kv_heads, "head_dim": g.requirement.head_dim,
                         "value_head_dim": g.requirement.value_dim,
                         "entries": len(g.entries), "pages": g.pool.count, "free": g.pool.available,
                         "high_water": g.pool.high_water, "reused": g.pool.reused} for g in self.groups],

@@ -64,10 +64,17 @@ class PagedKv:
     window: Optional[int] = None
     value_head_dim: Optional[int] = None     # 0: one vector per token and kv head only (a latent read as key and as value)
     keep_first: int = 0           # with a window: the request's first tokens whose pages are never given back
+    # positions are cut into runs of `chunk`; a query sees the keys of its own run only, so a run that is over is given back
+    chunk: Optional[int] = None
 
     @property
     def value_dim(self) -> int:
         return self.head_dim if self.value_head_dim is None else self.value_head_dim
+
+    @property
+    def releases(self) -> bool:
+        """Whether pages are given back while the request still lives."""
+        return self.window is not None or self.chunk is not None
 
     @property
     def elements_per_token(self) -> int:
@@ -243,6 +250,11 @@ class SoftmaxAttentionSpec(PartSpec):
     qk_norm_after_rotation: bool = False
     softcap: Optional[float] = None
     distance_bias: Optional[DistanceBiasSpec] = None
+    # chunk: the query at position i sees key j <= i only where i // chunk == j // chunk (positions of the request).
+    # head_mix: a stored square matrix over the query heads (tensor `head_mix`): head h applies the combination
+    # sum_g head_mix[h, g] weights_g of all heads' softmax weights to the values of its own kv head.
+    chunk: Optional[int] = None
+    head_mix: bool = False
     kind: str = field(init=False, default="softmax_attention")
 
     @property
@@ -254,6 +266,7 @@ class SoftmaxAttentionSpec(PartSpec):
 class SwiGluSpec(PartSpec):
     hidden_size: int = 0
     intermediate_size: int = 0
+    names: tuple = ()                        # (local name, stored name) pairs for checkpoints with names of their own
     kind: str = field(init=False, default="swiglu")
 
 
@@ -272,7 +285,8 @@ class GeluMlpSpec(PartSpec):
 class LatentAttentionSpec(PartSpec):
     """Softmax attention whose keys and values are up-projections of one cached latent per token, beside one rotated
     key part shared by all heads (parts/latent_attention.py).  Per head `head_dim` unrotated and `rotary_dim` rotated
-    query / key dims and `value_dim` value dims; `q_rank` and `kv_rank` are the widths of the two latents.
+    query / key dims and `value_dim` value dims; `q_rank` and `kv_rank` are the widths of the two latents.  `q_rank` 0:
+    queries are one projection of the mixer's input (tensor `q`), without a latent and its norm.
     `gate`: the concatenated heads are multiplied by the sigmoid of a projection of the mixer's input."""
 
     hidden_size: int = 0
@@ -369,6 +383,20 @@ class GatedDeltaRuleSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class SelectiveScanSpec(PartSpec):
+    """A diagonal state-space recurrence whose step size, input and read-out vectors depend on the token
+    (parts/selective_scan.py): `inner` channels with `state` numbers each, a short causal convolution of `conv_taps`
+    taps with a bias before it, step sizes through a low-rank pair of rank `dt_rank`."""
+
+    hidden_size: int = 0
+    inner: int = 0
+    state: int = 0
+    dt_rank: int = 0
+    conv_taps: int = 4
+    kind: str = field(init=False, default="selective_scan")
+
+
+@dataclass(frozen=True)
 class SideBySideSpec(PartSpec):
     """Several mixers that read the same input; the result is `scale` times the sum of their outputs, each first
     RMS-normed over the model width with a plain weight `<branch name>.<out_tensor>`."""
@@ -402,8 +430,9 @@ class LayerSpec:
     Arrangements: "pre_norm" (a norm before each of the two branches, one after the other), "parallel" (both
     branches read the same residual and their results are added to it together: through one norm, `mixer_norm`, if
     `feed_forward_norm` is None, else each through a norm of its own), "output_norm" (each branch reads the
-    residual itself and its RESULT goes through the norm: x += residual_scale * norm(branch(x)), one after the other)
-    and "streams" (the residual is ModelSpec.streams copies; each branch reads a mix of them through its norm and
+    residual itself and its RESULT goes through the norm: x += residual_scale * norm(branch(x)), one after the other),
+    "sandwich" (a norm before and a norm behind each branch: x += mixer_out_norm(mixer(mixer_norm(x))), then the same
+    with the feed-forward's two norms) and "streams" (the residual is ModelSpec.streams copies; each branch reads a mix of them through its norm and
     writes into all of them as `mixer_streams` / `feed_forward_streams`, StreamMixSpec, say).
     """
 
@@ -417,6 +446,8 @@ class LayerSpec:
     residual_scale: float = 1.0           # what a branch's (normed) result is multiplied by ("output_norm" only)
     mixer_streams: Optional[PartSpec] = None          # ("streams" only) how the mixer reads and writes the streams
     feed_forward_streams: Optional[PartSpec] = None   # the same for the feed-forward
+    mixer_out_norm: Optional[PartSpec] = None         # ("sandwich" only) the norm on the mixer's result
+    feed_forward_out_norm: Optional[PartSpec] = None  # the same for the feed-forward
 
 
 @dataclass(frozen=True)

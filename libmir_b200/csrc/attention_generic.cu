@@ -11,7 +11,7 @@
 // Replaces libmir's paged_attention_bf16.cu:14-93, paged_attention_batch_bf16.cu:14-102 and
 // paged_prefill_attention_batch_bf16.cu:14-124: score = (q . k) * scale, running maximum and
 // denominator, all in 32-bit; key j is visible to the query at position p iff j <= p and
-// (window == 0 or j > p - window or j < keep_first): with a window, the first keep_first keys of a request stay
+// (window == 0 or j > p - window or j < keep_first) and, with a chunk, j / chunk == p / chunk: with a window, the first keep_first keys of a request stay
 // visible to every later query (they keep their pages and their true positions).  Values may be narrower or wider
 // than keys (value_dim).  A query walks over the kept keys first, then over its window.  Consecutive value rows
 // lie value_row_width elements apart: value_dim in a cache of their own, head_dim where the values are the first
@@ -38,7 +38,7 @@ __global__ void paged_attention_generic_kernel(
     const int* __restrict__ row_of_token, const int* __restrict__ positions, int page_size, int heads, int kv_heads,
     int head_dim, int value_dim, int value_row_width, float scale, int window, int keep_first,
     const float* __restrict__ sinks, const T* __restrict__ gate, size_t gate_stride, int gate_per_head, float softcap,
-    const float* __restrict__ rel_bias, int rel_rows) {
+    const float* __restrict__ rel_bias, int rel_rows, int chunk_size) {
   __shared__ float q_shared[kWarpsPerBlock][kMaxHeadDim];
   const int lane = threadIdx.x;
   const int warp = threadIdx.y;
@@ -49,7 +49,8 @@ __global__ void paged_attention_generic_kernel(
   const int position = positions[token];
   const int kv_head = head / (heads / kv_heads);
   const int* table = block_table + (size_t)row * table_width;
-  const int first_key = (window > 0 && position + 1 > window) ? position + 1 - window : 0;
+  int first_key = (window > 0 && position + 1 > window) ? position + 1 - window : 0;
+  if (chunk_size > 0 && position >= 0) first_key = max(first_key, position - position % chunk_size);
 
   const T* q_row = q + (size_t)token * q_token_stride + (size_t)head * head_dim;
   for (int d = lane; d < head_dim; d += 32) q_shared[warp][d] = to_float(q_row[d]);
@@ -143,10 +144,10 @@ MIR_EXPORT int mir_paged_attention_generic(int bf16, const void* q, long long q_
                                            float scale, int window, int keep_first, int value_row_width,
                                            const float* sinks, const void* gate, long long gate_stride,
                                            int gate_per_head, float softcap, const float* rel_bias, int rel_rows,
-                                           cudaStream_t stream) {
+                                           int chunk, cudaStream_t stream) {
   if (tokens == 0) return MIR_OK;
   if (tokens < 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || page_size <= 0 || table_width <= 0 ||
-      window < 0 || keep_first < 0) {
+      window < 0 || keep_first < 0 || chunk < 0 || (chunk > 0 && keep_first > 0)) {
     mir_set_error("paged_attention: bad sizes (tokens %d, heads %d, kv heads %d, page %d, table width %d)", tokens,
                   heads, kv_heads, page_size, table_width);
     return MIR_BAD_ARGUMENT;
@@ -168,12 +169,12 @@ MIR_EXPORT int mir_paged_attention_generic(int bf16, const void* q, long long q_
         (const __nv_bfloat16*)q, (size_t)q_token_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_pages,
         (const __nv_bfloat16*)v_pages, block_table, table_width, row_of_token, positions, page_size, heads, kv_heads,
         head_dim, value_dim, value_row_width, scale, window, keep_first, sinks, (const __nv_bfloat16*)gate,
-        (size_t)gate_stride, gate_per_head, softcap, rel_bias, rel_rows);
+        (size_t)gate_stride, gate_per_head, softcap, rel_bias, rel_rows, chunk);
   else
     paged_attention_generic_kernel<<<grid, block, 0, stream>>>(
         (const float*)q, (size_t)q_token_stride, (float*)out, (const float*)k_pages, (const float*)v_pages,
         block_table, table_width, row_of_token, positions, page_size, heads, kv_heads, head_dim, value_dim,
         value_row_width, scale, window, keep_first, sinks, (const float*)gate, (size_t)gate_stride, gate_per_head, softcap,
-        rel_bias, rel_rows);
+        rel_bias, rel_rows, chunk);
   return mir_check_launch("paged_attention_generic");
 }

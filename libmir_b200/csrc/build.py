@@ -34,7 +34,7 @@ LIBRARIES = {
     "core": {
         "sources": ["runtime.cu", "elementwise.cu", "qk_rope_store.cu", "attention_generic.cu", "gemm_f32.cu",
                     "sampling.cu", "executor.cu", "delta_rule.cu", "latent_attention.cu", "wkv.cu", "moe.cu",
-                    "retention.cu", "streams.cu", "qk_prepare.cu"],
+                    "retention.cu", "streams.cu", "qk_prepare.cu", "short_conv.cu", "selective_scan.cu", "attention_mixed.cu"],
         "link": [],
         "defines": [],
     },
@@ -50,7 +50,7 @@ LIBRARIES = {
 }
 # the bfloat16 library with time stamps inside its kernels (trace.cuh), for bench.py --phase trace
 LIBRARIES["bf16_trace"] = dict(LIBRARIES["bf16"], defines=LIBRARIES["bf16"]["defines"] + ["-DMIR_TRACE"])
-HEADERS = ["common.cuh", "launchers.h", "trace.cuh"]
+HEADERS = ["common.cuh", "launchers.h", "trace.cuh", "short_conv.cuh"]
 
 
 def _nvcc() -> str:

@@ -8,9 +8,7 @@
 // sigmoid of beta, softplus, both exponentials of the decay.
 //
 // Kernels of this file:
-//   short_conv_silu   y[t, c] = silu(sum_j w[c, j] x[t - (taps-1) + j, c]) over a request's own tokens, with the
-//                     taps-1 inputs before the portion taken from the request's state; then the state's update.
-//   delta_rule_prepare the same convolution, then what else the recurrence needs of a token: q and k as unit vectors,
+//   delta_rule_prepare the short convolution (short_conv.cu), then what else the recurrence needs of a token: q and k as unit vectors,
 //                     sigmoid(beta), the decay; all tokens in parallel.
 //   delta_rule_scan   the recurrence: a few lanes per (request, head, value channel) hold one column of S in
 //                     registers, walk over the request's tokens of this step, and write the column back.  No shared
@@ -19,62 +17,17 @@
 //   gated_head_norm   out = o / rms(o) * weight * act(gate) per (token, head), act = silu or sigmoid.
 // A row of a captured decode batch whose position is negative is padding: nothing of it is read or written.
 #include "common.cuh"
+#include "short_conv.cuh"
 
 using namespace mir;
 
 namespace {
 
-constexpr int kMaxTaps = 16;
 constexpr int kMaxPerLane = 8;          // key channels per lane: key_dim <= 256
 
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
-
-// grid (tokens, ceil(channels / 256)).  x: the packed projection rows, channel c of token t at x[t * ldx + c].
-template <typename T>
-__global__ void short_conv_silu_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w,
-                                       const float* __restrict__ tail, const int* __restrict__ row_of_token,
-                                       const int* __restrict__ query_starts, const int* __restrict__ state_slots,
-                                       const int* __restrict__ positions, float* __restrict__ out, int channels,
-                                       int taps) {
-  grid_launch_dependents();
-  grid_dependency_wait();
-  const int token = blockIdx.x;
-  const int c = blockIdx.y * blockDim.x + threadIdx.x;
-  if (c >= channels || positions[token] < 0) return;
-  const int row = row_of_token[token];
-  const int start = query_starts[row];
-  const int local = token - start;
-  const float* old = tail + (size_t)state_slots[row] * (taps - 1) * channels;
-  float acc = 0.0f;
-  for (int j = 0; j < taps; ++j) {
-    const int src = local - (taps - 1) + j;
-    const float value = src >= 0 ? to_float(x[(size_t)(start + src) * ldx + c]) : old[(size_t)(taps - 1 + src) * channels + c];
-    acc = fmaf(to_float(w[(size_t)c * taps + j]), value, acc);
-  }
-  out[(size_t)token * channels + c] = silu(acc);
-}
-
-// grid (rows, ceil(channels / 256)): the last taps-1 inputs of the request, old ones where the portion is shorter.
-template <typename T>
-__global__ void short_conv_tail_kernel(const T* __restrict__ x, long long ldx, float* __restrict__ tail,
-                                       const int* __restrict__ query_starts, const int* __restrict__ state_slots,
-                                       const int* __restrict__ positions, int channels, int taps, int skip_single) {
-  grid_launch_dependents();
-  grid_dependency_wait();
-  const int row = blockIdx.x;
-  const int c = blockIdx.y * blockDim.x + threadIdx.x;
-  const int start = query_starts[row], count = query_starts[row + 1] - start;
-  if (c >= channels || count <= 0 || positions[start] < 0 || (skip_single && count == 1)) return;
-  float* mine = tail + (size_t)state_slots[row] * (taps - 1) * channels;
-  float keep[kMaxTaps];
-  for (int j = 0; j < taps - 1; ++j) {
-    const int src = count - (taps - 1) + j;
-    keep[j] = src >= 0 ? to_float(x[(size_t)(start + src) * ldx + c]) : mine[(size_t)(taps - 1 + src) * channels + c];
-  }
-  for (int j = 0; j < taps - 1; ++j) mine[(size_t)j * channels + c] = keep[j];
-}
 
 // Everything the recurrence needs of a token, in 32-bit, one CTA per token: the short convolution and silu of
 // q | k | v (as short_conv_silu), q and k made unit vectors per key head (q also times key_dim^-1/2),
@@ -476,37 +429,6 @@ int launch_scan(cudaStream_t stream, const float* qkv, const float* beta, const 
 }
 
 }  // namespace
-
-// x: first convolved channel of token 0 (q | k | v lie side by side in the packed projection); w [channels, taps]
-// in the activations' type; tail [slots, taps - 1, channels] 32-bit; out [tokens, channels] 32-bit.
-MIR_EXPORT int mir_short_conv_silu(int bf16, const void* x, long long ldx, const void* w, float* tail,
-                                   const int* row_of_token, const int* query_starts, const int* state_slots,
-                                   const int* positions, float* out, int tokens, int rows, int channels, int taps,
-                                   cudaStream_t stream) {
-  if (tokens == 0 || rows == 0) return MIR_OK;
-  if (tokens < 0 || rows < 0 || channels <= 0 || taps < 1 || taps > kMaxTaps) {
-    mir_set_error("short_conv_silu: bad sizes (tokens %d, rows %d, channels %d, taps %d; at most %d taps)", tokens, rows,
-                  channels, taps, kMaxTaps);
-    return MIR_BAD_ARGUMENT;
-  }
-  const int threads = channels >= 256 ? 256 : ((channels + 31) / 32) * 32;
-  const dim3 grid(tokens, (channels + threads - 1) / threads), tail_grid(rows, (channels + threads - 1) / threads);
-  int status;
-  if (bf16)
-    status = mir_launch("short_conv_silu", short_conv_silu_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, 0,
-                        (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)w, (const float*)tail, row_of_token,
-                        query_starts, state_slots, positions, out, channels, taps);
-  else
-    status = mir_launch("short_conv_silu", short_conv_silu_kernel<float>, grid, dim3(threads), 0, stream, 0,
-                        (const float*)x, ldx, (const float*)w, (const float*)tail, row_of_token, query_starts,
-                        state_slots, positions, out, channels, taps);
-  if (status != MIR_OK || taps == 1) return status;
-  if (bf16)
-    return mir_launch("short_conv_tail", short_conv_tail_kernel<__nv_bfloat16>, tail_grid, dim3(threads), 0, stream, 0,
-                      (const __nv_bfloat16*)x, ldx, tail, query_starts, state_slots, positions, channels, taps, 0);
-  return mir_launch("short_conv_tail", short_conv_tail_kernel<float>, tail_grid, dim3(threads), 0, stream, 0,
-                    (const float*)x, ldx, tail, query_starts, state_slots, positions, channels, taps, 0);
-}
 
 // bf16: the type of x, w and beta_raw (and of decay_raw unless decay_f32).  decay_width: heads, or heads * key_dim for
 // one decay per key channel.  Writes qkv [tokens, channels], beta [tokens, heads], decay [tokens, decay_width] (32-bit)

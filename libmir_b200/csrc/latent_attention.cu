@@ -3,7 +3,8 @@
 //
 //   latent_prepare   per token: RMS norm of the query latent (out: the normed latent for the query up-projection),
 //                    RMS norm of the key/value latent and rotation of the shared key part, both written to the
-//                    token's cache row [kv_rank | rotary dims]
+//                    token's cache row [kv_rank | rotary dims]; without a query latent (q_rank 0) the queries' rotated
+//                    parts are turned by the same launch
 //   rope_rows        rotation of [tokens, heads, dims] views by position, half-split or interleaved pairs, cos and sin
 //                    times a magnitude; in place or into another buffer
 //   head_linear      out[t, h, :] = W_h x[t, h, :], a product per head on strided views, optionally times the
@@ -38,7 +39,9 @@ __global__ void latent_prepare_kernel(const T* __restrict__ packed, long long ld
                                       int kv_rank, int rotary, const float* __restrict__ q_norm,
                                       const float* __restrict__ kv_norm, float eps, const int* __restrict__ positions,
                                       const int* __restrict__ slot_mapping, const float* __restrict__ inv_freq,
-                                      float magnitude, int interleaved, T* __restrict__ latent_q, T* __restrict__ pages) {
+                                      float magnitude, int interleaved, T* __restrict__ latent_q, T* __restrict__ pages,
+                                      const T* __restrict__ turn_src, long long src_token, long long src_head,
+                                      T* __restrict__ turn_dst, long long dst_token, long long dst_head, int turn_heads) {
   __shared__ float scratch[32];
   grid_launch_dependents();
   grid_dependency_wait();
@@ -46,15 +49,29 @@ __global__ void latent_prepare_kernel(const T* __restrict__ packed, long long ld
   const int position = positions[token];
   if (position < 0) return;                                      // a padding row of a captured batch
   const T* row = packed + (size_t)token * ld;
+  const int half = rotary / 2;
   float sum = 0.0f;
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
-    const float x = to_float(row[q_offset + i]);
-    sum = fmaf(x, x, sum);
+  if (q_rank > 0) {
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
+      const float x = to_float(row[q_offset + i]);
+      sum = fmaf(x, x, sum);
+    }
+    sum = block_sum(sum, scratch);
+    const float q_inverse = rsqrtf(sum / (float)q_rank + eps);
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
+      latent_q[(size_t)token * q_rank + i] = from_float<T>(to_float(row[q_offset + i]) * q_inverse * q_norm[i]);
   }
-  sum = block_sum(sum, scratch);
-  const float q_inverse = rsqrtf(sum / (float)q_rank + eps);
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
-    latent_q[(size_t)token * q_rank + i] = from_float<T>(to_float(row[q_offset + i]) * q_inverse * q_norm[i]);
+  // the queries' rotated parts: threads side by side take the pairs of a head, then the next head's
+  for (int index = threadIdx.x; index < turn_heads * half; index += blockDim.x) {
+    const int head = index / half, i = index - head * half;
+    const int first = interleaved ? 2 * i : i, second = interleaved ? 2 * i + 1 : i + half;
+    const T* from = turn_src + (size_t)token * src_token + (size_t)head * src_head;
+    T* to = turn_dst + (size_t)token * dst_token + (size_t)head * dst_head;
+    float u = to_float(from[first]), v = to_float(from[second]);
+    rotate_pair(u, v, position, inv_freq[i], magnitude);
+    to[first] = from_float<T>(u);
+    to[second] = from_float<T>(v);
+  }
   const int slot = slot_mapping != nullptr ? slot_mapping[token] : -1;
   if (slot < 0) return;                                          // (uniform over the CTA)
   sum = 0.0f;
@@ -67,7 +84,6 @@ __global__ void latent_prepare_kernel(const T* __restrict__ packed, long long ld
   T* cached = pages + (size_t)slot * (kv_rank + rotary);
   for (int i = threadIdx.x; i < kv_rank; i += blockDim.x)
     cached[i] = from_float<T>(to_float(row[kv_offset + i]) * kv_inverse * kv_norm[i]);
-  const int half = rotary / 2;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     const int first = interleaved ? 2 * i : i, second = interleaved ? 2 * i + 1 : i + half;
     float u = to_float(row[kv_offset + kv_rank + first]), v = to_float(row[kv_offset + kv_rank + second]);
@@ -170,9 +186,11 @@ MIR_EXPORT int mir_sigmoid_gate(int bf16, void* x, long long x_stride, const voi
 MIR_EXPORT int mir_latent_prepare(int bf16, const void* packed, long long ld, int q_offset, int q_rank, int kv_offset,
                                   int kv_rank, int rotary, const float* q_norm, const float* kv_norm, float eps,
                                   const int* positions, const int* slot_mapping, const float* inv_freq, float magnitude,
-                                  int interleaved, void* latent_q, void* pages, int tokens, cudaStream_t stream) {
+                                  int interleaved, void* latent_q, void* pages, const void* turn_src, long long src_token,
+                                  long long src_head, void* turn_dst, long long dst_token, long long dst_head,
+                                  int turn_heads, int tokens, cudaStream_t stream) {
   if (tokens == 0) return MIR_OK;
-  if (tokens < 0 || q_rank <= 0 || kv_rank <= 0 || rotary < 0 || rotary % 2) {
+  if (tokens < 0 || q_rank < 0 || turn_heads < 0 || (turn_heads > 0 && (turn_src == nullptr || turn_dst == nullptr)) || kv_rank <= 0 || rotary < 0 || rotary % 2) {
     mir_set_error("latent_prepare: bad sizes (tokens %d, ranks %d and %d, rotary %d)", tokens, q_rank, kv_rank, rotary);
     return MIR_BAD_ARGUMENT;
   }
@@ -180,10 +198,12 @@ MIR_EXPORT int mir_latent_prepare(int bf16, const void* packed, long long ld, in
     return mir_launch("latent_prepare", latent_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, stream, 0,
                       (const __nv_bfloat16*)packed, ld, q_offset, q_rank, kv_offset, kv_rank, rotary, q_norm, kv_norm, eps,
                       positions, slot_mapping, inv_freq, magnitude, interleaved, (__nv_bfloat16*)latent_q,
-                      (__nv_bfloat16*)pages);
+                      (__nv_bfloat16*)pages, (const __nv_bfloat16*)turn_src, src_token, src_head,
+                      (__nv_bfloat16*)turn_dst, dst_token, dst_head, turn_heads);
   return mir_launch("latent_prepare", latent_prepare_kernel<float>, dim3(tokens), dim3(256), 0, stream, 0,
                     (const float*)packed, ld, q_offset, q_rank, kv_offset, kv_rank, rotary, q_norm, kv_norm, eps, positions,
-                    slot_mapping, inv_freq, magnitude, interleaved, (float*)latent_q, (float*)pages);
+                    slot_mapping, inv_freq, magnitude, interleaved, (float*)latent_q, (float*)pages, (const float*)turn_src,
+                    src_token, src_head, (float*)turn_dst, dst_token, dst_head, turn_heads);
 }
 
 MIR_EXPORT int mir_rope_rows(int bf16, const void* src, long long src_token, long long src_head, void* dst,

@@ -8,6 +8,8 @@
 //   layer_norm      out = (u - mean) / sqrt(var + eps) * w + b, var the mean of the squared deviations (two passes over
 //                   the row, which stays in shared memory), u a plain 32-bit row or the mix above of a token's streams
 //                   formed on the way in; optional row gather; result in the engine's type
+//   add_layer_norm  x += layer_norm(y) (+ further rows), and in the same pass over a token the layer norm of the new x for
+//                   whoever reads it next: what stands between two sublayers that have a norm before and a norm behind them
 //   streams_write   the update above, in place: a thread takes one column of one token, reads its S old values and
 //                   writes the S new ones
 //   streams_write_norm  that update and the layer norm of the next reader's mix of the new streams in one pass over a
@@ -114,6 +116,68 @@ __global__ void __launch_bounds__(512, 3) layer_norm_kernel(const float* __restr
     }
   }
   norm_row<T, V>(row_values, sum, scratch, weight, bias, out + (size_t)blockIdx.x * width, width, eps);
+}
+
+// One CTA per token.  x [tokens, width] in place; y [tokens, width]; rows (or null) [tokens, width] is added to x as well;
+// out (or null): the layer norm of the new x with the reader's weight, bias and eps.
+template <typename T, int V>
+__global__ void __launch_bounds__(512, 2) add_layer_norm_kernel(
+    float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ weight, const float* __restrict__ bias,
+    float eps, const float* __restrict__ rows, const float* __restrict__ next_weight, const float* __restrict__ next_bias,
+    float next_eps, T* __restrict__ out, int width) {
+  extern __shared__ float row_values[];            // [width] the branch's row, then the new residual's; [width] the residual
+  __shared__ float scratch[128];
+  float* const old = row_values + width;
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const size_t base = (size_t)blockIdx.x * width;
+  float sum = 0.0f;
+  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+    if constexpr (V == 4) {
+      const float4 branch = *reinterpret_cast<const float4*>(y + base + c);
+      float4 residual = *reinterpret_cast<const float4*>(x + base + c);
+      *reinterpret_cast<float4*>(row_values + c) = branch;
+      *reinterpret_cast<float4*>(old + c) = residual;
+      sum += branch.x; sum += branch.y; sum += branch.z; sum += branch.w;
+    } else {
+      row_values[c] = y[base + c];
+      old[c] = x[base + c];
+      sum += row_values[c];
+    }
+  }
+  const float mean = block_sum_once(sum, scratch) / (float)width;
+  float squares = 0.0f;
+  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      const float d = row_values[c + v] - mean;
+      squares = fmaf(d, d, squares);
+    }
+  }
+  const float inverse = rsqrtf(block_sum_once(squares, scratch + 32) / (float)width + eps);
+  float total = 0.0f;
+  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+    alignas(16) float w[V], b[V], more[V], fresh[V];
+    if constexpr (V == 4) {
+      *reinterpret_cast<float4*>(w) = __ldg(reinterpret_cast<const float4*>(weight + c));
+      *reinterpret_cast<float4*>(b) = __ldg(reinterpret_cast<const float4*>(bias + c));
+      *reinterpret_cast<float4*>(more) = rows != nullptr ? *reinterpret_cast<const float4*>(rows + base + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    } else {
+      w[0] = weight[c];
+      b[0] = bias[c];
+      more[0] = rows != nullptr ? rows[base + c] : 0.0f;
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      fresh[v] = old[c + v] + fmaf((row_values[c + v] - mean) * inverse, w[v], b[v]);
+      if (rows != nullptr) fresh[v] += more[v];
+      row_values[c + v] = fresh[v];
+      total += fresh[v];
+    }
+    if constexpr (V == 4) *reinterpret_cast<float4*>(x + base + c) = *reinterpret_cast<const float4*>(fresh);
+    else x[base + c] = fresh[0];
+  }
+  if (out != nullptr) norm_row<T, V>(row_values, total, scratch + 64, next_weight, next_bias, out + base, width, next_eps);
 }
 
 __global__ void streams_write_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ mix,
@@ -309,6 +373,35 @@ MIR_EXPORT int mir_layer_norm(int bf16, const float* x, int streams, const float
   if (wide) MIR_LAYER_NORM(float, 4);
   MIR_LAYER_NORM(float, 1);
 #undef MIR_LAYER_NORM
+}
+
+// x [tokens, width] += layer_norm(y; weight, bias, eps) (+ rows [tokens, width], or null), 32-bit; out (bfloat16 or 32-bit,
+// or null) = layer_norm(x; next_weight, next_bias, next_eps) of the new x.
+MIR_EXPORT int mir_add_layer_norm(int bf16, float* x, const float* y, const float* weight, const float* bias, float eps,
+                                  const float* rows, const float* next_weight, const float* next_bias, float next_eps,
+                                  void* out, int tokens, int width, cudaStream_t stream) {
+  if (tokens == 0) return MIR_OK;
+  const size_t smem = 2 * (size_t)width * sizeof(float);
+  if (tokens < 0 || width <= 0 || smem > 200 * 1024 || (out != nullptr && (next_weight == nullptr || next_bias == nullptr))) {
+    mir_set_error("add_layer_norm: bad sizes (tokens %d, width %d)", tokens, width);
+    return MIR_BAD_ARGUMENT;
+  }
+  const bool wide = width % 4 == 0;
+  const int threads = width >= 4096 ? 512 : (width >= 1024 || !wide ? 256 : 128);
+#define MIR_ADD_NORM(T, V)                                                                                             \
+  do {                                                                                                                 \
+    if (smem > 48 * 1024)                                                                                              \
+      cudaFuncSetAttribute(add_layer_norm_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
+    return mir_launch("add_layer_norm", add_layer_norm_kernel<T, V>, dim3(tokens), dim3(threads), smem, stream, 0, x, y, \
+                      weight, bias, eps, rows, next_weight, next_bias, next_eps, (T*)out, width);                      \
+  } while (0)
+  if (bf16) {
+    if (wide) MIR_ADD_NORM(__nv_bfloat16, 4);
+    MIR_ADD_NORM(__nv_bfloat16, 1);
+  }
+  if (wide) MIR_ADD_NORM(float, 4);
+  MIR_ADD_NORM(float, 1);
+#undef MIR_ADD_NORM
 }
 
 // x [tokens, streams, width] in place; y [tokens, width]; mix [streams, streams] indexed [from, to]; write [streams].

@@ -123,6 +123,10 @@ class StepContext(PartContext):
     # rows that the update before left for that reader
     streams_reader_after_block: Optional[tuple] = None
     normed_streams: Optional[torch.Tensor] = None
+    # rows the block that runs now may add to the residual it leaves, and (norm, residual data_ptr, normed rows) that a
+    # block left for the norm the next block starts with
+    rows_after_block: Optional[torch.Tensor] = None
+    normed_residual: Optional[tuple] = None
 
     def alloc(self, shape, dtype: torch.dtype) -> torch.Tensor:
         return self.arena.alloc(shape, dtype)

@@ -284,7 +284,7 @@ class StepRunner:
             rows = len(entries)
             keys = [(e.request_id, 0) for e in entries]
             manager = self.manager
-            if manager.prefix is None and len(manager.groups) == 1 and manager.groups[0].window is None:
+            if manager.prefix is None and len(manager.groups) == 1 and not manager.groups[0].releases:
                 settings = None if options is None else [(s.temperature, s.top_p, s.top_k, s.repetition_penalty)
                                                          for s in samplers]
                 self._again = ([e.request_id for e in entries], list(sequences), graph, keys, settings)
@@ -337,7 +337,7 @@ class StepRunner:
             draws = [s.next_draw() for s in samplers]          # (one per row, as the ordinary path takes them)
         graph.load_again(tokens, sequences, draws)
         graph.replay()
-        for seq in sequences:                                  # (no window to release pages, no prefix to remember)
+        for seq in sequences:                                  # (nothing releases pages, no prefix to remember)
             seq.length += 1
             seq.reserved = max(seq.reserved, seq.length)
         rows = len(ids)

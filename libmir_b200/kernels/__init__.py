@@ -34,7 +34,15 @@ _SIGNATURES = {
         "mir_paged_attention_generic": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
                                         c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_float, c_void_p, c_int,
-                                        c_void_p],
+                                        c_int, c_void_p],
+        "mir_paged_attention_mixed": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                      c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int,
+                                      c_void_p],
+        "mir_selective_scan": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
+                               c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                               c_int, c_int, c_int, c_int, c_void_p],
+        "mir_add_layer_norm": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_float,
+                               c_void_p, c_int, c_int, c_void_p],
         "mir_qk_prepare": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                            c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
         "mir_layer_norm": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
@@ -49,8 +57,8 @@ _SIGNATURES = {
         "mir_gelu_tanh": [c_int, c_void_p, c_size_t, c_void_p],
         "mir_add_normed_branches": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_float,
                                     c_void_p],
-        "mir_short_conv_silu": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        "mir_short_conv_silu": [c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "mir_delta_rule_prepare": [c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
                                    c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                    c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -64,7 +72,8 @@ _SIGNATURES = {
         "mir_add_rows": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "mir_rms_norm_pair": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
         "mir_latent_prepare": [c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
-                               c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_int, c_void_p],
+                               c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p, c_longlong,
+                               c_longlong, c_void_p, c_longlong, c_longlong, c_int, c_int, c_void_p],
         "mir_rope_rows": [c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p,
                           c_float, c_int, c_int, c_int, c_int, c_void_p],
         "mir_sigmoid_gate": [c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p],
@@ -442,25 +451,65 @@ def add_normed_branches(branches, weights, residual: torch.Tensor, eps: float, s
 
 def short_conv_silu(x: torch.Tensor, weight: torch.Tensor, tail: torch.Tensor, row_of_token: torch.Tensor,
                     query_starts: torch.Tensor, state_slots: torch.Tensor, positions: torch.Tensor,
-                    out: torch.Tensor) -> None:
-    """out[t, c] = silu(sum_j weight[c, j] * x[t - (taps - 1) + j, c]) within each request, 32-bit: x is a column
-    range [tokens, channels] of the packed projection (a view with unit column stride), weight [channels, taps] with
-    the current token's tap last, tail [slots, taps - 1, channels] the request's last inputs (32-bit, zero at its
-    start), read for what lies before the portion and then moved on."""
-    _cuda(x, weight, tail, row_of_token, query_starts, state_slots, positions, out)
+                    out: torch.Tensor, bias: Optional[torch.Tensor] = None, single_tokens_only: bool = False) -> None:
+    """out[t, c] = silu(sum_j weight[c, j] * x[t - (taps - 1) + j, c] + bias[c]) within each request, computed in 32-bit
+    and left in x's dtype or in float32: x is a column range [tokens, channels] of the packed projection (a view with
+    unit column stride), weight [channels, taps] with the current token's tap last, bias float32 [channels] or None,
+    tail [slots, taps - 1, channels] the request's last inputs (32-bit, zero at its start), read for what lies before
+    the portion and then moved on.  `single_tokens_only`: every request brings one token."""
+    _cuda(x, weight, tail, row_of_token, query_starts, state_slots, positions, out, bias)
     tokens, channels = x.shape
     taps = weight.shape[1]
     rows = query_starts.numel() - 1
     _require(x.stride(1) == 1 and weight.is_contiguous() and weight.shape[0] == channels and weight.dtype == x.dtype
              and tail.dtype == torch.float32 and tail.is_contiguous() and tail.shape[1:] == (max(taps - 1, 0), channels)
-             and out.dtype == torch.float32 and out.is_contiguous() and out.shape == (tokens, channels),
+             and out.dtype in (x.dtype, torch.float32) and out.is_contiguous() and out.shape == (tokens, channels)
+             and (bias is None or (bias.dtype == torch.float32 and bias.numel() == channels and bias.is_contiguous())),
              "short_conv_silu: shapes or dtypes do not fit")
     _require(all(t.dtype == torch.int32 for t in (row_of_token, query_starts, state_slots, positions)),
              "short_conv_silu: the batch description is int32")
     lib = library("core")
-    _check(lib, lib.mir_short_conv_silu(_is_bf16(x), x.data_ptr(), x.stride(0), weight.data_ptr(), tail.data_ptr(),
-                                        row_of_token.data_ptr(), query_starts.data_ptr(), state_slots.data_ptr(),
-                                        positions.data_ptr(), out.data_ptr(), tokens, rows, channels, taps, _stream()))
+    _check(lib, lib.mir_short_conv_silu(_is_bf16(x), int(out.dtype == torch.float32), x.data_ptr(), x.stride(0),
+                                        weight.data_ptr(), _ptr(bias), tail.data_ptr(), row_of_token.data_ptr(),
+                                        query_starts.data_ptr(), state_slots.data_ptr(), positions.data_ptr(),
+                                        out.data_ptr(), tokens, rows, channels, taps, int(single_tokens_only), _stream()))
+
+
+SELECTIVE_SCAN_MAX_STATE = 256
+
+
+def selective_scan(x: torch.Tensor, raw_step: torch.Tensor, step_bias: torch.Tensor, b: torch.Tensor, c: torch.Tensor,
+                   z: torch.Tensor, rates: torch.Tensor, skip: torch.Tensor, state: torch.Tensor,
+                   query_starts: torch.Tensor, state_slots: torch.Tensor, positions: torch.Tensor,
+                   out: torch.Tensor) -> None:
+    """The selective scan over the tokens of each request row, from and into state [slots, channels, n] (32-bit): with
+    dt = softplus(raw_step + step_bias) per token and channel, S <- 2^(dt * rates) S + dt x b, and out = (sum_n S c +
+    skip * x) * silu(z).  x and z [tokens, channels] and b, c [tokens, columns] (the first n of a row count) are views
+    with unit column stride in the activations' dtype, b and c with one row stride; raw_step [tokens, channels],
+    step_bias and skip [channels] and rates [channels, n] (at most zero: A log2 e) are float32; out [tokens, channels]
+    in the activations' dtype.  channels and columns are multiples of 8; rows start on 16-byte boundaries."""
+    _cuda(x, raw_step, step_bias, b, c, z, rates, skip, state, query_starts, state_slots, positions, out)
+    tokens, channels = x.shape
+    n = rates.shape[1]
+    rows = query_starts.numel() - 1
+    _require(z.shape == x.shape and b.shape == c.shape and b.shape[0] == tokens and b.shape[1] >= n
+             and all(t.dtype == x.dtype and t.stride(1) == 1 for t in (x, z, b, c)) and b.stride(0) == c.stride(0)
+             and out.dtype == x.dtype and out.is_contiguous() and out.shape == x.shape,
+             "selective_scan: x, z, b, c and out share a dtype and have unit column strides")
+    for tensor, shape in ((raw_step, (tokens, channels)), (step_bias, (channels,)), (rates, (channels, n)),
+                          (skip, (channels,))):
+        _require(tensor.dtype == torch.float32 and tensor.is_contiguous() and tensor.shape == shape,
+                 "selective_scan: raw_step, step_bias, rates and skip are contiguous float32 of the stated shapes")
+    _require(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (channels, n),
+             "selective_scan: the state is float32 [slots, channels, n]")
+    _require(all(t.dtype == torch.int32 for t in (query_starts, state_slots, positions)),
+             "selective_scan: the batch description is int32")
+    lib = library("core")
+    _check(lib, lib.mir_selective_scan(_is_bf16(x), x.data_ptr(), x.stride(0), raw_step.data_ptr(), step_bias.data_ptr(),
+                                       b.data_ptr(), c.data_ptr(), b.stride(0), z.data_ptr(), z.stride(0), rates.data_ptr(),
+                                       skip.data_ptr(), state.data_ptr(), query_starts.data_ptr(), state_slots.data_ptr(),
+                                       positions.data_ptr(), out.data_ptr(), tokens, rows, channels, n, b.shape[1],
+                                       _stream()))
 
 
 def delta_rule_prepare(x: torch.Tensor, weight: torch.Tensor, tail: torch.Tensor, beta_raw: torch.Tensor,
@@ -620,19 +669,28 @@ def rms_norm_pair(x: torch.Tensor, weight_a: torch.Tensor, weight_b: torch.Tenso
 
 # --------------------------------------------------------------------------- latent attention
 def latent_prepare(packed: torch.Tensor, q_offset: int, q_rank: int, kv_offset: int, kv_rank: int, rotary_dim: int,
-                   q_norm: torch.Tensor, kv_norm: torch.Tensor, eps: float, positions: torch.Tensor,
+                   q_norm: Optional[torch.Tensor], kv_norm: torch.Tensor, eps: float, positions: torch.Tensor,
                    slot_mapping: Optional[torch.Tensor], inv_freq: Optional[torch.Tensor], magnitude: float,
-                   interleaved: bool, latent_q: torch.Tensor, pages: Optional[torch.Tensor]) -> None:
+                   interleaved: bool, latent_q: Optional[torch.Tensor], pages: Optional[torch.Tensor],
+                   turn: Optional[tuple] = None) -> None:
     """Per token of the packed projection `packed` [tokens, >= offsets + widths]: latent_q = rmsnorm(packed[q_offset :
     + q_rank]) * q_norm; the token's cache row pages[slot] = [rmsnorm(packed[kv_offset : + kv_rank]) * kv_norm | the
     rotary_dim columns behind it rotated by the token's position].  Norms and angles are 32-bit.  A token whose slot
-    is negative (or with slot_mapping None) writes no cache row."""
+    is negative (or with slot_mapping None) writes no cache row.  With q_rank 0 there is no query latent (q_norm and
+    latent_q are None); `turn` = (source, target), views [tokens, heads, rotary_dim] with unit stride in the last
+    dimension: the source's rows rotated by their token's position go to the target in the same launch."""
     _cuda(packed, q_norm, kv_norm, positions, slot_mapping, inv_freq, latent_q, pages)
     tokens = packed.shape[0]
+    source, target = turn if turn is not None else (None, None)
     _require(packed.stride(1) == 1 and q_offset + q_rank <= packed.shape[1]
-             and kv_offset + kv_rank + rotary_dim <= packed.shape[1] and latent_q.dtype == packed.dtype
-             and latent_q.is_contiguous() and latent_q.shape == (tokens, q_rank)
-             and q_norm.dtype == torch.float32 and q_norm.numel() == q_rank and kv_norm.dtype == torch.float32
+             and kv_offset + kv_rank + rotary_dim <= packed.shape[1]
+             and (q_rank == 0 or (latent_q.dtype == packed.dtype and latent_q.is_contiguous()
+                                  and latent_q.shape == (tokens, q_rank) and q_norm.dtype == torch.float32
+                                  and q_norm.numel() == q_rank))
+             and (turn is None or (rotary_dim > 0 and all(t.dim() == 3 and t.shape == (tokens, source.shape[1], rotary_dim)
+                                                          and t.stride(2) == 1 and t.dtype == packed.dtype and t.is_cuda
+                                                          for t in turn)))
+             and kv_norm.dtype == torch.float32
              and kv_norm.numel() == kv_rank and positions.dtype == torch.int32 and positions.numel() >= tokens,
              "latent_prepare: shapes or dtypes do not fit")
     if slot_mapping is not None:
@@ -644,9 +702,13 @@ def latent_prepare(packed: torch.Tensor, q_offset: int, q_rank: int, kv_offset: 
                  "latent_prepare: the angle table must hold rotary_dim / 2 float32 values")
     lib = library("core")
     _check(lib, lib.mir_latent_prepare(_is_bf16(packed), packed.data_ptr(), packed.stride(0), q_offset, q_rank, kv_offset,
-                                       kv_rank, rotary_dim, q_norm.data_ptr(), kv_norm.data_ptr(), eps,
+                                       kv_rank, rotary_dim, _ptr(q_norm), kv_norm.data_ptr(), eps,
                                        positions.data_ptr(), _ptr(slot_mapping), _ptr(inv_freq), float(magnitude),
-                                       int(interleaved), latent_q.data_ptr(), _ptr(pages), tokens, _stream()))
+                                       int(interleaved), _ptr(latent_q), _ptr(pages), _ptr(source),
+                                       source.stride(0) if turn is not None else 0, source.stride(1) if turn is not None else 0,
+                                       _ptr(target), target.stride(0) if turn is not None else 0,
+                                       target.stride(1) if turn is not None else 0,
+                                       source.shape[1] if turn is not None else 0, tokens, _stream()))
 
 
 def rope_rows(src: torch.Tensor, dst: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, magnitude: float,
@@ -1024,6 +1086,28 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
                                    out.data_ptr(), _ptr(rows), n_rows, width, eps, _stream()))
 
 
+def add_layer_norm(residual: torch.Tensor, branch: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float,
+                   rows: Optional[torch.Tensor] = None, next_weight: Optional[torch.Tensor] = None,
+                   next_bias: Optional[torch.Tensor] = None, next_eps: float = 0.0,
+                   out: Optional[torch.Tensor] = None) -> None:
+    """residual += layer_norm(branch; weight, bias, eps) (+ rows), all float32 [tokens, width]; with `out` (bfloat16 or
+    float32), in the same pass over a token, out = layer_norm(residual; next_weight, next_bias, next_eps) of the rows as
+    the addition leaves them."""
+    _cuda(residual, branch, weight, bias, rows, next_weight, next_bias, out)
+    tokens, width = residual.shape
+    _require(all(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == residual.shape)
+                 for t in (residual, branch, rows))
+             and all(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == width)
+                     for t in (weight, bias, next_weight, next_bias))
+             and (out is None or (out.is_contiguous() and out.shape == residual.shape and next_weight is not None
+                                  and next_bias is not None and out.dtype in (torch.bfloat16, torch.float32))),
+             "add_layer_norm: bad arguments")
+    lib = library("core")
+    _check(lib, lib.mir_add_layer_norm(int(out is not None and out.dtype == torch.bfloat16), residual.data_ptr(),
+                                       branch.data_ptr(), weight.data_ptr(), bias.data_ptr(), eps, _ptr(rows),
+                                       _ptr(next_weight), _ptr(next_bias), next_eps, _ptr(out), tokens, width, _stream()))
+
+
 def streams_write(streams: torch.Tensor, branch: torch.Tensor, mix: torch.Tensor, write: torch.Tensor) -> None:
     """A residual of S streams [tokens, S, width] takes a sublayer's result `branch` [tokens, width], in place and all
     streams at once from the old ones: x_t <- sum_s mix[s, t] x_s + write[t] * branch.  All 32-bit."""
@@ -1252,7 +1336,8 @@ def paged_attention_generic(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
                             window: Optional[int], value_dim: Optional[int] = None, keep_first: int = 0,
                             values_in_keys: bool = False, sinks: Optional[torch.Tensor] = None,
                             gate: Optional[torch.Tensor] = None, gate_per_head: bool = False,
-                            softcap: Optional[float] = None, distance_bias: Optional[torch.Tensor] = None) -> None:
+                            softcap: Optional[float] = None, distance_bias: Optional[torch.Tensor] = None,
+                            chunk: Optional[int] = None) -> None:
     """out[t, h] = softmax over the visible cached keys of token t's request; q is read from the packed qkv rows.
     `value_dim`: width of a value head (head_dim if None); `keep_first`: with a window, the request's first keys
     that stay visible to every query; `values_in_keys`: a value is the first value_dim elements of its key (a cached
@@ -1260,7 +1345,8 @@ def paged_attention_generic(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
     denominator of head h's softmax.  `gate` ([tokens, heads * value_dim] view, unit column stride, out's dtype): the
     result is multiplied by its sigmoid; with `gate_per_head` it is [tokens, heads], one number per head.  `softcap`:
     score <- softcap * tanh(score / softcap) after the scale.  `distance_bias` (float32 [heads, rows]): row
-    min(query position - key position, rows - 1) is added to the scores after the cap."""
+    min(query position - key position, rows - 1) is added to the scores after the cap.  `chunk`: positions are cut into
+    runs of that many, and a query sees the keys of its own run only."""
     if values_in_keys:
         v_pages = k_pages
     _cuda(qkv, out, k_pages, v_pages, block_table, row_of_token, positions, sinks, gate, distance_bias)
@@ -1286,7 +1372,47 @@ def paged_attention_generic(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
         page_size, heads, kv_heads, head_dim, value_dim, scale, int(window or 0), int(keep_first or 0),
         head_dim if values_in_keys else 0, _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0,
         int(gate_per_head), float(softcap or 0.0), _ptr(distance_bias),
-        distance_bias.shape[1] if distance_bias is not None else 0, _stream()))
+        distance_bias.shape[1] if distance_bias is not None else 0, int(chunk or 0), _stream()))
+
+
+MIXED_TENSOR_CORES = True        # False: attention with mixed heads always runs the reference kernel
+
+
+def _check_mixed(what: str, qkv, out, k_pages, v_pages, block_table, head_mix, heads, kv_heads, dim, value_dim) -> None:
+    _cuda(qkv, out, k_pages, v_pages, block_table, head_mix)
+    _require(out.is_contiguous() and out.shape[1] == heads * value_dim and qkv.stride(1) == 1 and qkv.shape[1] >= heads * dim
+             and qkv.dtype == out.dtype and k_pages.dtype == out.dtype and v_pages.dtype == out.dtype
+             and k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.shape[1:] == (kv_heads, dim)
+             and v_pages.shape[1:] == (kv_heads, value_dim), f"{what}: bad tensors")
+    _require(block_table.dtype == torch.int32 and block_table.dim() == 2 and block_table.is_contiguous(), f"{what}: bad metadata")
+    _require(head_mix.dtype == torch.float32 and head_mix.is_contiguous() and head_mix.shape == (heads, heads),
+             f"{what}: the heads' mixing matrix is float32 [heads, heads]")
+
+
+def paged_attention_mixed(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
+                          block_table: torch.Tensor, row_of_token: torch.Tensor, positions: torch.Tensor, page_size: int,
+                          heads: int, kv_heads: int, dim: int, value_dim: int, scale: float, head_mix: torch.Tensor,
+                          window: Optional[int] = None, chunk: Optional[int] = None) -> None:
+    """out[t, h] = sum_j (sum_g head_mix[h, g] w_g(t, j)) v(j): every head's softmax weights over the visible cached keys
+    of token t's request (all up to its position, the last `window`, those of its own run of `chunk` positions), mixed
+    over the heads, applied to the values of head h's kv head.  The reference kernel: any sizes, both dtypes."""
+    _check_mixed("paged_attention_mixed", qkv, out, k_pages, v_pages, block_table, head_mix, heads, kv_heads, dim, value_dim)
+    _require(row_of_token.dtype == torch.int32 and positions.dtype == torch.int32, "paged_attention_mixed: bad metadata")
+    lib = library("core")
+    _check(lib, lib.mir_paged_attention_mixed(
+        _is_bf16(out), qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(),
+        block_table.data_ptr(), block_table.shape[1], row_of_token.data_ptr(), positions.data_ptr(), out.shape[0], page_size,
+        heads, kv_heads, dim, value_dim, scale, head_mix.data_ptr(), int(window or 0), int(chunk or 0), _stream()))
+
+
+def mixed_decode_takes(heads: int, kv_heads: int, dim: int, value_dim: int) -> bool:
+    """Whether single tokens of these sizes run the split-key kernels for mixed heads (bfloat16 only)."""
+    return False
+
+
+def mixed_prefill_takes(heads: int, dim: int, value_dim: int) -> bool:
+    """Whether prompt portions of these sizes run the tile kernels for mixed heads (bfloat16 only)."""
+    return False
 
 
 def _check_extras(what: str, sinks, gate, out: torch.Tensor, heads: int, gate_per_head: bool = False,

@@ -44,7 +44,7 @@ class DecoderModel:
         self.loop_steps: Optional[torch.Tensor] = None          # [passes, hidden] 32-bit: what each pass of a loop adds
         self.head: Optional[torch.Tensor] = None
         self._runs_key, self._runs_list, self._native = None, [], {}
-        self.after_entry = None      # for inspection: called with (schedule index, streams) after every run of a layer
+        self.after_entry = None      # for inspection: called with (schedule index, residual) after every run of a layer
 
     # -- what the cache manager must provide ------------------------------------
     def cache_plan(self) -> List[CacheEntryPlan]:
@@ -150,6 +150,11 @@ class DecoderModel:
         total += self.final_norm.weight_bytes() + self.head.numel() * self.head.element_size()
         return total
 
+    def pass_adds(self, entry) -> bool:
+        """Whether the pass that starts with `entry` (if one does) adds anything to the residual."""
+        return entry.opens_pass is not None and (self.loop_steps is not None
+                                                 or (self.spec.loop.add_embedding and entry.opens_pass > 0))
+
     def open_pass(self, ctx, entry, residual: torch.Tensor, embedded: Optional[torch.Tensor]) -> None:
         """What a pass of the model's loop starts with: every pass but the first adds the embedding's output to the
         residual, every pass adds its row of the step tensor."""
@@ -179,25 +184,40 @@ class DecoderModel:
             embedded = ctx.alloc(tuple(residual.shape), torch.float32)       # later passes add the embedding's output again
             embedded.copy_(residual)
         ctx.rounded_residual = None          # (a block leaves one only for the block right behind it, which takes it)
+        ctx.normed_residual = None
+        opened = None                        # the entry whose pass the block before it has opened
         for run in self._runs(ctx):
             if run.layers is not None:
                 run.execute(ctx, residual)
                 continue
             index = run.first
             entry = spec.schedule[index]
-            if entry.opens_pass is not None:
+            if entry.opens_pass is not None and opened != index:
                 self.open_pass(ctx, entry, residual, embedded)
             # the norm that the next block in the schedule starts with: this block's last product may prepare it
             following = self.blocks[spec.schedule[index + 1].layer] if index + 1 < len(spec.schedule) else None
             ctx.norm_after_block = following.first_norm() if following is not None else None
-            if index + 1 < len(spec.schedule) and (self._native.get(index + 1) is not None
-                                                   or spec.schedule[index + 1].opens_pass is not None):
+            ctx.rows_after_block = self.rows_before(index + 1, self.blocks[entry.layer], embedded)
+            if ctx.rows_after_block is not None:
+                opened = index + 1
+            elif index + 1 < len(spec.schedule) and (self._native.get(index + 1) is not None
+                                                     or self.pass_adds(spec.schedule[index + 1])):
                 ctx.norm_after_block = None          # the next block starts from a residual that this one has not seen
             ctx.next_reads_residual = (following is not None and getattr(following, "reads_residual_itself", False)
                                        and self._native.get(index + 1) is None
                                        and spec.schedule[index + 1].opens_pass is None)
             self.blocks[entry.layer].forward(ctx, ctx.cache_view(index), residual)
+            if self.after_entry is not None:
+                self.after_entry(index, residual)
         return residual
+
+    def rows_before(self, index: int, block, embedded: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
+        """What opens the pass that starts with schedule entry `index`, if `block`, which runs right before it, can add it
+        in its own update of the residual (the embedding's rows alone, and nobody looks at the residual in between)."""
+        if index >= len(self.spec.schedule) or self.after_entry is not None or self.loop_steps is not None \
+                or not getattr(block, "adds_rows_after", False) or self._native.get(index) is not None:
+            return None
+        return embedded if self.pass_adds(self.spec.schedule[index]) else None
 
     def forward_streams(self, ctx) -> torch.Tensor:
         """A residual kept as several streams [T, S, H]: every stream starts as the embedding's output, the blocks (of

@@ -13,7 +13,10 @@ cache of the schedule entry that its own entry names).  Further forms, also from
 the design (fixed_sink), a gate with one number per head (gate_per_head), a q/k norm over all heads of the projection
 at once, a norm without weights or one that follows the rotation (these run the kernel of csrc/qk_prepare.cu), scores
 capped by softcap * tanh(score / softcap), and a stored bias by the bucket of the distance between query and key (the
-table is spread out to one row per distance when the weights are bound).
+table is spread out to one row per distance when the weights are bound).  Positions cut into runs (`chunk`): a query
+sees the keys of its own run only.  Mixed heads (head_mix, a stored matrix M over the query heads): head h applies
+sum_g M[h, g] weights_g, the combination of all heads' softmax weights, to the values of its own kv head
+(csrc/attention_mixed.cu, csrc/attention_mixed_mma.cu).
 """
 
 from __future__ import annotations
@@ -61,7 +64,12 @@ class SoftmaxAttention(Mixer):
         if self.other_norm and not s.own_kv:
             raise ValueError("these q/k norms need keys of the mixer's own")
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = self.q_norm = self.k_norm = self.sinks = None
-        self.distance_bias = None
+        self.distance_bias = self.head_mix = None
+        if s.head_mix and (s.keep_first or s.sinks or s.fixed_sink is not None or s.gate or s.softcap is not None
+                           or s.distance_bias is not None):
+            raise ValueError("mixed heads go with plain scores: no sinks, gate, cap, bias or kept first tokens")
+        if s.chunk is not None and s.keep_first:
+            raise ValueError("runs of positions do not go with kept first tokens")
         if s.fixed_sink is not None:
             self.sinks = torch.full((s.heads,), float(s.fixed_sink), dtype=torch.float32, device=env.device)
 
@@ -72,7 +80,7 @@ class SoftmaxAttention(Mixer):
     def cache_requirement(self):
         s = self.spec
         return PagedKv(s.kv_heads, s.head_dim, s.window, s.value_head_dim if s.value_dim != s.head_dim else None,
-                       s.keep_first if s.window is not None else 0)
+                       s.keep_first if s.window is not None else 0, s.chunk)
 
     # names under which checkpoints store query, key and value as one row-stacked tensor [Wq; Wk; Wv]
     # (models/src/weights/binding/roles/parse.rs: "self_attn.qkv_proj.weight" | "self_attn.query_key_value.weight")
@@ -109,6 +117,8 @@ class SoftmaxAttention(Mixer):
         if s.distance_bias is not None:
             table["rel_bias"] = ParamSpec((s.distance_bias.rows, s.heads), init="normal", store="float32",
                                           accept_transposed=False)
+        if s.head_mix:
+            table["head_mix"] = ParamSpec((s.heads, s.heads), store="float32", accept_transposed=False)
         if s.sinks:
             table["sinks"] = ParamSpec((s.heads,), init="zeros", store="float32")
         return {self.stored.get(local, local): param for local, param in table.items()}
@@ -142,6 +152,8 @@ class SoftmaxAttention(Mixer):
         if self.spec.fixed_sink is not None:
             self.sinks = torch.full((self.spec.heads,), float(self.spec.fixed_sink), dtype=torch.float32,
                                     device=self.w_o.device)
+        if self.spec.head_mix:
+            self.head_mix = tensors["head_mix"].contiguous()
         if self.spec.distance_bias is not None:
             self.distance_bias = self.bias_by_distance(tensors["rel_bias"].float())
 
@@ -169,7 +181,7 @@ class SoftmaxAttention(Mixer):
 
     def weight_bytes(self):
         return sum(t.numel() * t.element_size() for t in (self.w_qkv, self.w_o, self.b_qkv, self.b_o, self.sinks,
-                                                          self.distance_bias) if t is not None)
+                                                          self.distance_bias, self.head_mix) if t is not None)
 
     def forward(self, ctx, cache, x, residual, overwrite=False):
         """residual += attention(x) W_o^T; with `overwrite` the result replaces `residual` (a 32-bit buffer of a
@@ -242,11 +254,15 @@ class SoftmaxAttention(Mixer):
         bfloat16 with head_dim 64 or 128 runs on tensor cores (split over the keys when every row is a
         single decoded token), everything else runs the reference kernel."""
         s = self.spec
+        if s.head_mix:
+            self.attend_mixed(ctx, group, cache, qkv, out)
+            return
         kept = s.keep_first if s.window is not None else 0
         first = self.q_width + self.kv_columns
         gate = qkv[:, first:first + self.gate_width] if s.gate else None        # [tokens, heads * value_dim] or [tokens, heads]
         scored = s.softcap is not None or self.distance_bias is not None or s.gate_per_head
-        fast = self.env.dtype == torch.bfloat16 and s.head_dim in kernels.FAST_HEAD_DIMS and s.value_dim == s.head_dim
+        fast = self.env.dtype == torch.bfloat16 and s.head_dim in kernels.FAST_HEAD_DIMS and s.value_dim == s.head_dim \
+            and s.chunk is None                  # (runs of positions without mixed heads: the reference kernel)
         if fast and scored and not kept:
             # capped or biased scores, or a gate per head: single tokens split over the keys, portions as tiles of
             # queries, each on the tcgen05 or the mma.sync kernel by size
@@ -314,4 +330,34 @@ class SoftmaxAttention(Mixer):
                                         s.window, value_dim=s.value_dim,
                                         keep_first=s.keep_first if s.window is not None else 0, sinks=self.sinks,
                                         gate=gate, gate_per_head=s.gate_per_head, softcap=s.softcap,
-                                        distance_bias=self.distance_bias)
+                                        distance_bias=self.distance_bias, chunk=s.chunk)
+
+    def attend_mixed(self, ctx, group, cache, qkv, out):
+        """Attention whose heads' weights are mixed: a key's weight in one head needs its weight in all of them, so the
+        softmax comes first.  bfloat16: single tokens split over the keys (scores, then weights and values, then the
+        sum of the parts), portions as tiles (the rows' log-sums, the mixed weights, the products with the values);
+        32-bit and sizes those kernels refuse: the reference kernel."""
+        s = self.spec
+        singles = ctx.num_rows if ctx.decode_only else ctx.single_rows
+        fast = self.env.dtype == torch.bfloat16 and kernels.MIXED_TENSOR_CORES
+        decode = fast and kernels.mixed_decode_takes(s.heads, s.kv_heads, s.head_dim, s.value_dim)
+        tiles = fast and kernels.mixed_prefill_takes(s.heads, s.head_dim, s.value_dim)
+        done = 0
+        if decode and singles:
+            longest = ctx.max_context if ctx.decode_only else ctx.single_context
+            kernels.mixed_decode_attention(qkv[:singles], out[:singles], cache.k_pages, cache.v_pages,
+                                           group.block_table[:singles], ctx.positions, cache.page_size, s.heads, s.kv_heads,
+                                           s.head_dim, s.value_dim, s.scale, self.head_mix, s.window, s.chunk, longest,
+                                           ctx.alloc)
+            done = singles
+        if tiles and done == singles and singles < ctx.num_rows:
+            kernels.mixed_prefill_attention(qkv, out, cache.k_pages, cache.v_pages, group.block_table[singles:],
+                                            ctx.query_starts[singles:], ctx.context_lens[singles:], cache.page_size,
+                                            s.heads, s.kv_heads, s.head_dim, s.value_dim, s.scale, self.head_mix, s.window,
+                                            s.chunk, out.shape[0] - singles, ctx.max_context, ctx.alloc)
+            return
+        if done == out.shape[0]:
+            return
+        kernels.paged_attention_mixed(qkv[done:], out[done:], cache.k_pages, cache.v_pages, group.block_table,
+                                      ctx.row_of_token[done:], ctx.positions[done:], cache.page_size, s.heads, s.kv_heads,
+                                      s.head_dim, s.value_dim, s.scale, self.head_mix, s.window, s.chunk)

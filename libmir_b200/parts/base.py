@@ -66,6 +66,11 @@ class PartContext:
     `rounded_residual`, and the next block takes it (`take_rounded`) instead of casting."""
 
     dtype: Optional[torch.dtype] = None
+    # An arrangement that updates the residual in a kernel of its own can norm it there for the next block's first norm
+    # (`norm_after_block`) and add further rows to it (`rows_after_block`: what a repeated run of layers adds before
+    # its next pass): the block leaves the normed rows, the next one takes them.
+    rows_after_block = None
+    normed_residual = None
     upcoming_norm = None
     norm_after_block = None
     residual_stats = None
@@ -75,6 +80,16 @@ class PartContext:
     # block (set by the model, None at the end), and the normed rows the block before left for it.
     streams_reader_after_block = None
     normed_streams = None
+
+    def leave_normed(self, norm, residual: torch.Tensor, rows: Optional[torch.Tensor]) -> None:
+        self.normed_residual = (norm, residual.data_ptr(), rows) if rows is not None else None
+
+    def take_normed(self, norm, residual: torch.Tensor) -> Optional[torch.Tensor]:
+        """What the block before left for `norm`: the normed rows of this very residual, or None."""
+        left, self.normed_residual = self.normed_residual, None
+        if left is not None and left[0] is norm and left[1] == residual.data_ptr() and left[2].shape == residual.shape:
+            return left[2]
+        return None
 
     def take_rounded(self, residual: torch.Tensor) -> torch.Tensor:
         """The residual in the engine dtype: the copy the block before left, if it left one, else a cast."""

@@ -17,6 +17,11 @@ Each branch reads the residual itself (cast to the engine's dtype) and its RESUL
 writes its result into a 32-bit buffer, and one kernel norms that buffer and adds m times it into the residual, so
 the norm and the residual sum are 32-bit.  m is LayerSpec.residual_scale.
 
+sandwich:  x += norm_1b(mixer(norm_1(x)));  x += norm_2b(feed_forward(norm_2(x)))
+A norm before and a norm behind each branch.  The branch writes its result into a 32-bit buffer; where the norms are
+layer norms one kernel norms that buffer, adds it to the residual and, in the same pass over a token, norms the new
+residual for whoever reads it next (this block's feed-forward or the next block's mixer).
+
 streams:  the residual is S copies x_1 .. x_S per token (hyper-connections).  For each of the two sublayers, with its
 stored mixing tensors in [S], mix [S, S] and out [S]:  u = sum_s in[s] x_s;  y = sublayer(norm(u));  then all streams
 at once from the old ones, x_t <- sum_s mix[s, t] x_s + out[t] y.  Everything outside the sublayer is 32-bit: the
@@ -236,6 +241,66 @@ class OutputNormBlock(Block):
         ctx.residual_stats = None
 
 
+class SandwichBlock(Block):
+    """x += norm_1b(mixer(norm_1(x))), then x += norm_2b(feed_forward(norm_2(x))): norms around both branches."""
+
+    adds_rows_after = True               # it can add further rows to the residual it leaves (PartContext.rows_after_block)
+
+    SLOTS = ("mixer_norm", "mixer", "mixer_out_norm", "feed_forward_norm", "feed_forward", "feed_forward_out_norm")
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        for slot in self.SLOTS:
+            setattr(self, slot, build_part(getattr(spec, slot), env))
+        if self.mixer_norm is None or self.mixer_out_norm is None or \
+                (self.feed_forward is not None and (self.feed_forward_norm is None or self.feed_forward_out_norm is None)):
+            raise ValueError("the sandwich arrangement takes a norm before and a norm behind every branch")
+
+    def parts(self):
+        return [(slot, getattr(self, slot)) for slot in self.SLOTS if getattr(self, slot) is not None]
+
+    def cache_requirement(self):
+        return self.mixer.cache_requirement()
+
+    def first_norm(self):
+        return self.mixer_norm
+
+    def forward(self, ctx, cache, residual):
+        after, rows_after = ctx.norm_after_block, ctx.rows_after_block
+        ctx.upcoming_norm = None             # the branches' results go through a norm of their own, not into the residual
+        ctx.residual_stats = None
+        x = ctx.take_normed(self.mixer_norm, residual)
+        if x is None:
+            x = self.mixer_norm.forward(ctx, residual)
+        result = ctx.alloc(tuple(residual.shape), torch.float32)
+        self.mixer.forward(ctx, cache, x, result, overwrite=True)
+        if self.feed_forward is not None:
+            x = self._add(ctx, residual, result, self.mixer_out_norm, None, self.feed_forward_norm)
+            self.feed_forward.forward(ctx, x, result, overwrite=True)
+            out_norm = self.feed_forward_out_norm
+        else:
+            out_norm = self.mixer_out_norm
+        ctx.leave_normed(after, residual, self._add(ctx, residual, result, out_norm, rows_after, after))
+        ctx.residual_stats = None
+
+    def _add(self, ctx, residual, result, norm, rows, reader):
+        """residual += norm(result) (+ rows); returns reader(residual) in the engine dtype, or None without a reader."""
+        from .. import kernels
+        from .norm import LayerNorm
+        out = ctx.alloc(tuple(residual.shape), self.env.dtype) if reader is not None else None
+        if type(norm) is LayerNorm and (reader is None or type(reader) is LayerNorm):
+            kernels.add_layer_norm(residual, result, norm.weight, norm.bias, norm.spec.eps, rows,
+                                   reader.weight if reader is not None else None,
+                                   reader.bias if reader is not None else None,
+                                   reader.spec.eps if reader is not None else 0.0, out)
+            return out
+        normed = norm.forward(ctx, result, out=ctx.alloc(tuple(residual.shape), torch.float32))
+        kernels.add_rows(residual, normed, None)
+        if rows is not None:
+            kernels.add_rows(residual, rows, None)
+        return reader.forward(ctx, residual, out=out) if reader is not None else None
+
+
 class StreamMix(Part):
     """The three small tensors by which one sublayer reads and writes a residual of several streams."""
 
@@ -324,7 +389,7 @@ class StreamsBlock(Block):
 
 
 ARRANGEMENTS = {"pre_norm": PreNormBlock, "parallel": ParallelBlock, "output_norm": OutputNormBlock,
-                "streams": StreamsBlock}
+                "sandwich": SandwichBlock, "streams": StreamsBlock}
 
 
 def build_block(layer_spec, env):

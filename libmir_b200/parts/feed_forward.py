@@ -21,29 +21,38 @@ class SwiGlu(FeedForward):
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
+        self.stored = dict(spec.names)           # local name -> the name the checkpoint uses
         self.w_gate_up = self.w_down = None
 
     def parameters(self):
         s = self.spec
-        return {
+        table = {
             "gate_proj.weight": ParamSpec((s.intermediate_size, s.hidden_size)),
             "up_proj.weight": ParamSpec((s.intermediate_size, s.hidden_size)),
             "down_proj.weight": ParamSpec((s.hidden_size, s.intermediate_size)),
         }
+        return {self.stored.get(local, local): param for local, param in table.items()}
 
     def bind(self, tensors):
+        local_of = {stored: local for local, stored in self.stored.items()}
+        tensors = {local_of.get(name, name): tensor for name, tensor in tensors.items()}
         self.w_gate_up = torch.cat([tensors["gate_proj.weight"], tensors["up_proj.weight"]], dim=0)
         self.w_down = tensors["down_proj.weight"].contiguous()
 
     def weight_bytes(self):
         return (self.w_gate_up.numel() + self.w_down.numel()) * self.w_down.element_size()
 
-    def forward(self, ctx, x, residual):
+    def forward(self, ctx, x, residual, overwrite=False):
+        """residual += down(silu(gate(x)) * up(x)); with `overwrite` the result replaces `residual` (a 32-bit buffer of
+        an arrangement that norms the branch's result) instead of being added to it."""
         s = self.spec
         tokens = x.shape[0]
         hidden = ctx.alloc((tokens, s.intermediate_size), self.env.dtype)
         kernels.gate_up_silu(x, self.w_gate_up, hidden, ctx.alloc)
-        ctx.accumulate(hidden, self.w_down, residual)      # may also prepare the norm that follows
+        if overwrite:
+            kernels.linear(hidden, self.w_down, residual, alloc=ctx.alloc)
+        else:
+            ctx.accumulate(hidden, self.w_down, residual)      # may also prepare the norm that follows
 
 
 class GeluMlp(FeedForward):
