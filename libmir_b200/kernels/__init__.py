@@ -186,6 +186,14 @@ _SIGNATURES = {
         "mir_latent_attention_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int,
                                       c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p,
                                       c_void_p],
+        "mir_mixed_prefill_takes": [c_int, c_int, c_int],
+        "mir_mixed_prefill_attention_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
+                                             c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
+        "mir_mixed_decode_takes": [c_int, c_int, c_int, c_int],
+        "mir_mixed_decode_attention_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                            c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int,
+                                            c_void_p, c_void_p, c_void_p, c_void_p],
         "mir_set_option": [ctypes.c_char_p, c_int],
         "mir_get_option": [ctypes.c_char_p],
         "mir_gemm_bf16_lt_batched": [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_int,
@@ -1407,12 +1415,71 @@ def paged_attention_mixed(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.T
 
 def mixed_decode_takes(heads: int, kv_heads: int, dim: int, value_dim: int) -> bool:
     """Whether single tokens of these sizes run the split-key kernels for mixed heads (bfloat16 only)."""
-    return False
+    return bool(library("bf16").mir_mixed_decode_takes(heads, kv_heads, dim, value_dim))
 
 
 def mixed_prefill_takes(heads: int, dim: int, value_dim: int) -> bool:
     """Whether prompt portions of these sizes run the tile kernels for mixed heads (bfloat16 only)."""
-    return False
+    return bool(library("bf16").mir_mixed_prefill_takes(heads, dim, value_dim))
+
+
+def _visible_span(longest: int, window: Optional[int], chunk: Optional[int]) -> int:
+    """The most keys a query of a request with `longest` tokens sees."""
+    return max(1, min(reach for reach in (longest, window, chunk) if reach))
+
+
+def mixed_decode_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
+                           block_table: torch.Tensor, positions: torch.Tensor, page_size: int, heads: int, kv_heads: int,
+                           dim: int, value_dim: int, scale: float, head_mix: torch.Tensor, window: Optional[int],
+                           chunk: Optional[int], longest: int, alloc) -> None:
+    """paged_attention_mixed for a batch of single tokens (row r of qkv belongs to request row r, none of which has more
+    than `longest` tokens), bfloat16, the keys in parts of 64 over CTAs: scores, weights and values, sum of the parts."""
+    _check_mixed("mixed_decode_attention", qkv, out, k_pages, v_pages, block_table, head_mix, heads, kv_heads, dim, value_dim)
+    rows = out.shape[0]
+    _require(out.dtype == torch.bfloat16 and positions.dtype == torch.int32 and positions.numel() >= rows
+             and block_table.shape[0] >= rows, "mixed_decode_attention: bad metadata")
+    parts = -(-_visible_span(longest, window, chunk) // 64)
+    scores = alloc((rows, heads, parts * 64), torch.float32)
+    stats = alloc((rows, heads, parts, 2), torch.float32)
+    partial = alloc((rows, parts, heads, value_dim), torch.float32)
+    lib = library("bf16")
+    _check(lib, lib.mir_mixed_decode_attention_bf16(
+        qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
+        block_table.shape[1], positions.data_ptr(), rows, page_size, heads, kv_heads, dim, value_dim, scale,
+        head_mix.data_ptr(), int(window or 0), int(chunk or 0), parts, scores.data_ptr(), stats.data_ptr(),
+        partial.data_ptr(), _stream()))
+
+
+MIXED_SLAB_BYTES = 256 << 20     # how much of the mixed weights of a prompt is in memory at a time
+MIXED_SEGMENT_TILES = 4          # tiles of 64 keys that a CTA of the mixing kernel goes through
+
+
+def mixed_prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
+                            block_table: torch.Tensor, query_starts: torch.Tensor, context_lens: torch.Tensor,
+                            page_size: int, heads: int, kv_heads: int, dim: int, value_dim: int, scale: float,
+                            head_mix: torch.Tensor, window: Optional[int], chunk: Optional[int], portion_tokens: int,
+                            longest: int, alloc) -> None:
+    """paged_attention_mixed for any mix of portions (row r owns the tokens query_starts[r] .. query_starts[r + 1] of qkv
+    and out; the rows may be a part of the batch, with portion_tokens tokens together and at most `longest` tokens each),
+    bfloat16, on tensor cores: the rows' log-sums, the mixed weights, the products with the values."""
+    _check_mixed("mixed_prefill_attention", qkv, out, k_pages, v_pages, block_table, head_mix, heads, kv_heads, dim, value_dim)
+    rows, tokens = context_lens.numel(), out.shape[0]
+    _require(out.dtype == torch.bfloat16 and query_starts.dtype == torch.int32 and context_lens.dtype == torch.int32
+             and query_starts.numel() == rows + 1 and block_table.shape[0] >= rows, "mixed_prefill_attention: bad metadata")
+    tiles = portion_tokens // 64 + rows              # (a row's last tile may be short)
+    # keys of a tile of 16 queries: what the first and the last of them see, from the multiple of 64 below on
+    span = min(longest, _visible_span(longest, window, chunk) + 15)
+    key_blocks = 8 * min(-(-(span + 63) // 64), -(-longest // 64))
+    tile_bytes = 4 * heads * key_blocks * 256
+    slab_tiles = max(1, min(tiles, MIXED_SLAB_BYTES // tile_bytes))
+    log_sums = alloc((heads, tokens), torch.float32)
+    mixed = alloc((slab_tiles * tile_bytes,), torch.uint8)
+    lib = library("bf16")
+    _check(lib, lib.mir_mixed_prefill_attention_bf16(
+        qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
+        block_table.shape[1], query_starts.data_ptr(), context_lens.data_ptr(), rows, tokens, page_size, heads, kv_heads,
+        dim, value_dim, scale, head_mix.data_ptr(), int(window or 0), int(chunk or 0), tiles, slab_tiles, key_blocks,
+        MIXED_SEGMENT_TILES, log_sums.data_ptr(), mixed.data_ptr(), _stream()))
 
 
 def _check_extras(what: str, sinks, gate, out: torch.Tensor, heads: int, gate_per_head: bool = False,
