@@ -1,4 +1,4 @@
-"""`bench.py --design doderax | zufotar | dalesun | gumazen`: prefill and decode throughput of a design at layer sizes that resemble a
+"""`bench.py --design doderax | zufotar | dalesun | gumazen | pedotar`: prefill and decode throughput of a design at layer sizes that resemble a
 real model's (random weights), beside the dense SwiGLU decoder of equal width, depth and parameter count (and, for
 Zufotar, beside Doderax, the closest model of the framework: recurrent mixers and attention in parallel layers), and
 every kernel the design adds alone, with the fraction of its roofline, beside the like kernel of the closest model.
@@ -522,6 +522,188 @@ def gumazen_kernel_table(s, tools) -> dict:
     return table
 
 
+# Pedotar: selective scans without a feed-forward, latent attention and attention with mixed heads (each with a SwiGLU) in
+# turn; a run of layers repeats.  The chunk is such that single tokens behind a 2,048-token prompt see a third of one.
+PEDOTAR_SIZES = {
+    "w2048": dict(width=2048, layers=8, runs=12, loop=(2, 6, 2), inner=4096, state=16, dt_rank=128, heads=16, kv_heads=4,
+                  dim=128, chunk=1536, rot=64, vdim=128, kv_rank=512, ff=8192, vocab=65536),
+    "w4096": dict(width=4096, layers=6, runs=8, loop=(2, 4, 2), inner=8192, state=16, dt_rank=256, heads=32, kv_heads=8,
+                  dim=128, chunk=1536, rot=64, vdim=128, kv_rank=512, ff=14336, vocab=65536),
+}
+
+
+def pedotar_config(s: dict) -> dict:
+    scan = {"type": "mamba1", "mixer": {"inner": s["inner"], "state": s["state"], "dt_rank": s["dt_rank"], "conv": 4}, "mlp": None}
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot"], "vdim": s["vdim"], "kv_rank": s["kv_rank"],
+        "scale": (s["dim"] + s["rot"]) ** -0.5, "rot": {"dims": s["rot"], "base": 1000000.0}}}
+    mixed = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+        "mask": {"size": s["chunk"]}}}
+    kinds = (scan, latent, scan, mixed)
+    start, stop, times = s["loop"]
+    return {"architecture": "Pedotar", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
+            "loop": {"start": start, "stop": stop, "times": times}, "layers": [kinds[i % 4] for i in range(s["layers"])]}
+
+
+def pedotar_beside(s: dict) -> dict:
+    """Zufotar with the same width, kinds of layers in turn (wkv for the selective scan, latent attention for both kinds of
+    attention), loop and feed-forward weights, without routed experts."""
+    latent = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": s["ff"] * 3 // 2}, "mixer": {
+        "heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot"], "vdim": s["vdim"], "q_rank": 3 * s["width"] // 8,
+        "kv_rank": s["kv_rank"], "scale": (s["dim"] + s["rot"]) ** -0.5, "rot": {"dims": s["rot"], "base": 1000000.0}}}
+    wkv = {"type": "wkv", "mlp": None, "mixer": {"heads": s["width"] // 64, "dim": 64, "decay_rank": 64}}
+    start, stop, times = s["loop"]
+    return {"architecture": "Zufotar", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
+            "loop": {"start": start, "stop": stop, "times": times},
+            "layers": [(wkv, latent)[i % 2] for i in range(s["layers"])]}
+
+
+def pedotar_kernel_table(s, tools) -> dict:
+    """Every kernel the design adds or extends, alone, at the sizes of a 2,048-token prompt and of a step of 8 decoded
+    tokens: [microseconds, fraction of its roofline], beside the like kernel of the closest models (Zufotar's and
+    Doderax's recurrences and preparations, Dalesun's addition of a normed branch, the dense decoder's attention over as
+    many keys).  Attention of a prompt against the matrix peak (scores, mixture of the heads and values), everything else
+    against the copy bandwidth."""
+    import torch
+    from libmir_b200 import kernels
+    timed, copies, rand, device, hbm, flops_peak = (tools[k] for k in ("timed", "copies", "rand", "device", "hbm", "flops_peak"))
+    bf16, f32, i32 = torch.bfloat16, torch.float32, torch.int32
+    width, heads, kv_heads, dim, chunk = s["width"], s["heads"], s["kv_heads"], s["dim"], s["chunk"]
+    inner, n, dt_rank, rot, rank = s["inner"], s["state"], s["dt_rank"], s["rot"], s["kv_rank"]
+    alloc_pool = {}
+
+    def alloc(shape, kind):                              # scratch that calls of one size share, as a step's arena does
+        key = (tuple(shape), kind, alloc_pool.setdefault("turn", 0))
+        alloc_pool["turn"] = alloc_pool["turn"] + 1
+        if key not in alloc_pool:
+            alloc_pool[key] = torch.empty(shape, dtype=kind, device=device)
+        return alloc_pool[key]
+
+    def with_scratch(call):
+        def run():
+            alloc_pool["turn"] = 0
+            call()
+        return run
+    table = {}
+    for label, rows, portion in ((f"prefill_{PROMPT}", 1, PROMPT), (f"decode_b{BATCH}", BATCH, 1)):
+        tokens, prompt = rows * portion, portion > 1
+        starts = torch.arange(0, tokens + 1, portion, dtype=i32, device=device)
+        row_of = torch.arange(tokens, dtype=i32, device=device) // portion
+        slots = torch.arange(rows, dtype=i32, device=device)
+        context = PROMPT if prompt else chunk                # (single tokens: the last position of a chunk sees all of it)
+        positions = (torch.arange(tokens, dtype=i32, device=device) % portion) + (context - portion)
+        # ---- the recurrence and its convolution
+        packs = copies(lambda: (rand(tokens, 2 * inner), rand(tokens, inner, dtype=f32), rand(tokens, inner),
+                                torch.zeros(rows, inner, n, device=device)), tokens * inner * 10 + rows * inner * n * 4)
+        low = rand(tokens, dt_rank + 2 * n)
+        vector = rand(inner, dtype=f32)
+        rates = -torch.rand(inner, n, device=device)
+        out = torch.empty(tokens, inner, device=device, dtype=bf16)
+        calls = [lambda p=p: kernels.selective_scan(p[2], p[1], vector, low[:, dt_rank:dt_rank + n], low[:, dt_rank + n:],
+                                                    p[0][:, inner:], rates, vector, p[3], starts, slots, positions, out)
+                 for p in packs]
+        table[f"{label}_selective_scan"] = timed(calls, tokens * inner * 10 + rows * inner * n * 8, hbm)
+        conv_w, tail = rand(inner, 4), torch.zeros(rows, 3, inner, device=device)
+        calls = [lambda p=p: kernels.short_conv_silu(p[0][:, :inner], conv_w, tail, row_of, starts, slots, positions, out,
+                                                     bias=vector, single_tokens_only=not prompt) for p in packs]
+        table[f"{label}_short_conv_bias"] = timed(calls, tokens * inner * 4 + rows * 3 * inner * 8, hbm)
+        del packs
+        wkv_heads = width // 64
+        packs = copies(lambda: (rand(3, tokens, width), rand(tokens, width, dtype=f32, scale=0.2),
+                                torch.zeros(rows, wkv_heads, 64, 64, device=device)), tokens * width * 10 + rows * width * 64 * 4)
+        bias, bonus = rand(width, dtype=f32, scale=0.2), rand(width, dtype=f32, scale=0.2)
+        read = torch.empty(tokens, width, device=device, dtype=f32)
+        calls = [lambda p=p: kernels.wkv_scan(p[0][0], p[0][1], p[0][2], p[1], bias, bonus, p[2], starts, slots, positions,
+                                              read, wkv_heads, 64) for p in packs]
+        table[f"{label}_zufotar_wkv_scan"] = timed(calls, tokens * width * 14 + rows * width * 64 * 8, hbm)
+        channels = 3 * heads * dim
+        raw, delta_w = [rand(tokens, channels + 64) for _ in range(4)], rand(channels, 4)
+        delta_tail = torch.zeros(rows, 3, channels, device=device)
+        beta_raw, decay_raw = rand(tokens, heads), rand(tokens, heads)
+        small = rand(heads, dtype=f32)
+        prepared = torch.empty(tokens, channels, device=device, dtype=f32)
+        beta, decay = (torch.empty(tokens, heads, device=device, dtype=f32) for _ in range(2))
+        calls = [lambda r=r: kernels.delta_rule_prepare(r[:, :channels], delta_w, delta_tail, beta_raw, decay_raw, small, small,
+                                                        row_of, starts, slots, positions, prepared, beta, decay, heads, heads,
+                                                        dim, dim) for r in raw]
+        table[f"{label}_doderax_convolution_and_gates"] = timed(calls, tokens * channels * 6 + rows * 3 * channels * 8, hbm)
+        del packs, raw
+        # ---- between two sublayers
+        packs = copies(lambda: (rand(tokens, width, dtype=f32), rand(tokens, width, dtype=f32)), tokens * width * 8)
+        w_a, w_b = rand(width, dtype=f32), rand(width, dtype=f32)
+        out_w = torch.empty(tokens, width, device=device, dtype=bf16)
+        calls = [lambda p=p: kernels.add_layer_norm(p[0], p[1], w_a, w_b, 1e-5, None, w_a, w_b, 1e-5, out_w) for p in packs]
+        table[f"{label}_add_layer_norm_and_next_norm"] = timed(calls, tokens * width * 14, hbm)
+        calls = [lambda p=p: kernels.add_normed_branches([p[1]], [w_a], p[0], 1e-6, 1.0, rounded=out_w) for p in packs]
+        table[f"{label}_dalesun_add_normed_branch"] = timed(calls, tokens * width * 14, hbm)
+        # ---- latent attention: the preparation with the queries' rotation, beside Zufotar's two kernels
+        key_width, per_head = rank + rot, dim + rot
+        pages_per_row = -(-(context + PAGE) // PAGE)
+        cache_rows = rows * pages_per_row * PAGE
+        block_table = torch.arange(rows * pages_per_row, dtype=i32, device=device).view(rows, pages_per_row).contiguous()
+        contexts = torch.full((rows,), context, dtype=i32, device=device)
+        slot_map = (torch.arange(tokens, dtype=i32, device=device) // portion) * (pages_per_row * PAGE) + positions
+        latents = [rand(cache_rows, 1, key_width) for _ in range(4)]
+        rows_q = [rand(tokens, heads * per_head + key_width) for _ in range(4)]
+        folded = torch.empty(tokens, heads, key_width, device=device, dtype=bf16)
+        freq, ones = torch.rand(rot // 2, device=device), torch.ones(rank, device=device)
+        q_of = lambda p: p[:, :heads * per_head].unflatten(1, (heads, per_head))[:, :, dim:]
+        calls = [lambda p=p, c=c: kernels.latent_prepare(p, 0, 0, heads * per_head, rank, rot, None, ones, 1e-5, positions, slot_map,
+                                                         freq, 1.0, False, None, c, (q_of(p), folded[:, :, rank:]))
+                 for p, c in zip(rows_q, latents)]
+        moved = tokens * (key_width * 4 + heads * rot * 4)
+        table[f"{label}_latent_prepare_with_queries"] = timed(calls, moved, hbm)
+        latent_q = torch.empty(tokens, 3 * width // 8, device=device, dtype=bf16)
+        zufotar_rows = [rand(tokens, 3 * width // 8 + key_width) for _ in range(4)]
+        norm_q = torch.ones(3 * width // 8, device=device)
+
+        def zufotar_prepare(p, z, c):
+            kernels.latent_prepare(z, 0, 3 * width // 8, 3 * width // 8, rank, rot, norm_q, ones, 1e-5, positions, slot_map, freq,
+                                   1.0, True, latent_q, c)
+            kernels.rope_rows(q_of(p), folded[:, :, rank:], positions, freq, 1.0, True)
+        calls = [lambda p=p, z=z, c=c: zufotar_prepare(p, z, c) for p, z, c in zip(rows_q, zufotar_rows, latents)]
+        table[f"{label}_zufotar_latent_prepare_and_rotation"] = timed(calls, moved + tokens * 3 * width // 8 * 4, hbm)
+        # ---- attention with mixed heads, beside the dense decoder's over as many keys
+        banks = max(2, min(24, -(-(300 << 20) // (cache_rows * kv_heads * dim * 4))))
+        k_cache = [rand(cache_rows, kv_heads, dim, scale=0.5) for _ in range(banks)]
+        v_cache = [rand(cache_rows, kv_heads, dim, scale=0.5) for _ in range(banks)]
+        qkv = rand(tokens, (heads + 2 * kv_heads) * dim, scale=0.3)
+        mix = rand(heads, heads, dtype=f32, scale=0.3)
+        result = torch.empty(tokens, heads * dim, device=device, dtype=bf16)
+        scale = dim ** -0.5
+        if prompt:
+            seen = sum(p % chunk + 1 for p in range(PROMPT))
+            calls = [with_scratch(lambda k=k, v=v: kernels.mixed_prefill_attention(
+                qkv, result, k, v, block_table, starts, contexts, PAGE, heads, kv_heads, dim, dim, scale, mix, None, chunk, tokens,
+                context, alloc)) for k, v in zip(k_cache, v_cache)]
+            table[f"{label}_mixed_attention"] = timed(calls, seen * (4.0 * dim * heads + 2.0 * heads * heads), flops_peak)
+            in_window = sum(min(p + 1, chunk // 2) for p in range(PROMPT))
+            calls = [lambda k=k, v=v: kernels.prefill_attention(qkv, result, k, v, block_table, starts, contexts, PAGE, heads,
+                                                                 kv_heads, dim, scale, chunk // 2) for k, v in zip(k_cache, v_cache)]
+            table[f"{label}_dense_attention_window"] = timed(calls, 4.0 * in_window * dim * heads, flops_peak)
+            bias = rand(heads, 513, dtype=f32)
+            calls = [lambda k=k, v=v: kernels.prefill_attention(qkv, result, k, v, block_table, starts, contexts, PAGE, heads,
+                                                                 kv_heads, dim, scale, chunk // 2, softcap=30.0,
+                                                                 distance_bias=bias) for k, v in zip(k_cache, v_cache)]
+            table[f"{label}_gumazen_attention_window_capped_biased"] = timed(calls, 4.0 * in_window * dim * heads, flops_peak)
+        else:
+            key_bytes = rows * context * kv_heads * dim * 2 * 2
+            calls = [with_scratch(lambda k=k, v=v: kernels.mixed_decode_attention(
+                qkv, result, k, v, block_table, positions, PAGE, heads, kv_heads, dim, dim, scale, mix, None, chunk, context,
+                alloc)) for k, v in zip(k_cache, v_cache)]
+            table[f"{label}_mixed_attention"] = timed(calls, key_bytes, hbm)
+            partition, parts, floats = kernels.decode_attention_plan(rows, heads, kv_heads, dim, PAGE, context)
+            scratch = torch.empty(max(floats, 1), device=device, dtype=f32)
+            calls = [lambda k=k, v=v: kernels.decode_attention(qkv, result, k, v, block_table, positions, PAGE, heads, kv_heads, dim,
+                                                                scale, None, partition, parts, scratch if floats else None)
+                     for k, v in zip(k_cache, v_cache)]
+            table[f"{label}_dense_attention"] = timed(calls, key_bytes, hbm)
+        alloc_pool.clear()
+    return table
+
+
 def doderax_config(s: dict) -> dict:
     delta = {"heads": s["heads"], "kv_heads": s["heads"], "dim": s["dim"], "vdim": s["dim"], "conv": 4,
              "decay_rank": 64, "gate_rank": 64}
@@ -796,6 +978,21 @@ def run(args, peaks: dict) -> dict:
             entry["gumazen"] = model_numbers(gumazen_config(s), s["vocab"])
             entry["zufotar"] = model_numbers(zufotar_config(ZUFOTAR_SIZES[name]), s["vocab"])
             entry["dense_swiglu"] = model_numbers(dense_config(dict(DESIGN_SIZES[name], layers=s["runs"])), s["vocab"])
+            report[name] = entry
+        return report
+    if args.design == "pedotar":
+        rand = lambda *shape, dtype=bf16, scale=1.0: (torch.randn(*shape, device=device, dtype=f32) * scale).to(dtype)
+        tools = {"timed": timed, "copies": copies, "rand": rand, "device": device, "hbm": hbm, "flops_peak": flops_peak}
+        report = {}
+        for name in [n for n in PEDOTAR_SIZES if args.design_sizes in ("all", n)]:
+            s = PEDOTAR_SIZES[name]
+            entry = {"sizes": s}
+            if not args.skip_points:
+                entry["kernels_us_and_fraction_of_roofline"] = pedotar_kernel_table(s, tools)
+                torch.cuda.empty_cache()
+            entry["pedotar"] = model_numbers(pedotar_config(s), s["vocab"])
+            entry["zufotar_dense_feed_forwards"] = model_numbers(pedotar_beside(s), s["vocab"])
+            entry["dense_swiglu"] = model_numbers(dense_config(dict(s, layers=s["runs"])), s["vocab"])
             report[name] = entry
         return report
     if args.design == "dalesun":
