@@ -537,15 +537,22 @@ mixed_decode_values_kernel(const bf16* __restrict__ v_pages, const int* __restri
       raw[p] = *reinterpret_cast<const uint4*>(
           v_pages + (((size_t)table[key / page_size] * page_size + key % page_size) * kv_heads + kv_head) * value_dim + piece * 8);
   }
-  for (int g = thread; g < heads; g += 128) {
+  // a head's parts over the lanes (more parts than lanes: a running maximum), then over the warp
+  for (int g = warp; g < heads; g += 4) {
     const float2* mine_stats = stats + ((size_t)row * heads + g) * parts;
-    float top = -INFINITY;
-    for (int p = 0; p < filled; ++p) top = fmaxf(top, mine_stats[p].x);
-    float sum = 0.0f;
-    for (int p = 0; p < filled; ++p) sum = fmaf(mine_stats[p].y, exp2f(mine_stats[p].x - top), sum);
-    log_sums[g] = top + log2f(sum);
+    float top = -INFINITY, sum = 0.0f;
+    for (int p = lane; p < filled; p += 32) {
+      const float2 one = mine_stats[p];
+      const float next = fmaxf(top, one.x);
+      sum = fmaf(one.y, exp2f(one.x - next), sum * exp2f(top - next));
+      top = next;
+    }
+    const float all = warp_max(top);
+    sum = warp_sum(top == -INFINITY ? 0.0f : sum * exp2f(top - all));
+    if (lane == 0) log_sums[g] = all + log2f(sum);
   }
   __syncthreads();
+#pragma unroll 4
   for (int i = thread; i < heads * kKeys; i += 128) {
     const int g = i / kKeys, j = i % kKeys;
     weights[i] = j < count ? exp2f(scores[((size_t)row * heads + g) * parts * kKeys + part * kKeys + j] - log_sums[g]) : 0.0f;
@@ -554,8 +561,11 @@ mixed_decode_values_kernel(const bf16* __restrict__ v_pages, const int* __restri
   for (int i = thread; i < R * kKeys; i += 128) {
     const int r = i / kKeys, j = i % kKeys;
     float sum = 0.0f;
-    if (r < mine)
-      for (int g = 0; g < heads; ++g) sum = fmaf(mix[(size_t)(head0 + r) * heads + g], weights[g * kKeys + j], sum);
+    if (r < mine) {
+      const float* factors = mix + (size_t)(head0 + r) * heads;
+#pragma unroll 8
+      for (int g = 0; g < heads; ++g) sum = fmaf(__ldg(factors + g), weights[g * kKeys + j], sum);
+    }
     mixed[i] = sum;
   }
   __syncthreads();

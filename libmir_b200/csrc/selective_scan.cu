@@ -5,234 +5,386 @@
 // portion and written at its end; softplus, exponentials, state and sums are 32-bit whatever the activations' type T.
 //
 // A CTA takes 32 channels of one request and walks over the request's tokens of this step.  Four lanes share a channel
-// and hold its state in registers, PER numbers each.  Tokens come in chunks: the raw inputs of the next chunk are copied
-// asynchronously into one of two buffers while the current one is worked on; each chunk's step sizes (and their products
-// with x), B and C are first turned into 32-bit numbers in shared memory, once per CTA.  The chain from token to token is
-// one fused multiply-add per state number; exponentials and products hang off it.  The read-outs of four tokens are
-// reduced over the four lanes together, in three shuffles, which leaves each lane one token's sum: it adds the term with
-// D, applies the gate and puts the result where z was, and whole rows leave in 16-byte pieces.  The order of a sum depends
-// on N alone, never on how a prompt was cut or what else is in the batch.
+// and hold its state in registers, PER numbers each.  The chain from token to token is one fused multiply-add per state
+// number; exponentials and products hang off it.  The read-outs of four tokens are reduced over the four lanes together,
+// in three shuffles, which leaves each lane one token's sum.  The order of a sum depends on N alone, never on how a prompt
+// was cut or what else is in the batch, and both kernels below do the same arithmetic in the same order.
+//
+//   selective_scan         portions: four warps walk, four others work for them.  While the walkers go through one chunk
+//                          of tokens, the others turn the next chunk's step sizes (and their products with x), B and C
+//                          into 32-bit numbers in shared memory, fetch the raw inputs of the chunk behind it, and finish
+//                          the chunk before (the term with D, the gate, the result's rows); one barrier per chunk.
+//   selective_scan_single  a step of single tokens: four warps, nothing staged ahead.
 #include "common.cuh"
 
 using namespace mir;
 
 namespace {
 
-constexpr int kThreads = 128;
+constexpr int kWalkers = 128;                       // threads that hold the state
+constexpr int kHelpers = 128;                       // threads that prepare and finish for them (portions)
 constexpr int kLanes = 4;                           // lanes that share a channel
-constexpr int kChannels = kThreads / kLanes;        // channels a CTA takes
+constexpr int kChannels = kWalkers / kLanes;        // channels a CTA takes
+constexpr int kMaxChunk = 32;
+constexpr int kSumRow = 40;                         // floats between two tokens' sums (lanes of a warp on 32 banks)
 
 __device__ __forceinline__ float softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 // 2^v for v <= 0: the hardware's approximation (2 ulp), results below the smallest normal number are zero.
 __device__ __forceinline__ float exp2_below_one(float v) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v));
   return y;
 }
+// Two 32-bit numbers side by side: one instruction multiplies (and adds) both.
+typedef unsigned long long pair32;
+__device__ __forceinline__ pair32 make_pair(float a, float b) {
+  pair32 p;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(p) : "f"(a), "f"(b));
+  return p;
+}
+__device__ __forceinline__ void split_pair(pair32 p, float& a, float& b) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(p));
+}
+__device__ __forceinline__ pair32 mul_pair(pair32 a, pair32 b) {
+  pair32 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ pair32 fma_pair(pair32 a, pair32 b, pair32 c) {
+  pair32 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
 __device__ __forceinline__ void copy16(void* dst, const void* src) {
   const unsigned target = (unsigned)__cvta_generic_to_shared(dst);
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(target), "l"(src) : "memory");
 }
 
-// Shared memory of a chunk of `chunk` tokens, in bytes from the start; every part starts on 16 bytes.
+// What a lane knows of its channel: PER numbers of state and their rates, in pairs.  An odd number (one) is a pair whose
+// second half stays zero.  numbers: how many of them there are (PER, less at the end of a channel, none without one);
+// wide: all of them, on 16-byte boundaries.
+template <int PER>
+struct Channel {
+  static constexpr int PAIRS = (PER + 1) / 2;
+  pair32 s[PAIRS], rate[PAIRS];
+  __device__ __forceinline__ static void load(pair32 (&v)[PAIRS], const float* from, int numbers, bool wide) {
+    if (PER % 4 == 0 && wide) {
+#pragma unroll
+      for (int i = 0; i + 1 < PAIRS; i += 2) {
+        const float4 a = *reinterpret_cast<const float4*>(from + 2 * i);
+        v[i] = make_pair(a.x, a.y);
+        v[i + 1] = make_pair(a.z, a.w);
+      }
+      return;
+    }
+#pragma unroll
+    for (int i = 0; i < PAIRS; ++i)
+      v[i] = make_pair(2 * i < numbers ? from[2 * i] : 0.0f, 2 * i + 1 < numbers ? from[2 * i + 1] : 0.0f);
+  }
+  __device__ __forceinline__ void store(float* to, int numbers, bool wide) const {
+    if (PER % 4 == 0 && wide) {
+#pragma unroll
+      for (int i = 0; i + 1 < PAIRS; i += 2) {
+        float4 a;
+        split_pair(s[i], a.x, a.y);
+        split_pair(s[i + 1], a.z, a.w);
+        *reinterpret_cast<float4*>(to + 2 * i) = a;
+      }
+      return;
+    }
+#pragma unroll
+    for (int i = 0; i < PAIRS; ++i) {
+      float a, b;
+      split_pair(s[i], a, b);
+      if (2 * i < numbers) to[2 * i] = a;
+      if (2 * i + 1 < numbers) to[2 * i + 1] = b;
+    }
+  }
+  // One token: the state moves on; returns this lane's share of the read-out.
+  __device__ __forceinline__ float advance(float step, float step_x, const pair32 (&b)[PAIRS], const pair32 (&c)[PAIRS]) {
+    const pair32 steps = make_pair(step, step), inputs = make_pair(step_x, step_x);
+    pair32 sum = 0ull;
+#pragma unroll
+    for (int i = 0; i < PAIRS; ++i) {
+      float low, high;
+      split_pair(mul_pair(steps, rate[i]), low, high);
+      s[i] = fma_pair(make_pair(exp2_below_one(low), exp2_below_one(high)), s[i], mul_pair(inputs, b[i]));
+      sum = fma_pair(s[i], c[i], sum);
+    }
+    float even, odd;
+    split_pair(sum, even, odd);
+    return even + odd;
+  }
+};
+
+// ---------------------------------------------------------------------------------------------- portions
+// Shared memory of chunks of `chunk` tokens, in bytes from the start; every part starts on 16 bytes and is there twice.
 template <typename T>
 struct Layout {
-  int dt, x, z, b, c, raw;                          // offsets in a raw buffer, and its size
-  int du, bf, cf, total;                            // the 32-bit parts behind the two raw buffers
+  int du, b, c, raw_b, raw_c, sums, total;
   __host__ __device__ Layout(int chunk, int columns, int padded) {
-    dt = 0;
-    x = dt + chunk * kChannels * 4;
-    z = x + chunk * kChannels * (int)sizeof(T);
-    b = z + chunk * kChannels * (int)sizeof(T);
-    c = b + chunk * columns * (int)sizeof(T);
-    raw = c + chunk * columns * (int)sizeof(T);
-    du = 2 * raw;
-    bf = du + chunk * kChannels * 8;
-    cf = bf + chunk * padded * 4;
-    total = cf + chunk * padded * 4;
+    du = 0;                                         // [2][chunk][kChannels] (step, step * x)
+    b = du + 2 * chunk * kChannels * 8;             // [2][chunk][padded] 32-bit
+    c = b + 2 * chunk * padded * 4;
+    raw_b = c + 2 * chunk * padded * 4;             // [2][chunk][columns] as they come
+    raw_c = raw_b + 2 * chunk * columns * (int)sizeof(T);
+    sums = raw_c + 2 * chunk * columns * (int)sizeof(T);        // [2][chunk][kSumRow]
+    total = sums + 2 * chunk * kSumRow * 4;
   }
 };
 
 template <int PER>
-__device__ __forceinline__ void load_row(const float* p, float (&v)[PER]) {
-  if constexpr (PER % 4 == 0) {
+struct Operands {
+  static constexpr int PAIRS = (PER + 1) / 2;
+  float2 du;
+  pair32 b[PAIRS], c[PAIRS];
+  __device__ __forceinline__ static void load_pairs(const float* p, pair32 (&v)[PAIRS]) {
+    if constexpr (PER % 4 == 0) {
 #pragma unroll
-    for (int i = 0; i < PER; i += 4) {
-      const float4 a = *reinterpret_cast<const float4*>(p + i);
-      v[i] = a.x; v[i + 1] = a.y; v[i + 2] = a.z; v[i + 3] = a.w;
+      for (int i = 0; i < PAIRS; i += 2) {
+        const ulonglong2 both = *reinterpret_cast<const ulonglong2*>(p + 2 * i);
+        v[i] = both.x;
+        v[i + 1] = both.y;
+      }
+    } else if constexpr (PER % 2 == 0) {
+#pragma unroll
+      for (int i = 0; i < PAIRS; ++i) v[i] = *reinterpret_cast<const pair32*>(p + 2 * i);
+    } else {
+      v[0] = make_pair(p[0], 0.0f);
     }
-  } else if constexpr (PER % 2 == 0) {
-#pragma unroll
-    for (int i = 0; i < PER; i += 2) {
-      const float2 a = *reinterpret_cast<const float2*>(p + i);
-      v[i] = a.x; v[i + 1] = a.y;
-    }
-  } else {
-#pragma unroll
-    for (int i = 0; i < PER; ++i) v[i] = p[i];
   }
-}
+  __device__ __forceinline__ void load(const float2* du_at, const float* b_at, const float* c_at) {
+    du = *du_at;
+    load_pairs(b_at, b);
+    load_pairs(c_at, c);
+  }
+};
 
-// grid (rows, ceil(channels / kChannels)), kThreads threads.
-//   x, z    element (t, c) at x[t * ldx + c], z[t * ldz + c];  raw: (t, c) at raw[t * channels + c], 32-bit
+// grid (rows, ceil(channels / kChannels)), kWalkers + kHelpers threads.
+//   x, z    element (t, c) at x[t * ldx + c], z[t * ldz + c];  raw_step: (t, c) at raw_step[t * channels + c], 32-bit
 //   b, c    element (t, n) at b[t * ldb + n], c[t * ldb + n]; rows readable up to `columns`, a multiple of 8
 //   rates   [channels, n]: A log2(e);  skip: D;  state [slots, channels, n];  out [tokens, channels]
 template <typename T, int PER>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kWalkers + kHelpers)
 selective_scan_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ raw_step,
                       const float* __restrict__ step_bias, const T* __restrict__ b, const T* __restrict__ c, long long ldb,
                       const T* __restrict__ z, long long ldz, const float* __restrict__ rates,
                       const float* __restrict__ skip, float* __restrict__ state, const int* __restrict__ query_starts,
                       const int* __restrict__ state_slots, const int* __restrict__ positions, T* __restrict__ out,
                       int channels, int n, int columns, int chunk) {
+  static_assert(PER == 1 || PER % 2 == 0, "numbers a lane holds come in pairs");
   extern __shared__ __align__(16) unsigned char shared[];
   constexpr int PADDED = kLanes * PER;
   constexpr int V = 16 / sizeof(T);                 // elements in 16 bytes
+  constexpr int STRIDE = kHelpers / kChannels;
+  constexpr int TOKENS = kMaxChunk / STRIDE;        // of a chunk, for a helper
   const Layout<T> at(chunk, columns, PADDED);
-  float2* const du = reinterpret_cast<float2*>(shared + at.du);
-  float* const bf = reinterpret_cast<float*>(shared + at.bf);
-  float* const cf = reinterpret_cast<float*>(shared + at.cf);
-  const int thread = threadIdx.x, l = thread % kLanes, mine = thread / kLanes;
+  float2* const du_s = reinterpret_cast<float2*>(shared + at.du);
+  float* const b_s = reinterpret_cast<float*>(shared + at.b);
+  float* const c_s = reinterpret_cast<float*>(shared + at.c);
+  T* const raw_b = reinterpret_cast<T*>(shared + at.raw_b);
+  T* const raw_c = reinterpret_cast<T*>(shared + at.raw_c);
+  float* const sums = reinterpret_cast<float*>(shared + at.sums);
   const int first_channel = blockIdx.y * kChannels;
-  const int channel = first_channel + mine;
-  const bool active = channel < channels;
-  const int here = min(kChannels, channels - first_channel);     // (a multiple of 8)
-
-  float rate[PER], s[PER];
-#pragma unroll
-  for (int e = 0; e < PER; ++e)
-    rate[e] = (active && l * PER + e < n) ? rates[(size_t)channel * n + l * PER + e] : 0.0f;
-  const float skip_factor = active ? skip[channel] : 0.0f;
   grid_launch_dependents();
   grid_dependency_wait();
   const int row = blockIdx.x;
   const int start = query_starts[row], end = query_starts[row + 1];
   if (end <= start || positions[start] < 0) return;              // the whole CTA: an empty or padding row
-  float* const own_state = state + ((size_t)state_slots[row] * channels + (active ? channel : 0)) * n + l * PER;
-  const bool whole = n == PADDED;                                // (then a lane's numbers start on PER * 4 bytes)
-  if (whole && active) load_row<PER>(own_state, s);
-  else {
+  const int chunks = (end - start + chunk - 1) / chunk;
+
+  if (threadIdx.x < kWalkers) {
+    const int l = threadIdx.x % kLanes, mine = threadIdx.x / kLanes;
+    const int channel = first_channel + mine;
+    const int numbers = channel < channels ? min(PER, n - l * PER) : 0;
+    const bool wide = numbers == PER && n % 4 == 0;
+    const size_t own = (size_t)(channel < channels ? channel : 0) * n + l * PER;
+    float* const own_state = state + (size_t)state_slots[row] * channels * n + own;
+    Channel<PER> held;
+    held.load(held.s, own_state, numbers, wide);
+    held.load(held.rate, rates + own, numbers, wide);
+    for (int phase = 0; phase < chunks + 2; ++phase) {
+      if (phase >= 1 && phase <= chunks) {
+        const int which = (phase - 1) & 1;
+        const int count = min(chunk, end - start - (phase - 1) * chunk);
+        const float2* du_at = du_s + which * chunk * kChannels + mine;
+        const float* b_at = b_s + which * chunk * PADDED + l * PER;
+        const float* c_at = c_s + which * chunk * PADDED + l * PER;
+        float* sum_at = sums + which * chunk * kSumRow + l * kSumRow + mine;
+        auto reduce = [&](const float (&y)[4], int t) {          // four tokens over four lanes: lane l is left with t + l
+          const bool low = (l & 1) == 0, front = (l & 2) == 0;
+          float first = low ? y[0] : y[1], second = low ? y[2] : y[3];
+          first += __shfl_xor_sync(0xffffffffu, low ? y[1] : y[0], 1);
+          second += __shfl_xor_sync(0xffffffffu, low ? y[3] : y[2], 1);
+          float sum = front ? first : second;
+          sum += __shfl_xor_sync(0xffffffffu, front ? second : first, 2);
+          sum_at[t * kSumRow] = sum;                             // (behind the last token: a place nobody reads)
+        };
+        int t = 0;
+        if constexpr (PER <= 8) {                                // the next four tokens' operands are on their way
+          Operands<PER> next[4];
+          if (count >= 4) {
 #pragma unroll
-    for (int e = 0; e < PER; ++e) s[e] = (active && l * PER + e < n) ? own_state[e] : 0.0f;
+            for (int i = 0; i < 4; ++i) next[i].load(du_at + i * kChannels, b_at + i * PADDED, c_at + i * PADDED);
+          }
+          for (; t + 4 <= count; t += 4) {
+            float y[4];
+            const bool more = t + 8 <= count;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              y[i] = held.advance(next[i].du.x, next[i].du.y, next[i].b, next[i].c);
+              if (more) next[i].load(du_at + (t + 4 + i) * kChannels, b_at + (t + 4 + i) * PADDED, c_at + (t + 4 + i) * PADDED);
+            }
+            reduce(y, t);
+          }
+        } else {
+          for (; t + 4 <= count; t += 4) {
+            float y[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              Operands<PER> now;
+              now.load(du_at + (t + i) * kChannels, b_at + (t + i) * PADDED, c_at + (t + i) * PADDED);
+              y[i] = held.advance(now.du.x, now.du.y, now.b, now.c);
+            }
+            reduce(y, t);
+          }
+        }
+        if (t < count) {
+          float y[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+          for (int i = 0; i < 3; ++i) {
+            if (t + i < count) {
+              Operands<PER> now;
+              now.load(du_at + (t + i) * kChannels, b_at + (t + i) * PADDED, c_at + (t + i) * PADDED);
+              y[i] = held.advance(now.du.x, now.du.y, now.b, now.c);
+            }
+          }
+          reduce(y, t);
+        }
+      }
+      __syncthreads();
+    }
+    held.store(own_state, numbers, wide);
+    return;
   }
 
-  auto fetch = [&](int from, unsigned char* buffer) {
-    const int count = min(chunk, end - from);
-    const int step_pieces = here / 4, wide_pieces = here / V, state_pieces = columns / V;
-    const int per_token = step_pieces + 2 * wide_pieces + 2 * state_pieces;
-    // a warp takes a token at a time: its lanes walk over the token's pieces
-    for (int t = thread >> 5; t < count; t += kThreads / 32) {
-      for (int p = thread & 31; p < per_token; p += 32) {
-        int i = p;
-        if (i < step_pieces) {
-          copy16(buffer + at.dt + (t * kChannels + i * 4) * 4, raw_step + (size_t)(from + t) * channels + first_channel + i * 4);
-          continue;
-        }
-        i -= step_pieces;
-        if (i < wide_pieces) {
-          copy16(buffer + at.x + (t * kChannels + i * V) * (int)sizeof(T), x + (size_t)(from + t) * ldx + first_channel + i * V);
-          continue;
-        }
-        i -= wide_pieces;
-        if (i < wide_pieces) {
-          copy16(buffer + at.z + (t * kChannels + i * V) * (int)sizeof(T), z + (size_t)(from + t) * ldz + first_channel + i * V);
-          continue;
-        }
-        i -= wide_pieces;
-        if (i < state_pieces) {
-          copy16(buffer + at.b + (t * columns + i * V) * (int)sizeof(T), b + (size_t)(from + t) * ldb + i * V);
-          continue;
-        }
-        i -= state_pieces;
-        copy16(buffer + at.c + (t * columns + i * V) * (int)sizeof(T), c + (size_t)(from + t) * ldb + i * V);
-      }
+  // helpers: a thread always works for the same channel
+  const int thread = threadIdx.x - kWalkers;
+  const int mine = thread % kChannels, first_token = thread / kChannels;
+  const int channel = first_channel + mine;
+  const bool active = channel < channels;
+  const float bias = active ? step_bias[channel] : 0.0f, skip_factor = active ? skip[channel] : 0.0f;
+  float steps[TOKENS], inputs[TOKENS];
+  auto fetch = [&](int number) {                                 // the raw inputs of a chunk: registers, and B and C
+    const int from = start + number * chunk, count = min(chunk, end - from);
+#pragma unroll
+    for (int k = 0; k < TOKENS; ++k) {
+      const int t = first_token + k * STRIDE;
+      const bool there = active && t < count;
+      steps[k] = there ? raw_step[(size_t)(from + t) * channels + channel] : 0.0f;
+      inputs[k] = there ? to_float(x[(size_t)(from + t) * ldx + channel]) : 0.0f;
+    }
+    const int pieces = columns / V, which = number & 1;
+    for (int i = thread; i < count * pieces; i += kHelpers) {
+      const int t = i / pieces, p = i - t * pieces;
+      copy16(raw_b + (size_t)(which * chunk + t) * columns + p * V, b + (size_t)(from + t) * ldb + p * V);
+      copy16(raw_c + (size_t)(which * chunk + t) * columns + p * V, c + (size_t)(from + t) * ldb + p * V);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-
-  fetch(start, shared);
-  // what the lane turns into 32-bit numbers of a chunk: always the same channel (thread % kChannels)
-  const int staged_channel = thread % kChannels;
-  const float bias = first_channel + staged_channel < channels ? step_bias[first_channel + staged_channel] : 0.0f;
-  int buffer = 0;
-  for (int from = start; from < end; from += chunk, buffer ^= 1) {
-    const int count = min(chunk, end - from);
-    unsigned char* const in = shared + buffer * at.raw;
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                             // this chunk is here; the other buffer has been read
-    if (from + chunk < end) fetch(from + chunk, shared + (buffer ^ 1) * at.raw);
-    const T* const xs = reinterpret_cast<const T*>(in + at.x);
-    T* const zs = reinterpret_cast<T*>(in + at.z);
-    if (staged_channel < here) {
-      const float* steps = reinterpret_cast<const float*>(in + at.dt);
-      for (int t = thread / kChannels; t < count; t += kThreads / kChannels) {
-        const float step = softplus(steps[t * kChannels + staged_channel] + bias);
-        du[t * kChannels + staged_channel] = make_float2(step, step * to_float(xs[t * kChannels + staged_channel]));
+  // (B and C of the first chunk are copied by all helpers before any of them reads: a barrier among the helpers)
+  fetch(0);
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  asm volatile("bar.sync 1, %0;" ::"n"(kHelpers) : "memory");
+  for (int phase = 0; phase < chunks + 2; ++phase) {
+    const int finished = phase - 2;
+    float gates[TOKENS], skipped[TOKENS];
+    if (finished >= 0) {                                         // (asked for first, used last)
+      const int from = start + finished * chunk, count = min(chunk, end - from);
+#pragma unroll
+      for (int k = 0; k < TOKENS; ++k) {
+        const int t = first_token + k * STRIDE;
+        const bool there = active && t < count;
+        gates[k] = there ? to_float(z[(size_t)(from + t) * ldz + channel]) : 0.0f;
+        skipped[k] = there ? to_float(x[(size_t)(from + t) * ldx + channel]) : 0.0f;
       }
     }
-    const T* const bs = reinterpret_cast<const T*>(in + at.b);
-    const T* const cs = reinterpret_cast<const T*>(in + at.c);
-    for (int i = thread; i < count * PADDED; i += kThreads) {
-      const int t = i / PADDED, k = i - t * PADDED;
-      bf[i] = k < n ? to_float(bs[t * columns + k]) : 0.0f;
-      cf[i] = k < n ? to_float(cs[t * columns + k]) : 0.0f;
+    if (phase < chunks) {
+      const int which = phase & 1, count = min(chunk, end - start - phase * chunk);
+#pragma unroll
+      for (int k = 0; k < TOKENS; ++k) {
+        const int t = first_token + k * STRIDE;
+        if (t < count) {
+          const float step = softplus(steps[k] + bias);
+          du_s[(which * chunk + t) * kChannels + mine] = make_float2(step, step * inputs[k]);
+        }
+      }
+      for (int i = thread; i < count * PADDED; i += kHelpers) {
+        const int t = i / PADDED, k = i % PADDED;
+        b_s[which * chunk * PADDED + i] = k < n ? to_float(raw_b[(size_t)(which * chunk + t) * columns + k]) : 0.0f;
+        c_s[which * chunk * PADDED + i] = k < n ? to_float(raw_c[(size_t)(which * chunk + t) * columns + k]) : 0.0f;
+      }
+      if (phase + 1 < chunks) fetch(phase + 1);
     }
+    if (finished >= 0) {
+      const int which = finished & 1, from = start + finished * chunk, count = min(chunk, end - from);
+#pragma unroll
+      for (int k = 0; k < TOKENS; ++k) {
+        const int t = first_token + k * STRIDE;
+        if (active && t < count) {
+          const float value = fmaf(skip_factor, skipped[k], sums[(which * chunk + t) * kSumRow + mine]);
+          out[(size_t)(from + t) * channels + channel] = from_float<T>(value * silu(gates[k]));
+        }
+      }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");         // (the next chunk's B and C are here behind the barrier)
     __syncthreads();
-    const float* b_at = bf + l * PER;
-    const float* c_at = cf + l * PER;
-    const float2* du_at = du + mine;
-    auto advance = [&](int t) {
-      const float2 step = du_at[t * kChannels];
-      float bb[PER], cc[PER];
-      load_row<PER>(b_at + t * PADDED, bb);
-      load_row<PER>(c_at + t * PADDED, cc);
-      float even = 0.0f, odd = 0.0f;
-#pragma unroll
-      for (int e = 0; e < PER; ++e) {
-        s[e] = fmaf(exp2_below_one(step.x * rate[e]), s[e], step.y * bb[e]);
-        if (e & 1) odd = fmaf(s[e], cc[e], odd);
-        else even = fmaf(s[e], cc[e], even);
-      }
-      return even + odd;
-    };
-    for (int t = 0; t < count; t += 4) {
-      float y[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-      if (t + 4 <= count) {
-#pragma unroll
-        for (int i = 0; i < 4; ++i) y[i] = advance(t + i);
-      } else {
-#pragma unroll
-        for (int i = 0; i < 3; ++i)
-          if (t + i < count) y[i] = advance(t + i);
-      }
-      // four tokens over four lanes: lane l is left with token t + l
-      const bool low = (l & 1) == 0, front = (l & 2) == 0;
-      float first = low ? y[0] : y[1], second = low ? y[2] : y[3];
-      first += __shfl_xor_sync(0xffffffffu, low ? y[1] : y[0], 1);
-      second += __shfl_xor_sync(0xffffffffu, low ? y[3] : y[2], 1);
-      float sum = front ? first : second;
-      sum += __shfl_xor_sync(0xffffffffu, front ? second : first, 2);
-      const int token = t + l;
-      if (token < count && active) {
-        const int place = token * kChannels + mine;
-        const float value = fmaf(skip_factor, to_float(xs[place]), sum);
-        zs[place] = from_float<T>(value * silu(to_float(zs[place])));
-      }
-    }
-    __syncthreads();
-    const int wide_pieces = here / V;
-    for (int i = thread; i < count * (kChannels / V); i += kThreads) {
-      const int t = i / (kChannels / V), p = i % (kChannels / V);
-      if (p < wide_pieces)
-        *reinterpret_cast<uint4*>(out + (size_t)(from + t) * channels + first_channel + p * V) =
-            *reinterpret_cast<const uint4*>(zs + t * kChannels + p * V);
-    }
   }
-  if (!active) return;
+}
+
+// ---------------------------------------------------------------------------------------------- single tokens
+// The same grid, kWalkers threads: request row r brings token query_starts[r].
+template <typename T, int PER>
+__global__ void __launch_bounds__(kWalkers)
+selective_scan_single_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ raw_step,
+                             const float* __restrict__ step_bias, const T* __restrict__ b, const T* __restrict__ c,
+                             long long ldb, const T* __restrict__ z, long long ldz, const float* __restrict__ rates,
+                             const float* __restrict__ skip, float* __restrict__ state, const int* __restrict__ query_starts,
+                             const int* __restrict__ state_slots, const int* __restrict__ positions, T* __restrict__ out,
+                             int channels, int n) {
+  constexpr int PAIRS = Channel<PER>::PAIRS;
+  grid_launch_dependents();
+  const int l = threadIdx.x % kLanes;
+  const int channel = blockIdx.y * kChannels + threadIdx.x / kLanes;
+  const bool active = channel < channels;
+  const int numbers = active ? min(PER, n - l * PER) : 0;
+  const bool wide = numbers == PER && n % 4 == 0;
+  const size_t own = (size_t)(active ? channel : 0) * n + l * PER;
+  Channel<PER> held;
+  held.load(held.rate, rates + own, numbers, wide);
+  const float bias = active ? step_bias[channel] : 0.0f, skip_factor = active ? skip[channel] : 0.0f;
+  grid_dependency_wait();
+  const int token = query_starts[blockIdx.x];
+  if (query_starts[blockIdx.x + 1] <= token || positions[token] < 0) return;    // the whole CTA: an empty or padding row
+  float* const own_state = state + (size_t)state_slots[blockIdx.x] * channels * n + own;
+  held.load(held.s, own_state, numbers, wide);
+  const float input = active ? to_float(x[(size_t)token * ldx + channel]) : 0.0f;
+  const float gate = active ? to_float(z[(size_t)token * ldz + channel]) : 0.0f;
+  const float step = softplus((active ? raw_step[(size_t)token * channels + channel] : 0.0f) + bias);
+  pair32 bb[PAIRS], cc[PAIRS];
+  const T* b_at = b + (size_t)token * ldb + l * PER;
+  const T* c_at = c + (size_t)token * ldb + l * PER;
 #pragma unroll
-  for (int e = 0; e < PER; ++e)
-    if (l * PER + e < n) own_state[e] = s[e];
+  for (int i = 0; i < PAIRS; ++i) {
+    bb[i] = make_pair(2 * i < numbers ? to_float(b_at[2 * i]) : 0.0f, 2 * i + 1 < numbers ? to_float(b_at[2 * i + 1]) : 0.0f);
+    cc[i] = make_pair(2 * i < numbers ? to_float(c_at[2 * i]) : 0.0f, 2 * i + 1 < numbers ? to_float(c_at[2 * i + 1]) : 0.0f);
+  }
+  float sum = held.advance(step, step * input, bb, cc);
+  sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+  sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+  held.store(own_state, numbers, wide);
+  if (active && l == 0) out[(size_t)token * channels + channel] = from_float<T>(fmaf(skip_factor, input, sum) * silu(gate));
 }
 
 template <typename T, int PER>
@@ -240,7 +392,12 @@ int launch(const void* x, long long ldx, const float* raw_step, const float* ste
            long long ldb, const void* z, long long ldz, const float* rates, const float* skip, float* state,
            const int* query_starts, const int* state_slots, const int* positions, void* out, int tokens, int rows,
            int channels, int n, int columns, cudaStream_t stream) {
-  int chunk = tokens == rows ? 4 : 32;                           // (a step of single tokens stages one)
+  const dim3 grid(rows, (channels + kChannels - 1) / kChannels);
+  if (tokens == rows)                                            // a step of single tokens: every row brings one
+    return mir_launch("selective_scan", selective_scan_single_kernel<T, PER>, grid, dim3(kWalkers), 0, stream, 0, (const T*)x,
+                      ldx, raw_step, step_bias, (const T*)b, (const T*)c, ldb, (const T*)z, ldz, rates, skip, state,
+                      query_starts, state_slots, positions, (T*)out, channels, n);
+  int chunk = kMaxChunk;
   while (chunk > 4 && Layout<T>(chunk, columns, kLanes * PER).total > 96 * 1024) chunk /= 2;
   const int smem = Layout<T>(chunk, columns, kLanes * PER).total;
   if (smem > 48 * 1024) {
@@ -250,10 +407,9 @@ int launch(const void* x, long long ldx, const float* raw_step, const float* ste
       return MIR_CUDA_ERROR;
     }
   }
-  return mir_launch("selective_scan", selective_scan_kernel<T, PER>, dim3(rows, (channels + kChannels - 1) / kChannels),
-                    dim3(kThreads), smem, stream, 0, (const T*)x, ldx, raw_step, step_bias, (const T*)b, (const T*)c, ldb,
-                    (const T*)z, ldz, rates, skip, state, query_starts, state_slots, positions, (T*)out, channels, n,
-                    columns, chunk);
+  return mir_launch("selective_scan", selective_scan_kernel<T, PER>, grid, dim3(kWalkers + kHelpers), smem, stream, 0,
+                    (const T*)x, ldx, raw_step, step_bias, (const T*)b, (const T*)c, ldb, (const T*)z, ldz, rates, skip, state,
+                    query_starts, state_slots, positions, (T*)out, channels, n, columns, chunk);
 }
 
 template <typename T>

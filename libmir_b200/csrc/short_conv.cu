@@ -14,7 +14,7 @@ using namespace mir;
 
 namespace {
 
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 
 // grid (tokens, ceil(channels / 256)).  x: the packed projection rows, channel c of token t at x[t * ldx + c].
 template <typename T, typename TO>
@@ -71,18 +71,23 @@ __device__ __forceinline__ void load_floats(const float* p, float (&v)[V]) {
   }
 }
 
-// grid (ceil(tokens / run), ceil(pieces / blockDim.x)); every pointer and stride of x, out, tail and bias on 16 bytes.
-template <typename T, typename TO, int TAPS>
+// grid (ceil(tokens / RUN), ceil(pieces / blockDim.x)); every pointer and stride of x, out, tail and bias on 16 bytes.
+template <typename T, typename TO, int TAPS, int RUN>
 __global__ void __launch_bounds__(128)
 short_conv_silu_wide_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, const float* __restrict__ bias,
                             float* __restrict__ tail, const int* __restrict__ row_of_token,
                             const int* __restrict__ query_starts, const int* __restrict__ state_slots,
-                            const int* __restrict__ positions, TO* __restrict__ out, int tokens, int channels, int run) {
+                            const int* __restrict__ positions, TO* __restrict__ out, int tokens, int channels) {
   constexpr int V = Piece<T>::kCount;
   grid_launch_dependents();
   grid_dependency_wait();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (c >= channels) return;
+  const int first = blockIdx.x * RUN, count = min(RUN, tokens - first);
+  uint4 raw[RUN];                                   // all inputs of the run at once: one trip to memory
+#pragma unroll
+  for (int i = 0; i < RUN; ++i)
+    raw[i] = i < count ? *reinterpret_cast<const uint4*>(x + (size_t)(first + i) * ldx + c) : make_uint4(0u, 0u, 0u, 0u);
   float taps[V][TAPS], shift[V];
 #pragma unroll
   for (int v = 0; v < V; ++v)
@@ -92,9 +97,11 @@ short_conv_silu_wide_kernel(const T* __restrict__ x, long long ldx, const T* __r
   for (int v = 0; v < V; ++v) shift[v] = 0.0f;
   if (bias != nullptr) load_floats<V>(bias + c, shift);
   float past[TAPS][V];                              // past[j]: the input TAPS - 1 - j tokens back; the last is the token's own
-  const int first = blockIdx.x * run, last = min(first + run, tokens);
   int row = -1;
-  for (int token = first; token < last; ++token) {
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    if (i >= count) break;
+    const int token = first + i;
     if (positions[token] < 0) { row = -1; continue; }            // a padding row of a captured batch
     const int mine = row_of_token[token];
     if (mine == row) {
@@ -113,7 +120,7 @@ short_conv_silu_wide_kernel(const T* __restrict__ x, long long ldx, const T* __r
         else load_floats<V>(old + (size_t)(TAPS - 1 + src) * channels, past[j]);
       }
     }
-    load_piece(x + (size_t)token * ldx + c, past[TAPS - 1]);
+    load_piece(reinterpret_cast<const T*>(&raw[i]), past[TAPS - 1]);
     float result[V];
 #pragma unroll
     for (int v = 0; v < V; ++v) {
@@ -141,13 +148,14 @@ int launch(const T* x, long long ldx, const T* w, const float* bias, float* tail
   const int threads = channels >= 256 ? 256 : ((channels + 31) / 32) * 32;
   int status, skip_single = 0;
   if (aligned && taps <= 4) {
-    const int run = tokens >= 512 ? 8 : (tokens >= 128 ? 2 : 1);
+    const int run = tokens >= 512 ? 8 : 1;
     const int pieces = channels / V;
     const int wide_threads = pieces >= 128 ? 128 : ((pieces + 31) / 32) * 32;
     const dim3 grid((tokens + run - 1) / run, (pieces + wide_threads - 1) / wide_threads);
-#define MIR_CONV(N)                                                                                                     \
-  status = mir_launch("short_conv_silu_wide", short_conv_silu_wide_kernel<T, TO, N>, grid, dim3(wide_threads), 0, stream, 0, \
-                      x, ldx, w, bias, tail, row_of_token, query_starts, state_slots, positions, out, tokens, channels, run)
+#define MIR_CONV_RUN(N, R)                                                                                              \
+  mir_launch("short_conv_silu_wide", short_conv_silu_wide_kernel<T, TO, N, R>, grid, dim3(wide_threads), 0, stream, 0, x, ldx, \
+             w, bias, tail, row_of_token, query_starts, state_slots, positions, out, tokens, channels)
+#define MIR_CONV(N) status = run == 8 ? MIR_CONV_RUN(N, 8) : MIR_CONV_RUN(N, 1)
     switch (taps) {
       case 1: MIR_CONV(1); break;
       case 2: MIR_CONV(2); break;
@@ -155,6 +163,7 @@ int launch(const T* x, long long ldx, const T* w, const float* bias, float* tail
       default: MIR_CONV(4); break;
     }
 #undef MIR_CONV
+#undef MIR_CONV_RUN
     if (single_tokens_only) return status;
     skip_single = 1;
   } else {

@@ -119,65 +119,124 @@ __global__ void __launch_bounds__(512, 3) layer_norm_kernel(const float* __restr
 }
 
 // One CTA per token.  x [tokens, width] in place; y [tokens, width]; rows (or null) [tokens, width] is added to x as well;
-// out (or null): the layer norm of the new x with the reader's weight, bias and eps.
-template <typename T, int V>
-__global__ void __launch_bounds__(512, 2) add_layer_norm_kernel(
+// out (or null): the layer norm of the new x with the reader's weight, bias and eps.  A thread keeps its columns in
+// registers, V at a time in PIECES places blockDim.x * V columns apart: everything is read from memory once, ahead of the
+// first barrier.
+template <typename T, int V, int PIECES>
+__global__ void __launch_bounds__(512) add_layer_norm_kernel(
     float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ weight, const float* __restrict__ bias,
     float eps, const float* __restrict__ rows, const float* __restrict__ next_weight, const float* __restrict__ next_bias,
     float next_eps, T* __restrict__ out, int width) {
-  extern __shared__ float row_values[];            // [width] the branch's row, then the new residual's; [width] the residual
   __shared__ float scratch[128];
-  float* const old = row_values + width;
   grid_launch_dependents();
   grid_dependency_wait();
   const size_t base = (size_t)blockIdx.x * width;
-  float sum = 0.0f;
-  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+  auto load = [](float (&v)[V], const float* from) {
     if constexpr (V == 4) {
-      const float4 branch = *reinterpret_cast<const float4*>(y + base + c);
-      float4 residual = *reinterpret_cast<const float4*>(x + base + c);
-      *reinterpret_cast<float4*>(row_values + c) = branch;
-      *reinterpret_cast<float4*>(old + c) = residual;
-      sum += branch.x; sum += branch.y; sum += branch.z; sum += branch.w;
+      const float4 a = *reinterpret_cast<const float4*>(from);
+      v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
     } else {
-      row_values[c] = y[base + c];
-      old[c] = x[base + c];
-      sum += row_values[c];
+      v[0] = *from;
     }
+  };
+  float branch[PIECES][V], old[PIECES][V];
+  float sum = 0.0f;
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * V;
+#pragma unroll
+    for (int v = 0; v < V; ++v) branch[p][v] = old[p][v] = 0.0f;
+    if (c < width) {
+      load(branch[p], y + base + c);
+      load(old[p], x + base + c);
+      if (rows != nullptr) {
+        float more[V];
+        load(more, rows + base + c);
+#pragma unroll
+        for (int v = 0; v < V; ++v) old[p][v] += more[v];
+      }
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) sum += branch[p][v];
   }
   const float mean = block_sum_once(sum, scratch) / (float)width;
   float squares = 0.0f;
-  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    if ((p * blockDim.x + threadIdx.x) * V >= width) continue;
 #pragma unroll
     for (int v = 0; v < V; ++v) {
-      const float d = row_values[c + v] - mean;
+      const float d = branch[p][v] - mean;
       squares = fmaf(d, d, squares);
     }
   }
   const float inverse = rsqrtf(block_sum_once(squares, scratch + 32) / (float)width + eps);
   float total = 0.0f;
-  for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
-    alignas(16) float w[V], b[V], more[V], fresh[V];
-    if constexpr (V == 4) {
-      *reinterpret_cast<float4*>(w) = __ldg(reinterpret_cast<const float4*>(weight + c));
-      *reinterpret_cast<float4*>(b) = __ldg(reinterpret_cast<const float4*>(bias + c));
-      *reinterpret_cast<float4*>(more) = rows != nullptr ? *reinterpret_cast<const float4*>(rows + base + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    } else {
-      w[0] = weight[c];
-      b[0] = bias[c];
-      more[0] = rows != nullptr ? rows[base + c] : 0.0f;
-    }
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * V;
+    if (c >= width) continue;
+    float w[V], b[V];
+    load(w, weight + c);
+    load(b, bias + c);
 #pragma unroll
     for (int v = 0; v < V; ++v) {
-      fresh[v] = old[c + v] + fmaf((row_values[c + v] - mean) * inverse, w[v], b[v]);
-      if (rows != nullptr) fresh[v] += more[v];
-      row_values[c + v] = fresh[v];
-      total += fresh[v];
+      old[p][v] += fmaf((branch[p][v] - mean) * inverse, w[v], b[v]);
+      total += old[p][v];
     }
-    if constexpr (V == 4) *reinterpret_cast<float4*>(x + base + c) = *reinterpret_cast<const float4*>(fresh);
-    else x[base + c] = fresh[0];
+    store_columns<float, V>(x + base + c, old[p]);
   }
-  if (out != nullptr) norm_row<T, V>(row_values, total, scratch + 64, next_weight, next_bias, out + base, width, next_eps);
+  if (out == nullptr) return;
+  const float next_mean = block_sum_once(total, scratch + 64) / (float)width;
+  squares = 0.0f;
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    if ((p * blockDim.x + threadIdx.x) * V >= width) continue;
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      const float d = old[p][v] - next_mean;
+      squares = fmaf(d, d, squares);
+    }
+  }
+  const float next_inverse = rsqrtf(block_sum_once(squares, scratch + 96) / (float)width + next_eps);
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * V;
+    if (c >= width) continue;
+    float w[V], b[V];
+    load(w, next_weight + c);
+    load(b, next_bias + c);
+#pragma unroll
+    for (int v = 0; v < V; ++v) w[v] = fmaf((old[p][v] - next_mean) * next_inverse, w[v], b[v]);
+    store_columns<T, V>(out + base + c, w);
+  }
+}
+
+template <typename T>
+int launch_add_layer_norm(float* x, const float* y, const float* weight, const float* bias, float eps, const float* rows,
+                          const float* next_weight, const float* next_bias, float next_eps, void* out, int tokens, int width,
+                          cudaStream_t stream) {
+#define MIR_ADD_NORM(V, P)                                                                                               \
+  return mir_launch("add_layer_norm", add_layer_norm_kernel<T, V, P>, dim3(tokens), dim3(threads), 0, stream, 0, x, y, weight, \
+                    bias, eps, rows, next_weight, next_bias, next_eps, (T*)out, width)
+  // one piece a thread up to 512 threads, then more pieces
+  const int per_thread = width % 4 == 0 ? 4 : 1;
+  const int places = (width + per_thread - 1) / per_thread;
+  const int threads = places >= 512 ? 512 : (places + 31) / 32 * 32;
+  const int pieces = (places + threads - 1) / threads;
+  if (per_thread == 4) {
+    if (pieces <= 1) MIR_ADD_NORM(4, 1);
+    if (pieces <= 2) MIR_ADD_NORM(4, 2);
+    if (pieces <= 4) MIR_ADD_NORM(4, 4);
+    if (pieces <= 8) MIR_ADD_NORM(4, 8);
+  } else {
+    if (pieces <= 2) MIR_ADD_NORM(1, 2);
+    if (pieces <= 8) MIR_ADD_NORM(1, 8);
+    if (pieces <= 32) MIR_ADD_NORM(1, 32);
+  }
+#undef MIR_ADD_NORM
+  mir_set_error("add_layer_norm: rows of %d numbers are wider than the kernel takes", width);
+  return MIR_BAD_ARGUMENT;
 }
 
 __global__ void streams_write_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ mix,
@@ -381,27 +440,15 @@ MIR_EXPORT int mir_add_layer_norm(int bf16, float* x, const float* y, const floa
                                   const float* rows, const float* next_weight, const float* next_bias, float next_eps,
                                   void* out, int tokens, int width, cudaStream_t stream) {
   if (tokens == 0) return MIR_OK;
-  const size_t smem = 2 * (size_t)width * sizeof(float);
-  if (tokens < 0 || width <= 0 || smem > 200 * 1024 || (out != nullptr && (next_weight == nullptr || next_bias == nullptr))) {
+  if (tokens < 0 || width <= 0 || (out != nullptr && (next_weight == nullptr || next_bias == nullptr))) {
     mir_set_error("add_layer_norm: bad sizes (tokens %d, width %d)", tokens, width);
     return MIR_BAD_ARGUMENT;
   }
-  const bool wide = width % 4 == 0;
-  const int threads = width >= 4096 ? 512 : (width >= 1024 || !wide ? 256 : 128);
-#define MIR_ADD_NORM(T, V)                                                                                             \
-  do {                                                                                                                 \
-    if (smem > 48 * 1024)                                                                                              \
-      cudaFuncSetAttribute(add_layer_norm_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
-    return mir_launch("add_layer_norm", add_layer_norm_kernel<T, V>, dim3(tokens), dim3(threads), smem, stream, 0, x, y, \
-                      weight, bias, eps, rows, next_weight, next_bias, next_eps, (T*)out, width);                      \
-  } while (0)
-  if (bf16) {
-    if (wide) MIR_ADD_NORM(__nv_bfloat16, 4);
-    MIR_ADD_NORM(__nv_bfloat16, 1);
-  }
-  if (wide) MIR_ADD_NORM(float, 4);
-  MIR_ADD_NORM(float, 1);
-#undef MIR_ADD_NORM
+  if (bf16)
+    return launch_add_layer_norm<__nv_bfloat16>(x, y, weight, bias, eps, rows, next_weight, next_bias, next_eps, out, tokens,
+                                                width, stream);
+  return launch_add_layer_norm<float>(x, y, weight, bias, eps, rows, next_weight, next_bias, next_eps, out, tokens, width,
+                                      stream);
 }
 
 // x [tokens, streams, width] in place; y [tokens, width]; mix [streams, streams] indexed [from, to]; write [streams].
