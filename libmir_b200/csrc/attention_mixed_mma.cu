@@ -474,15 +474,33 @@ mixed_decode_scores_kernel(const bf16* __restrict__ q, long long q_stride, const
       k8[2 * i + 1] = f.y;
     }
     const int j = (p * 4 + warp) * SUBS + sub;
+    // R sums over LANES lanes: in each step a lane hands half of its heads over, as long as it has more than one
+    float dot[R];
 #pragma unroll
     for (int r = 0; r < R; ++r) {
-      float dot = 0.0f;
+      dot[r] = 0.0f;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) dot = fmaf(query[r][i], k8[i], dot);
-#pragma unroll
-      for (int o = LANES / 2; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-      if (piece == 0) s_s[r][j] = dot * scale2;
+      for (int i = 0; i < 8; ++i) dot[r] = fmaf(query[r][i], k8[i], dot[r]);
     }
+    int head = 0;
+#pragma unroll
+    for (int o = LANES / 2, held = R; o > 0; o >>= 1) {
+      const bool upper = (piece & o) != 0;
+      if (held > 1) {
+        held /= 2;
+        head += upper ? held : 0;
+#pragma unroll
+        for (int r = 0; r < R / 2; ++r) {
+          if (r < held) {
+            const float other = __shfl_xor_sync(0xffffffffu, upper ? dot[r] : dot[r + held], o);
+            dot[r] = (upper ? dot[r + held] : dot[r]) + other;
+          }
+        }
+      } else {
+        dot[0] += __shfl_xor_sync(0xffffffffu, dot[0], o);
+      }
+    }
+    if (piece % (LANES / R) == 0) s_s[head][j] = dot[0] * scale2;
   }
   __syncthreads();
   for (int r = warp; r < mine; r += 4) {
@@ -537,36 +555,53 @@ mixed_decode_values_kernel(const bf16* __restrict__ v_pages, const int* __restri
       raw[p] = *reinterpret_cast<const uint4*>(
           v_pages + (((size_t)table[key / page_size] * page_size + key % page_size) * kv_heads + kv_head) * value_dim + piece * 8);
   }
-  // a head's parts over the lanes (more parts than lanes: a running maximum), then over the warp
-  for (int g = warp; g < heads; g += 4) {
-    const float2* mine_stats = stats + ((size_t)row * heads + g) * parts;
+  // four threads go over a head's parts, then put their sums together
+  for (int base = 0; base < heads; base += 32) {
+    const int g = base + thread / 4;
+    const float2* mine_stats = stats + ((size_t)row * heads + min(g, heads - 1)) * parts;
     float top = -INFINITY, sum = 0.0f;
-    for (int p = lane; p < filled; p += 32) {
+#pragma unroll 4
+    for (int p = thread & 3; p < filled; p += 4) {
       const float2 one = mine_stats[p];
       const float next = fmaxf(top, one.x);
       sum = fmaf(one.y, exp2f(one.x - next), sum * exp2f(top - next));
       top = next;
     }
-    const float all = warp_max(top);
-    sum = warp_sum(top == -INFINITY ? 0.0f : sum * exp2f(top - all));
-    if (lane == 0) log_sums[g] = all + log2f(sum);
+    float all = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
+    all = fmaxf(all, __shfl_xor_sync(0xffffffffu, all, 2));
+    sum = top == -INFINITY ? 0.0f : sum * exp2f(top - all);
+    sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+    sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+    if ((thread & 3) == 0 && g < heads) log_sums[g] = all + log2f(sum);
   }
   __syncthreads();
+  // (behind `count` the scores are -inf)
+  const float* part_scores = scores + (size_t)row * heads * parts * kKeys + part * kKeys;
 #pragma unroll 4
-  for (int i = thread; i < heads * kKeys; i += 128) {
-    const int g = i / kKeys, j = i % kKeys;
-    weights[i] = j < count ? exp2f(scores[((size_t)row * heads + g) * parts * kKeys + part * kKeys + j] - log_sums[g]) : 0.0f;
+  for (int i = thread; i < heads * (kKeys / 4); i += 128) {
+    const int g = i / (kKeys / 4), j = i % (kKeys / 4) * 4;
+    const float4 four = *reinterpret_cast<const float4*>(part_scores + (size_t)g * parts * kKeys + j);
+    const float log_sum = log_sums[g];
+    *reinterpret_cast<float4*>(weights + g * kKeys + j) =
+        make_float4(exp2f(four.x - log_sum), exp2f(four.y - log_sum), exp2f(four.z - log_sum), exp2f(four.w - log_sum));
   }
   __syncthreads();
-  for (int i = thread; i < R * kKeys; i += 128) {
-    const int r = i / kKeys, j = i % kKeys;
-    float sum = 0.0f;
+  for (int i = thread; i < R * (kKeys / 4); i += 128) {
+    const int r = i / (kKeys / 4), j = i % (kKeys / 4) * 4;
+    float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     if (r < mine) {
       const float* factors = mix + (size_t)(head0 + r) * heads;
 #pragma unroll 8
-      for (int g = 0; g < heads; ++g) sum = fmaf(__ldg(factors + g), weights[g * kKeys + j], sum);
+      for (int g = 0; g < heads; ++g) {
+        const float m = __ldg(factors + g);
+        const float4 w = *reinterpret_cast<const float4*>(weights + g * kKeys + j);
+        sum.x = fmaf(m, w.x, sum.x);
+        sum.y = fmaf(m, w.y, sum.y);
+        sum.z = fmaf(m, w.z, sum.z);
+        sum.w = fmaf(m, w.w, sum.w);
+      }
     }
-    mixed[i] = sum;
+    *reinterpret_cast<float4*>(mixed + r * kKeys + j) = sum;
   }
   __syncthreads();
   float acc[R][8];
@@ -743,7 +778,7 @@ MIR_EXPORT int mir_mixed_decode_attention_bf16(const void* q, long long q_stride
   if (rows == 0) return MIR_OK;
   if (!mir_mixed_decode_takes(heads, kv_heads, dim, value_dim) || page_size <= 0 || table_width <= 0 || window < 0 ||
       chunk < 0 || rows < 0 || rows > 65535 || parts <= 0 || q_stride % 8 || (uintptr_t)q % 16 || (uintptr_t)out % 8 ||
-      (uintptr_t)k_pages % 16 || (uintptr_t)v_pages % 16 || (uintptr_t)partial % 16) {
+      (uintptr_t)k_pages % 16 || (uintptr_t)v_pages % 16 || (uintptr_t)partial % 16 || (uintptr_t)scores % 16) {
     mir_set_error("mixed_decode_attention: sizes or alignment the kernels do not take (heads %d over %d, widths %d and %d, "
                   "parts %d)", heads, kv_heads, dim, value_dim, parts);
     return MIR_BAD_ARGUMENT;

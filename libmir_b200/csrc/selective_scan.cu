@@ -10,7 +10,7 @@
 // in three shuffles, which leaves each lane one token's sum.  The order of a sum depends on N alone, never on how a prompt
 // was cut or what else is in the batch, and both kernels below do the same arithmetic in the same order.
 //
-//   selective_scan         portions: four warps walk, four others work for them.  While the walkers go through one chunk
+//   selective_scan         portions: four warps walk, eight others work for them.  While the walkers go through one chunk
 //                          of tokens, the others turn the next chunk's step sizes (and their products with x), B and C
 //                          into 32-bit numbers in shared memory, fetch the raw inputs of the chunk behind it, and finish
 //                          the chunk before (the term with D, the gate, the result's rows); one barrier per chunk.
@@ -22,13 +22,27 @@ using namespace mir;
 namespace {
 
 constexpr int kWalkers = 128;                       // threads that hold the state
-constexpr int kHelpers = 128;                       // threads that prepare and finish for them (portions)
+constexpr int kHelpers = 256;                       // threads that prepare and finish for them (portions)
 constexpr int kLanes = 4;                           // lanes that share a channel
 constexpr int kChannels = kWalkers / kLanes;        // channels a CTA takes
 constexpr int kMaxChunk = 32;
 constexpr int kSumRow = 40;                         // floats between two tokens' sums (lanes of a warp on 32 banks)
 
-__device__ __forceinline__ float softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+// log(1 + e^z) = max(z, 0) + log(1 + e) with e = e^-|z| in (0, 1], and log(1 + e) = 2 artanh(s), s = e / (2 + e) <= 1/3, by
+// the series 2 (s + s^3/3 + s^5/5 + ...): what is left out behind s^15 is below 2e-9 of the result.
+__device__ __forceinline__ float softplus(float z) {
+  const float e = expf(-fabsf(z));
+  const float s = __fdividef(e, 2.0f + e), q = s * s;
+  float sum = 1.0f / 15.0f;
+  sum = fmaf(sum, q, 1.0f / 13.0f);
+  sum = fmaf(sum, q, 1.0f / 11.0f);
+  sum = fmaf(sum, q, 1.0f / 9.0f);
+  sum = fmaf(sum, q, 1.0f / 7.0f);
+  sum = fmaf(sum, q, 1.0f / 5.0f);
+  sum = fmaf(sum, q, 1.0f / 3.0f);
+  sum = fmaf(sum, q, 1.0f);
+  return fmaxf(z, 0.0f) + 2.0f * s * sum;
+}
 __device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 // 2^v for v <= 0: the hardware's approximation (2 ulp), results below the smallest normal number are zero.
 __device__ __forceinline__ float exp2_below_one(float v) {
@@ -275,15 +289,18 @@ selective_scan_kernel(const T* __restrict__ x, long long ldx, const float* __res
   const int channel = first_channel + mine;
   const bool active = channel < channels;
   const float bias = active ? step_bias[channel] : 0.0f, skip_factor = active ? skip[channel] : 0.0f;
-  float steps[TOKENS], inputs[TOKENS];
-  auto fetch = [&](int number) {                                 // the raw inputs of a chunk: registers, and B and C
+  // raw inputs of the next chunk; x of the chunk that is staged now, walked through, and finished
+  float next_step[TOKENS], next_x[TOKENS], staged_x[TOKENS], walked_x[TOKENS], finished_x[TOKENS];
+#pragma unroll
+  for (int k = 0; k < TOKENS; ++k) staged_x[k] = walked_x[k] = 0.0f;
+  auto fetch = [&](int number) {
     const int from = start + number * chunk, count = min(chunk, end - from);
 #pragma unroll
     for (int k = 0; k < TOKENS; ++k) {
       const int t = first_token + k * STRIDE;
       const bool there = active && t < count;
-      steps[k] = there ? raw_step[(size_t)(from + t) * channels + channel] : 0.0f;
-      inputs[k] = there ? to_float(x[(size_t)(from + t) * ldx + channel]) : 0.0f;
+      next_step[k] = there ? raw_step[(size_t)(from + t) * channels + channel] : 0.0f;
+      next_x[k] = there ? to_float(x[(size_t)(from + t) * ldx + channel]) : 0.0f;
     }
     const int pieces = columns / V, which = number & 1;
     for (int i = thread; i < count * pieces; i += kHelpers) {
@@ -299,15 +316,21 @@ selective_scan_kernel(const T* __restrict__ x, long long ldx, const float* __res
   asm volatile("bar.sync 1, %0;" ::"n"(kHelpers) : "memory");
   for (int phase = 0; phase < chunks + 2; ++phase) {
     const int finished = phase - 2;
-    float gates[TOKENS], skipped[TOKENS];
-    if (finished >= 0) {                                         // (asked for first, used last)
+    float gates[TOKENS], steps[TOKENS];
+#pragma unroll
+    for (int k = 0; k < TOKENS; ++k) {
+      finished_x[k] = walked_x[k];
+      walked_x[k] = staged_x[k];
+      staged_x[k] = next_x[k];
+      steps[k] = next_step[k];
+    }
+    if (phase + 1 < chunks) fetch(phase + 1);                    // (memory is asked first, what it brings is used last)
+    if (finished >= 0) {
       const int from = start + finished * chunk, count = min(chunk, end - from);
 #pragma unroll
       for (int k = 0; k < TOKENS; ++k) {
         const int t = first_token + k * STRIDE;
-        const bool there = active && t < count;
-        gates[k] = there ? to_float(z[(size_t)(from + t) * ldz + channel]) : 0.0f;
-        skipped[k] = there ? to_float(x[(size_t)(from + t) * ldx + channel]) : 0.0f;
+        gates[k] = active && t < count ? to_float(z[(size_t)(from + t) * ldz + channel]) : 0.0f;
       }
     }
     if (phase < chunks) {
@@ -315,17 +338,14 @@ selective_scan_kernel(const T* __restrict__ x, long long ldx, const float* __res
 #pragma unroll
       for (int k = 0; k < TOKENS; ++k) {
         const int t = first_token + k * STRIDE;
-        if (t < count) {
-          const float step = softplus(steps[k] + bias);
-          du_s[(which * chunk + t) * kChannels + mine] = make_float2(step, step * inputs[k]);
-        }
+        const float step = softplus(steps[k] + bias);
+        if (t < count) du_s[(which * chunk + t) * kChannels + mine] = make_float2(step, step * staged_x[k]);
       }
       for (int i = thread; i < count * PADDED; i += kHelpers) {
         const int t = i / PADDED, k = i % PADDED;
         b_s[which * chunk * PADDED + i] = k < n ? to_float(raw_b[(size_t)(which * chunk + t) * columns + k]) : 0.0f;
         c_s[which * chunk * PADDED + i] = k < n ? to_float(raw_c[(size_t)(which * chunk + t) * columns + k]) : 0.0f;
       }
-      if (phase + 1 < chunks) fetch(phase + 1);
     }
     if (finished >= 0) {
       const int which = finished & 1, from = start + finished * chunk, count = min(chunk, end - from);
@@ -333,7 +353,7 @@ selective_scan_kernel(const T* __restrict__ x, long long ldx, const float* __res
       for (int k = 0; k < TOKENS; ++k) {
         const int t = first_token + k * STRIDE;
         if (active && t < count) {
-          const float value = fmaf(skip_factor, skipped[k], sums[(which * chunk + t) * kSumRow + mine]);
+          const float value = fmaf(skip_factor, finished_x[k], sums[(which * chunk + t) * kSumRow + mine]);
           out[(size_t)(from + t) * channels + channel] = from_float<T>(value * silu(gates[k]));
         }
       }
