@@ -12,11 +12,11 @@
 //   mixed_values       64 queries of one head: mixed weights times values
 // Key tiles start at multiples of 64 positions, so all three see the same tiles whatever the run or window.
 //
-// Single tokens (any head counts, widths that are multiples of 8 up to 256), three kernels, keys in parts of 64:
+// Single tokens (any head counts, widths that are multiples of 8 up to 256), two kernels, keys in parts of 64:
 //   mixed_decode_scores   the scores of one part and kv head, and the part's maximum and sum per head
 //   mixed_decode_values   every head's weights from its parts' sums, their mixture for this kv head's query heads, and the
-//                         part's share of the result
-//   mixed_decode_merge    the parts' shares added (they are normalised already)
+//                         part's share of the result; whoever finishes a kv head's last part adds the parts' shares (they
+//                         are normalised already)
 // Scores, softmax, mixture and sums are 32-bit.  A part or tile starts at a place that depends on the query's position
 // alone, and parts are added in ascending order.
 #include <algorithm>
@@ -428,7 +428,7 @@ __global__ void __launch_bounds__(128)
 mixed_decode_scores_kernel(const bf16* __restrict__ q, long long q_stride, const bf16* __restrict__ k_pages,
                            const int* __restrict__ block_table, int table_width, const int* __restrict__ positions,
                            int page_size, int heads, int kv_heads, int dim, float scale2, int window, int chunk, int parts,
-                           float* __restrict__ scores, float2* __restrict__ stats) {
+                           float* __restrict__ scores, float2* __restrict__ stats, int* __restrict__ arrived) {
   constexpr int PASSES = kKeys * LANES / 128, SUBS = 32 / LANES;
   __shared__ float s_s[R][kKeys];
   grid_launch_dependents();
@@ -443,6 +443,7 @@ mixed_decode_scores_kernel(const bf16* __restrict__ q, long long q_stride, const
   const int per_group = heads / kv_heads, blocks = (per_group + R - 1) / R;
   const int kv_head = blockIdx.z / blocks, head0 = kv_head * per_group + (blockIdx.z % blocks) * R;
   const int mine = min(R, (kv_head + 1) * per_group - head0);
+  if (part == 0 && threadIdx.x == 0) arrived[(size_t)row * gridDim.z + blockIdx.z] = 0;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int piece = lane % LANES, sub = lane / LANES;
   const bool reads = piece * 8 < dim;
@@ -516,13 +517,15 @@ mixed_decode_scores_kernel(const bf16* __restrict__ q, long long q_stride, const
 }
 
 // The same grid.  dynamic shared memory (floats): log_sums [heads] | weights [heads * 64] | mixed [R * 64] | sums [4 * R *
-// value_dim].  partial [rows, parts, heads, value_dim] 32-bit.
+// value_dim].  partial [rows, parts, heads, value_dim] 32-bit; arrived [rows, gridDim.z]: parts that are done, set to zero by
+// the kernel before.
 template <int R, int LANES>
 __global__ void __launch_bounds__(128)
 mixed_decode_values_kernel(const bf16* __restrict__ v_pages, const int* __restrict__ block_table, int table_width,
                            const int* __restrict__ positions, int page_size, int heads, int kv_heads, int value_dim,
                            int window, int chunk, int parts, const float* __restrict__ mix, const float* __restrict__ scores,
-                           const float2* __restrict__ stats, float* __restrict__ partial) {
+                           const float2* __restrict__ stats, float* __restrict__ partial, int* __restrict__ arrived,
+                           bf16* __restrict__ out) {
   constexpr int PASSES = kKeys * LANES / 128, SUBS = 32 / LANES;
   extern __shared__ __align__(16) float shared_f[];
   float* const log_sums = shared_f;
@@ -642,30 +645,30 @@ mixed_decode_values_kernel(const bf16* __restrict__ v_pages, const int* __restri
     }
   }
   __syncthreads();
-  float* to = partial + (((size_t)row * parts + part) * heads + head0) * value_dim;
+  // this part's share; the CTA that brings the last one of a row's parts adds them, in ascending order
+  const size_t stride = (size_t)heads * value_dim;
+  float* const shares = partial + ((size_t)row * parts * heads + head0) * value_dim;
+  __shared__ int last;
   for (int i = thread; i < mine * value_dim; i += 128) {
-    const int stride = R * value_dim;
-    to[i] = (sums[i] + sums[stride + i]) + (sums[2 * stride + i] + sums[3 * stride + i]);
+    const int quarter = R * value_dim;
+    shares[part * stride + i] = (sums[i] + sums[quarter + i]) + (sums[2 * quarter + i] + sums[3 * quarter + i]);
   }
-}
-
-// grid (ceil(heads * value_dim / 512), rows), 128 threads, four columns a thread.
-__global__ void mixed_decode_merge_kernel(const float* __restrict__ partial, bf16* __restrict__ out,
-                                          const int* __restrict__ positions, int columns, int window, int chunk, int parts) {
-  grid_launch_dependents();
-  grid_dependency_wait();
-  const int row = blockIdx.y, c = (blockIdx.x * 128 + threadIdx.x) * 4;
-  const int position = positions[row];
-  if (position < 0 || c >= columns) return;
-  const int filled = min(parts, (position - first_visible(position, window, chunk)) / kKeys + 1);
-  const float* from = partial + (size_t)row * parts * columns + c;
-  float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll 4
-  for (int p = 0; p < filled; ++p) {
-    const float4 piece = *reinterpret_cast<const float4*>(from + (size_t)p * columns);
-    sum.x += piece.x; sum.y += piece.y; sum.z += piece.z; sum.w += piece.w;
+  __threadfence();
+  __syncthreads();
+  if (thread == 0) last = atomicAdd(arrived + (size_t)row * gridDim.z + blockIdx.z, 1) == filled - 1;
+  __syncthreads();
+  if (!last) return;
+  __threadfence();
+  for (int c = thread * 4; c < mine * value_dim; c += 512) {
+    float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+    for (int p = 0; p < filled; ++p) {
+      const float4 share = __ldcg(reinterpret_cast<const float4*>(shares + p * stride + c));
+      sum.x += share.x; sum.y += share.y; sum.z += share.z; sum.w += share.w;
+    }
+    *reinterpret_cast<uint2*>(out + ((size_t)row * heads + head0) * value_dim + c) =
+        make_uint2(pack_bf16(sum.x, sum.y), pack_bf16(sum.z, sum.w));
   }
-  *reinterpret_cast<uint2*>(out + (size_t)row * columns + c) = make_uint2(pack_bf16(sum.x, sum.y), pack_bf16(sum.z, sum.w));
 }
 
 template <typename Kernel>
@@ -768,12 +771,13 @@ MIR_EXPORT int mir_mixed_decode_takes(int heads, int kv_heads, int dim, int valu
 }
 
 // Single tokens: row r's query is row r of q.  parts: at least the parts of 64 keys that any row sees; scores [rows, heads,
-// parts * 64], stats [rows, heads, parts, 2] and partial [rows, parts, heads, value_dim] are 32-bit scratch.
+// parts * 64], stats [rows, heads, parts, 2] and partial [rows, parts, heads, value_dim] are 32-bit scratch, arrived [rows,
+// heads] integers.
 MIR_EXPORT int mir_mixed_decode_attention_bf16(const void* q, long long q_stride, void* out, const void* k_pages,
                                                const void* v_pages, const int* block_table, int table_width,
                                                const int* positions, int rows, int page_size, int heads, int kv_heads,
                                                int dim, int value_dim, float scale, const float* mix, int window, int chunk,
-                                               int parts, float* scores, float* stats, float* partial,
+                                               int parts, float* scores, float* stats, float* partial, int* arrived,
                                                cudaStream_t stream) {
   if (rows == 0) return MIR_OK;
   if (!mir_mixed_decode_takes(heads, kv_heads, dim, value_dim) || page_size <= 0 || table_width <= 0 || window < 0 ||
@@ -802,7 +806,7 @@ MIR_EXPORT int mir_mixed_decode_attention_bf16(const void* q, long long q_stride
 #define MIR_SCORES_LANES(L)                                                                                              \
   status = mir_launch("mixed_decode_scores", mixed_decode_scores_kernel<kBlock, L>, grid, dim3(128), 0, stream, 0,      \
                       (const bf16*)q, q_stride, (const bf16*)k_pages, block_table, table_width, positions, page_size, heads, \
-                      kv_heads, dim, scale2, window, chunk, parts, scores, (float2*)stats)
+                      kv_heads, dim, scale2, window, chunk, parts, scores, (float2*)stats, arrived)
 #define MIR_SCORES(R)                       \
   do {                                      \
     constexpr int kBlock = R;               \
@@ -817,7 +821,8 @@ MIR_EXPORT int mir_mixed_decode_attention_bf16(const void* q, long long q_stride
     if (status == MIR_OK)                                                                                                \
       status = mir_launch("mixed_decode_values", mixed_decode_values_kernel<kBlock, L>, grid, dim3(128), smem, stream, 0, \
                           (const bf16*)v_pages, block_table, table_width, positions, page_size, heads, kv_heads,        \
-                          value_dim, window, chunk, parts, mix, (const float*)scores, (const float2*)stats, partial);   \
+                          value_dim, window, chunk, parts, mix, (const float*)scores, (const float2*)stats, partial,    \
+                          arrived, (bf16*)out);                                                                         \
   } while (0)
 #define MIR_VALUES(R)                          \
   do {                                         \
@@ -831,8 +836,5 @@ MIR_EXPORT int mir_mixed_decode_attention_bf16(const void* q, long long q_stride
 #undef MIR_SCORES_LANES
 #undef MIR_BY_BLOCK
 #undef MIR_BY_LANES
-  if (status != MIR_OK) return status;
-  const int columns = heads * value_dim;
-  return mir_launch("mixed_decode_merge", mixed_decode_merge_kernel, dim3((columns + 511) / 512, rows), dim3(128), 0, stream, 0,
-                    (const float*)partial, (bf16*)out, positions, columns, window, chunk, parts);
+  return status;
 }

@@ -193,7 +193,7 @@ _SIGNATURES = {
         "mir_mixed_decode_takes": [c_int, c_int, c_int, c_int],
         "mir_mixed_decode_attention_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                             c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int,
-                                            c_void_p, c_void_p, c_void_p, c_void_p],
+                                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
         "mir_set_option": [ctypes.c_char_p, c_int],
         "mir_get_option": [ctypes.c_char_p],
         "mir_gemm_bf16_lt_batched": [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_int,
@@ -1433,7 +1433,7 @@ def mixed_decode_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.
                            dim: int, value_dim: int, scale: float, head_mix: torch.Tensor, window: Optional[int],
                            chunk: Optional[int], longest: int, alloc) -> None:
     """paged_attention_mixed for a batch of single tokens (row r of qkv belongs to request row r, none of which has more
-    than `longest` tokens), bfloat16, the keys in parts of 64 over CTAs: scores, weights and values, sum of the parts."""
+    than `longest` tokens), bfloat16, the keys in parts of 64 over CTAs: scores, then weights and values (the last part of a kv head adds the parts)."""
     _check_mixed("mixed_decode_attention", qkv, out, k_pages, v_pages, block_table, head_mix, heads, kv_heads, dim, value_dim)
     rows = out.shape[0]
     _require(out.dtype == torch.bfloat16 and positions.dtype == torch.int32 and positions.numel() >= rows
@@ -1442,12 +1442,13 @@ def mixed_decode_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.
     scores = alloc((rows, heads, parts * 64), torch.float32)
     stats = alloc((rows, heads, parts, 2), torch.float32)
     partial = alloc((rows, parts, heads, value_dim), torch.float32)
+    arrived = alloc((rows, heads), torch.int32)
     lib = library("bf16")
     _check(lib, lib.mir_mixed_decode_attention_bf16(
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
         block_table.shape[1], positions.data_ptr(), rows, page_size, heads, kv_heads, dim, value_dim, scale,
         head_mix.data_ptr(), int(window or 0), int(chunk or 0), parts, scores.data_ptr(), stats.data_ptr(),
-        partial.data_ptr(), _stream()))
+        partial.data_ptr(), arrived.data_ptr(), _stream()))
 
 
 MIXED_SLAB_BYTES = 256 << 20     # how much of the mixed weights of a prompt is in memory at a time
