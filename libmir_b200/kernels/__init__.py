@@ -190,6 +190,11 @@ _SIGNATURES = {
         "mir_mixed_prefill_attention_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
                                              c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
+        "mir_mixed_attention_tc_error": [],
+        "mir_mixed_prefill_tc_takes": [c_int, c_int, c_int],
+        "mir_mixed_prefill_attention_tc_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                                c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
+                                                c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
         "mir_mixed_decode_takes": [c_int, c_int, c_int, c_int],
         "mir_mixed_decode_attention_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                             c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int,
@@ -1413,6 +1418,11 @@ def paged_attention_mixed(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.T
         heads, kv_heads, dim, value_dim, scale, head_mix.data_ptr(), int(window or 0), int(chunk or 0), _stream()))
 
 
+def mixed_attention_error() -> int:
+    """0, or which of the tcgen05 kernels for mixed heads gave up a bounded wait (synchronises the device)."""
+    return int(library("bf16").mir_mixed_attention_tc_error())
+
+
 def mixed_decode_takes(heads: int, kv_heads: int, dim: int, value_dim: int) -> bool:
     """Whether single tokens of these sizes run the split-key kernels for mixed heads (bfloat16 only)."""
     return bool(library("bf16").mir_mixed_decode_takes(heads, kv_heads, dim, value_dim))
@@ -1452,30 +1462,50 @@ def mixed_decode_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.
 
 
 MIXED_SLAB_BYTES = 256 << 20     # how much of the mixed weights of a prompt is in memory at a time
-MIXED_SEGMENT_TILES = 4          # tiles of 64 keys that a CTA of the mixing kernel goes through
+MIXED_SEGMENT_TILES = 4          # tiles of 64 keys that a CTA of the mma.sync mixing kernel goes through
+MIXED_TC_SEGMENT_TILES = 3       # tiles of 128 keys that a CTA of the tcgen05 mixing kernel goes through
 
 
 def mixed_prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                             block_table: torch.Tensor, query_starts: torch.Tensor, context_lens: torch.Tensor,
                             page_size: int, heads: int, kv_heads: int, dim: int, value_dim: int, scale: float,
                             head_mix: torch.Tensor, window: Optional[int], chunk: Optional[int], portion_tokens: int,
-                            longest: int, alloc) -> None:
+                            longest: int, alloc, tensor_cores: Optional[bool] = None) -> None:
     """paged_attention_mixed for any mix of portions (row r owns the tokens query_starts[r] .. query_starts[r + 1] of qkv
     and out; the rows may be a part of the batch, with portion_tokens tokens together and at most `longest` tokens each),
-    bfloat16, on tensor cores: the rows' log-sums, the mixed weights, the products with the values."""
+    bfloat16, on tensor cores: the rows' log-sums, the mixed weights, the products with the values.  `tensor_cores`: True
+    runs the tcgen05 kernels (heads of 128 channels), False the mma.sync kernels, None chooses: tcgen05 where they take
+    the sizes and the portions average PREFILL_TENSOR_CORE_MIN_PORTION tokens."""
     _check_mixed("mixed_prefill_attention", qkv, out, k_pages, v_pages, block_table, head_mix, heads, kv_heads, dim, value_dim)
     rows, tokens = context_lens.numel(), out.shape[0]
     _require(out.dtype == torch.bfloat16 and query_starts.dtype == torch.int32 and context_lens.dtype == torch.int32
              and query_starts.numel() == rows + 1 and block_table.shape[0] >= rows, "mixed_prefill_attention: bad metadata")
+    lib = library("bf16")
+    span = _visible_span(longest, window, chunk)
+    if tensor_cores is None:
+        tensor_cores = (PREFILL_TENSOR_CORES and portion_tokens >= PREFILL_TENSOR_CORE_MIN_PORTION * rows and scale > 0
+                        and bool(lib.mir_mixed_prefill_tc_takes(heads, dim, value_dim)))
+    log_sums = alloc((heads, tokens), torch.float32)
+    if tensor_cores:
+        tiles = portion_tokens // 128 + rows
+        # keys of a tile of 128 queries, from the multiple of 128 at or below the first one that is seen
+        key_columns = 128 * min(-(-(min(longest, span + 127) + 127) // 128), -(-longest // 128))
+        tile_bytes = heads * 128 * key_columns * 2
+        slab_tiles = max(1, min(tiles, MIXED_SLAB_BYTES // tile_bytes))
+        mixed = alloc((slab_tiles * tile_bytes,), torch.uint8)
+        _check(lib, lib.mir_mixed_prefill_attention_tc_bf16(
+            qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
+            block_table.shape[1], query_starts.data_ptr(), context_lens.data_ptr(), rows, tokens, page_size, heads, kv_heads,
+            dim, value_dim, scale, head_mix.data_ptr(), int(window or 0), int(chunk or 0), tiles, slab_tiles, key_columns,
+            MIXED_TC_SEGMENT_TILES, log_sums.data_ptr(), mixed.data_ptr(), _stream()))
+        return
     tiles = portion_tokens // 64 + rows              # (a row's last tile may be short)
     # keys of a tile of 16 queries: what the first and the last of them see, from the multiple of 64 below on
-    span = min(longest, _visible_span(longest, window, chunk) + 15)
+    span = min(longest, span + 15)
     key_blocks = 8 * min(-(-(span + 63) // 64), -(-longest // 64))
     tile_bytes = 4 * heads * key_blocks * 256
     slab_tiles = max(1, min(tiles, MIXED_SLAB_BYTES // tile_bytes))
-    log_sums = alloc((heads, tokens), torch.float32)
     mixed = alloc((slab_tiles * tile_bytes,), torch.uint8)
-    lib = library("bf16")
     _check(lib, lib.mir_mixed_prefill_attention_bf16(
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
         block_table.shape[1], query_starts.data_ptr(), context_lens.data_ptr(), rows, tokens, page_size, heads, kv_heads,

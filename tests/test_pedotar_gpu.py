@@ -251,6 +251,10 @@ MIXED_CASES = [
     (BF16, 1, 1, 64, 128, 4, None, 64, "tiles"),
     (BF16, 12, 3, 128, 128, 16, None, 50, "tiles"),
     (BF16, 32, 8, 128, 64, 32, None, 101, "tiles"),
+    (BF16, 32, 8, 128, 128, 16, None, 150, "tiles"),
+    (BF16, 6, 2, 128, 128, 8, 140, None, "tiles"),
+    (BF16, 24, 1, 128, 128, 16, None, None, "tiles"),
+    (BF16, 16, 4, 128, 128, 32, None, 128, "tiles"),
     (BF16, 16, 2, 64, 64, 8, 77, None, "tiles"),
     (BF16, 20, 20, 128, 128, 8, None, None, "tiles"),
     (BF16, 4, 4, 64, 64, 16, None, 1, "tiles"),
@@ -316,13 +320,15 @@ def test_mixed_heads_where_keys_at_the_edges_of_a_run_stand_out(dtype, heads, kv
             for slab in (kernels.MIXED_SLAB_BYTES, 1):           # (1: a slab of one tile at a time)
                 before, kernels.MIXED_SLAB_BYTES = kernels.MIXED_SLAB_BYTES, slab
                 try:
-                    out.fill_(float("nan"))
-                    kernels.mixed_prefill_attention(rows, out, k_pool, v_pool, table, starts, ints(lengths), page, heads,
-                                                    kv_heads, dim, vdim, scale, mix, window, chunk, sum(counts), max(lengths),
-                                                    scratch)
+                    for tensor_cores in (False, True) if dim == vdim == 128 else (False,):
+                        out.fill_(float("nan"))
+                        kernels.mixed_prefill_attention(rows, out, k_pool, v_pool, table, starts, ints(lengths), page, heads,
+                                                        kv_heads, dim, vdim, scale, mix, window, chunk, sum(counts),
+                                                        max(lengths), scratch, tensor_cores=tensor_cores)
+                        close(out, want, tol, f"tile kernels, tcgen05 {tensor_cores}, slab {slab}")
+                    assert kernels.mixed_attention_error() == 0
                 finally:
                     kernels.MIXED_SLAB_BYTES = before
-                close(out, want, tol, "tile kernels")
     if dtype == BF16:
         singles = [(r, n - 1, n) for r, n in enumerate(lengths)]
         want = torch.cat([wants[r][a:b] for r, a, b in singles])
