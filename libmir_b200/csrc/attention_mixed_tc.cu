@@ -97,19 +97,32 @@ __device__ __forceinline__ bool find_tile(int index, const int* query_starts, co
   return false;
 }
 
-// 128 rows of 128 elements (key or value rows of one kv head, from the pages) into the two swizzled halves at `dst`; rows at
-// `limit` and beyond and rows whose page was given back are zeros.
-template <int THREADS>
-__device__ __forceinline__ void load_rows(uint32_t dst, const bf16* __restrict__ pages, const int* __restrict__ table,
-                                          int page_size, int kv_heads, int kv_head, int key0, int limit) {
-  constexpr int ROWS = THREADS / 16;
-  const int sub = threadIdx.x / 16, piece = threadIdx.x % 16;
+// ROWS rows of 128 elements (key or value rows of one kv head, from the pages) into two swizzled halves at `dst`, by
+// WARPS warps: a warp copies whole rows, sixteen lanes a row, two rows at a time.  Which cache rows its 2 * COPIES rows are
+// is looked up once, a lane a row, and kept by the caller (the tile's other kv heads lie beside them): -1 for rows at `limit`
+// and beyond and rows whose page was given back, which become zeros.
+template <int ROWS, int WARPS>
+__device__ __forceinline__ int cache_row(const int* __restrict__ table, int page_size, int key0, int limit, int warp, int lane) {
+  constexpr int COPIES = ROWS / (2 * WARPS);
+  static_assert(ROWS % (2 * WARPS) == 0 && 2 * COPIES <= 32, "a warp looks up its rows at once");
+  const int key = key0 + (lane >> 1) * (2 * WARPS) + warp * 2 + (lane & 1);
+  if (lane >= 2 * COPIES || key >= limit) return -1;
+  const int block = key / page_size, page = table[block];
+  return page < 0 ? -1 : page * page_size + (key - block * page_size);
+}
+template <int ROWS, int WARPS>
+__device__ __forceinline__ void load_rows(uint32_t dst, const bf16* __restrict__ pages, int kv_heads, int kv_head, int mine,
+                                          int warp, int lane) {
+  constexpr int COPIES = ROWS / (2 * WARPS);
+  const int piece = lane & 15, second = lane >> 4;
+  const bf16* const from = pages + (size_t)kv_head * kDim + piece * 8;
+  const size_t row_stride = (size_t)kv_heads * kDim;
 #pragma unroll
-  for (int i = 0; i < kTile; i += ROWS) {
-    const int r = i + sub, key = key0 + r;
-    const int page = key < limit ? table[key / page_size] : -1;
-    const bf16* from = page >= 0 ? pages + (((size_t)page * page_size + key % page_size) * kv_heads + kv_head) * kDim + piece * 8 : pages;
-    copy16(dst + (piece >> 3) * kHalf + r * 128 + (((piece & 7) ^ (r & 7)) << 4), from, page >= 0);
+  for (int i = 0; i < COPIES; ++i) {
+    const int r = i * (2 * WARPS) + warp * 2 + second;
+    const int row = __shfl_sync(0xffffffffu, mine, i * 2 + second);
+    copy16(dst + (piece >> 3) * (ROWS * 128) + r * 128 + (((piece & 7) ^ (r & 7)) << 4),
+           row >= 0 ? from + row * row_stride : pages, row >= 0);
   }
 }
 
@@ -156,7 +169,8 @@ mixed_row_sums_tc_kernel(const bf16* __restrict__ q, long long q_stride, const b
   __shared__ __align__(8) uint64_t barriers[2];
   __shared__ float tops[2][kTile], sums[2][kTile];
   QueryTile w;
-  if (!find_tile(blockIdx.y, query_starts, context_lens, rows, window, chunk, w)) return;
+  // (late tiles of a request see the most keys: they come first)
+  if (!find_tile(gridDim.y - 1 - blockIdx.y, query_starts, context_lens, rows, window, chunk, w)) return;
   const uint32_t base = (smem_u32(dynamic) + 1023u) & ~1023u;
   const uint32_t q_at = base, k_at = base + kOperand;
   const int head = blockIdx.x, kv_head = head / (heads / kv_heads);
@@ -167,7 +181,8 @@ mixed_row_sums_tc_kernel(const bf16* __restrict__ q, long long q_stride, const b
 
   auto fetch = [&](int t) {
     if (t < tiles)
-      load_rows<256>(k_at + (t & 1) * kOperand, k_pages, table, page_size, kv_heads, kv_head, w.key_begin + t * kTile, w.key_end);
+      load_rows<kTile, 8>(k_at + (t & 1) * kOperand, k_pages, kv_heads, kv_head,
+                          cache_row<kTile, 8>(table, page_size, w.key_begin + t * kTile, w.key_end, warp, lane), warp, lane);
     copy_commit();
   };
   for (int i = threadIdx.x; i < kTile * 16; i += 256) {
@@ -266,11 +281,17 @@ __device__ __forceinline__ void tmem_request_wait(uint32_t (&r)[8]) {
 }
 
 __host__ __device__ constexpr int queries_for(int padded_heads) { return padded_heads == 32 ? 16 : 32; }
+constexpr int kMixers = 256, kLoaders = 128;
+constexpr int kMixerRegisters = 216, kLoaderRegisters = 72;      // together what 384 threads are launched with (168 each)
 
-// grid (segments of the keys, 128 / Q x tiles of 128 queries), 256 threads, Q queries and all heads.  Thread: key = its lane
-// of the accumulators (four warps), half of the queries (two sets of four warps).
+// Barriers of the mixing kernel: a stage's keys are there, its products are over, all scores of a tile are there.
+enum { KEYS_FULL = 0, KEYS_FREE = 2, SCORES_FULL = 4, WEIGHTS_BARRIERS = 5 };
+
+// grid (segments of the keys, 128 / Q x tiles of 128 queries), kMixers + kLoaders threads, Q queries and all heads.  Mixer:
+// key = its lane of the accumulators (four warps), half of the queries (two sets of four warps); the first of their warps
+// issues the products as keys arrive.  Loaders: the key tiles of one kv head after the other, two stages ahead.
 template <int HEADS>
-__global__ void __launch_bounds__(256, 1)
+__global__ void __launch_bounds__(kMixers + kLoaders, 1)
 mixed_weights_tc_kernel(const bf16* __restrict__ q, long long q_stride, const bf16* __restrict__ k_pages,
                         const int* __restrict__ block_table, int table_width, const int* __restrict__ query_starts,
                         const int* __restrict__ context_lens, int rows, int page_size, int heads, int kv_heads, float scale2,
@@ -278,15 +299,17 @@ mixed_weights_tc_kernel(const bf16* __restrict__ q, long long q_stride, const bf
                         int first_tile, int segment_tiles, int key_columns, bf16* __restrict__ mixed) {
   constexpr int Q = queries_for(HEADS), SUBS = kTile / Q;
   constexpr int QB = HEADS == 32 ? 4 : 8;                        // queries a thread mixes at a time
+  constexpr int GB = HEADS == 32 ? 4 : 2;                        // heads whose scores it asks for at a time
   constexpr uint32_t COLUMNS = HEADS * Q;
   extern __shared__ unsigned char dynamic[];
   __shared__ uint32_t tmem_place;
-  __shared__ __align__(8) uint64_t barriers[2];
+  __shared__ __align__(8) uint64_t barriers[WEIGHTS_BARRIERS];
   __shared__ __align__(16) float mix_s[HEADS * HEADS];           // [head][result head]
   __shared__ __align__(16) float sums_s[HEADS * Q];              // [head][query]
   QueryTile w;
-  if (!find_tile(first_tile + blockIdx.y / SUBS, query_starts, context_lens, rows, window, chunk, w)) return;
-  const int sub = blockIdx.y % SUBS;
+  const int index = gridDim.y - 1 - blockIdx.y;                  // (late tiles of a request see the most keys: they come first)
+  if (!find_tile(first_tile + index / SUBS, query_starts, context_lens, rows, window, chunk, w)) return;
+  const int sub = index % SUBS;
   const int here = min(Q, w.here - sub * Q);
   if (here <= 0) return;
   const int tiles = min((w.key_end - w.key_begin + kTile - 1) / kTile, key_columns / kTile);
@@ -296,11 +319,11 @@ mixed_weights_tc_kernel(const bf16* __restrict__ q, long long q_stride, const bf
   // the key tiles that one of these queries sees; the others of the segment are zeros
   const int seen_begin = max(segment_begin, (first_visible(position0, window, chunk) - w.key_begin) / kTile);
   const int seen_end = min(segment_end, (position0 + here - w.key_begin + kTile - 1) / kTile);
-  bf16* const result = mixed + ((size_t)(blockIdx.y / SUBS) * heads * kTile + sub * Q) * key_columns;
+  bf16* const result = mixed + ((size_t)(index / SUBS) * heads * kTile + sub * Q) * key_columns;
   const size_t head_stride = (size_t)kTile * key_columns;
   for (int kt = segment_begin; kt < segment_end; ++kt) {
     if (kt >= seen_begin && kt < seen_end) continue;
-    for (int i = threadIdx.x; i < heads * here * 16; i += 256) {
+    for (int i = threadIdx.x; i < heads * here * 16; i += kMixers + kLoaders) {
       const int row = i / 16, h = row / here, query = row - h * here;
       *reinterpret_cast<uint4*>(result + h * head_stride + (size_t)query * key_columns + kt * kTile + i % 16 * 8) = make_uint4(0u, 0u, 0u, 0u);
     }
@@ -310,133 +333,170 @@ mixed_weights_tc_kernel(const bf16* __restrict__ q, long long q_stride, const bf
   const uint32_t base = (smem_u32(dynamic) + 1023u) & ~1023u;
   const uint32_t q_half = (uint32_t)(Q * heads) * 128u;          // bytes of a 64-element half of all the queries' rows
   const uint32_t k_at = base, q_at = base + 2 * kOperand;
-  const int* table = block_table + (size_t)w.row * table_width;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int per_group = heads / kv_heads;
-  const uint32_t tmem = allocate(&tmem_place, COLUMNS, barriers, 2);
+  const uint32_t bar = smem_u32(barriers);
+  if (threadIdx.x == 0)
+    for (int i = 0; i < WEIGHTS_BARRIERS; ++i) barrier_init(bar + i * 8, i < KEYS_FREE ? kLoaders : 1);
+  const uint32_t tmem = allocate(&tmem_place, COLUMNS, nullptr, 0);
   const int steps = (seen_end - seen_begin) * kv_heads;
-  auto fetch = [&](int step) {
-    if (step < steps)
-      load_rows<256>(k_at + (step & 1) * kOperand, k_pages, table, page_size, kv_heads, step % kv_heads,
-                     w.key_begin + (seen_begin + step / kv_heads) * kTile, w.key_end);
-    copy_commit();
-  };
-  // row head * Q + query of the second operand
-  for (int i = threadIdx.x; i < heads * Q * 16; i += 256) {
-    const int row = i / 16, piece = i % 16, query = row % Q;
-    const bool there = query < here;
-    copy16(q_at + (piece >> 3) * q_half + row * 128 + (((piece & 7) ^ (row & 7)) << 4),
-           there ? q + (size_t)(token0 + query) * q_stride + (size_t)(row / Q) * kDim + piece * 8 : q, there);
-  }
-  fetch(0);
-  fetch(1);
-  for (int i = threadIdx.x; i < HEADS * HEADS; i += 256) {
-    const int g = i / HEADS, h = i % HEADS;
-    mix_s[i] = g < heads && h < heads ? mix[h * heads + g] : 0.0f;
-  }
-  for (int i = threadIdx.x; i < HEADS * Q; i += 256) {
-    const int g = i / Q, query = i % Q;
-    sums_s[i] = g < heads && query < here ? log_sums[(size_t)g * tokens + token0 + query] : 0.0f;
-  }
-  const int quarter = (warp & 3) * 32, half = warp >> 2;
-  const uint32_t lane_at = tmem + ((uint32_t)quarter << 16);
   bool alive = true;
-  int step = 0;
-  for (int kt = seen_begin; kt < seen_end; ++kt) {
-    for (int group = 0; group < kv_heads; ++group, ++step) {
-      const int stage = step & 1;
-      copy_wait<1>();
-      fence_for_tensor_cores();
+
+  if (threadIdx.x >= kMixers) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kLoaderRegisters));
+    const int* table = block_table + (size_t)w.row * table_width;
+    int mine = -1;
+    for (int step = 0; step < steps; ++step) {
+      const int stage = step & 1, kv_head = step % kv_heads;
+      if (kv_head == 0)
+        mine = cache_row<kTile, 4>(table, page_size, w.key_begin + (seen_begin + step / kv_heads) * kTile, w.key_end, warp - 8, lane);
+      if (step >= 2) wait_alive(bar + (KEYS_FREE + stage) * 8, ((step >> 1) - 1) & 1, alive, 2);
+      __syncwarp();
+      load_rows<kTile, 4>(k_at + stage * kOperand, k_pages, kv_heads, kv_head, mine, warp - 8, lane);
+      copy_commit();
+      if (step > 0) {                                            // the stage before: it has landed, and the tensor cores may see it
+        copy_wait<1>();
+        fence_for_tensor_cores();
+        barrier_arrive(bar + (KEYS_FULL + (stage ^ 1)) * 8);
+      }
+    }
+    copy_wait<0>();
+    fence_for_tensor_cores();
+    barrier_arrive(bar + (KEYS_FULL + ((steps - 1) & 1)) * 8);
+  } else {
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(kMixerRegisters));
+    // row head * Q + query of the second operand
+    for (int i = threadIdx.x; i < heads * Q * 16; i += kMixers) {
+      const int row = i / 16, piece = i % 16, query = row % Q;
+      const bool there = query < here;
+      copy16(q_at + (piece >> 3) * q_half + row * 128 + (((piece & 7) ^ (row & 7)) << 4),
+             there ? q + (size_t)(token0 + query) * q_stride + (size_t)(row / Q) * kDim + piece * 8 : q, there);
+    }
+    copy_commit();
+    for (int i = threadIdx.x; i < HEADS * HEADS; i += kMixers) {
+      const int g = i / HEADS, h = i % HEADS;
+      mix_s[i] = g < heads && h < heads ? mix[h * heads + g] : 0.0f;
+    }
+    for (int i = threadIdx.x; i < HEADS * Q; i += kMixers) {
+      const int g = i / Q, query = i % Q;
+      sums_s[i] = g < heads && query < here ? log_sums[(size_t)g * tokens + token0 + query] : 0.0f;
+    }
+    copy_wait<0>();
+    fence_for_tensor_cores();
+    const int quarter = (warp & 3) * 32, half = warp >> 2;
+    const uint32_t lane_at = tmem + ((uint32_t)quarter << 16);
+    int step = 0;
+    for (int kt = seen_begin; kt < seen_end; ++kt) {
       tensor_fence_before_sync();                                // (the last tile's scores have been read)
-      __syncthreads();
+      asm volatile("bar.sync 1, %0;" ::"n"(kMixers) : "memory");
       if (warp == 0) {
         tensor_fence_after_sync();
         const uint32_t elected = elect_one();
-        const uint32_t a = operand_low(k_at + stage * kOperand);
-        for (int n0 = 0; n0 < per_group * Q; n0 += 256) {
-          const uint32_t idesc = instruction_descriptor(kTile, min(256, per_group * Q - n0));
-          const uint32_t b = operand_low(q_at + (uint32_t)(group * per_group * Q + n0) * 128u);
+        for (int group = 0; group < kv_heads; ++group, ++step) {
+          const int stage = step & 1;
+          wait_alive(bar + (KEYS_FULL + stage) * 8, (step >> 1) & 1, alive, 2);
+          __syncwarp();
+          tensor_fence_after_sync();
+          const uint32_t a = operand_low(k_at + stage * kOperand);
+          for (int n0 = 0; n0 < per_group * Q; n0 += 256) {
+            const uint32_t idesc = instruction_descriptor(kTile, min(256, per_group * Q - n0));
+            const uint32_t b = operand_low(q_at + (uint32_t)(group * per_group * Q + n0) * 128u);
 #pragma unroll
-          for (int k = 0; k < 8; ++k)
-            mma_bf16_ss_halves(tmem + group * per_group * Q + n0, a + (k >> 2) * (kHalf >> 4) + (k & 3) * 2,
-                               b + (k >> 2) * (q_half >> 4) + (k & 3) * 2, idesc, (uint32_t)(k > 0), elected);
+            for (int k = 0; k < 8; ++k)
+              mma_bf16_ss_halves(tmem + group * per_group * Q + n0, a + (k >> 2) * (kHalf >> 4) + (k & 3) * 2,
+                                 b + (k >> 2) * (q_half >> 4) + (k & 3) * 2, idesc, (uint32_t)(k > 0), elected);
+          }
+          mma_commit_elected(bar + (KEYS_FREE + stage) * 8, elected);
         }
-        mma_commit_elected(smem_u32(barriers + stage), elected);
+        mma_commit_elected(bar + SCORES_FULL * 8, elected);
       }
-      wait_alive(smem_u32(barriers + stage), (step >> 1) & 1, alive, 2);
-      fetch(step + 2);
-    }
-    tensor_fence_after_sync();
-    const int key = w.key_begin + kt * kTile + quarter + lane;
+      wait_alive(bar + SCORES_FULL * 8, (kt - seen_begin) & 1, alive, 2);
+      __syncwarp();
+      tensor_fence_after_sync();
+      const int key = w.key_begin + kt * kTile + quarter + lane;
 #pragma unroll 1
-    for (int q0 = half * (Q / 2); q0 < (half + 1) * (Q / 2); q0 += QB) {
-      bool seen[QB];
-#pragma unroll
-      for (int i = 0; i < QB; ++i) {
-        const int position = position0 + q0 + i;
-        seen[i] = q0 + i < here && key <= position && key >= first_visible(position, window, chunk);
-      }
-      pair32 acc[QB][HEADS / 2];
-#pragma unroll
-      for (int i = 0; i < QB; ++i)
-#pragma unroll
-        for (int h = 0; h < HEADS / 2; ++h) acc[i][h] = 0ull;
-      auto add_head = [&](int g, const uint32_t (&scores)[QB]) {
-        pair32 weight[QB];
+      for (int q0 = half * (Q / 2); q0 < (half + 1) * (Q / 2); q0 += QB) {
+        bool seen[QB];
 #pragma unroll
         for (int i = 0; i < QB; ++i) {
-          const float v = seen[i] ? fast_exp2(fmaf(__uint_as_float(scores[i]), scale2, -sums_s[g * Q + q0 + i])) : 0.0f;
-          weight[i] = make_pair(v, v);
+          const int position = position0 + q0 + i;
+          seen[i] = q0 + i < here && key <= position && key >= first_visible(position, window, chunk);
         }
-        const ulonglong2* factors = reinterpret_cast<const ulonglong2*>(mix_s + g * HEADS);
+        pair32 acc[QB][HEADS / 2];
 #pragma unroll
-        for (int h = 0; h < HEADS / 4; ++h) {
-          const ulonglong2 m = factors[h];
+        for (int i = 0; i < QB; ++i)
 #pragma unroll
-          for (int i = 0; i < QB; ++i) {
-            acc[i][2 * h] = fma_pair(m.x, weight[i], acc[i][2 * h]);
-            acc[i][2 * h + 1] = fma_pair(m.y, weight[i], acc[i][2 * h + 1]);
+          for (int h = 0; h < HEADS / 2; ++h) acc[i][h] = 0ull;
+        auto request = [&](int g, uint32_t (&scores)[GB][QB]) {  // (columns behind the last head: read, and not used)
+#pragma unroll
+          for (int e = 0; e < GB; ++e) tmem_request<QB>(lane_at + (g + e) * Q + q0, scores[e]);
+        };
+        auto add_heads = [&](int g, uint32_t (&scores)[GB][QB]) {
+#pragma unroll
+          for (int e = 0; e < GB; ++e)
+#pragma unroll
+            for (int i = 0; i < QB; ++i) {
+              const float v = fast_exp2(fmaf(__uint_as_float(scores[e][i]), scale2, -sums_s[(g + e) * Q + q0 + i]));
+              scores[e][i] = seen[i] && g + e < heads ? __float_as_uint(v) : 0u;
+            }
+#pragma unroll
+          for (int e = 0; e < GB; ++e) {
+            const ulonglong2* factors = reinterpret_cast<const ulonglong2*>(mix_s + (g + e) * HEADS);
+            pair32 weight[QB];
+#pragma unroll
+            for (int i = 0; i < QB; ++i) weight[i] = make_pair(__uint_as_float(scores[e][i]), __uint_as_float(scores[e][i]));
+#pragma unroll
+            for (int h = 0; h < HEADS / 4; ++h) {
+              const ulonglong2 m = factors[h];
+#pragma unroll
+              for (int i = 0; i < QB; ++i) {
+                acc[i][2 * h] = fma_pair(m.x, weight[i], acc[i][2 * h]);
+                acc[i][2 * h + 1] = fma_pair(m.y, weight[i], acc[i][2 * h + 1]);
+              }
+            }
           }
-        }
-      };
-      // a head's scores are on their way while the head before is added
-      uint32_t even_head[QB], odd_head[QB];
-      tmem_request<QB>(lane_at + q0, even_head);
-      tmem_request_wait(even_head);
+        };
+        auto arrived = [&](uint32_t (&scores)[GB][QB]) {
+#pragma unroll
+          for (int e = 0; e < GB; ++e) tmem_request_wait(scores[e]);
+        };
+        // some heads' scores are on their way while the heads before are added
+        uint32_t front[GB][QB], back[GB][QB];
+        request(0, front);
+        arrived(front);
 #pragma unroll 1
-      for (int g = 0; g < heads; g += 2) {
-        if (g + 1 < heads) tmem_request<QB>(lane_at + (g + 1) * Q + q0, odd_head);
-        add_head(g, even_head);
-        if (g + 1 < heads) {
-          tmem_request_wait(odd_head);
-          if (g + 2 < heads) tmem_request<QB>(lane_at + (g + 2) * Q + q0, even_head);
-          add_head(g + 1, odd_head);
-          if (g + 2 < heads) tmem_request_wait(even_head);
+        for (int g = 0; g < heads; g += 2 * GB) {
+          request(g + GB, back);
+          add_heads(g, front);
+          arrived(back);
+          if (g + 2 * GB < heads) request(g + 2 * GB, front);
+          add_heads(g + GB, back);
+          if (g + 2 * GB < heads) arrived(front);
         }
-      }
-      // neighbouring lanes hold neighbouring keys: the even one stores both keys of a query, the odd one of the next query
-      const bool even = (lane & 1) == 0;
+        // neighbouring lanes hold neighbouring keys: the even one stores both keys of a query, the odd one of the next query
+        const bool even = (lane & 1) == 0;
 #pragma unroll
-      for (int i = 0; i < QB; i += 2) {
-        const int query = q0 + i + (even ? 0 : 1);
-        bf16* to = result + (size_t)query * key_columns + kt * kTile + quarter + (lane & ~1);
-        const bool there = query < here;
+        for (int i = 0; i < QB; i += 2) {
+          const int query = q0 + i + (even ? 0 : 1);
+          bf16* to = result + (size_t)query * key_columns + kt * kTile + quarter + (lane & ~1);
+          const bool there = query < here;
 #pragma unroll
-        for (int h = 0; h < HEADS / 2; ++h) {
-          float a0, a1, b0, b1;
-          split_pair(acc[i][h], a0, a1);
-          split_pair(acc[i + 1][h], b0, b1);
-          const float other0 = __shfl_xor_sync(0xffffffffu, even ? b0 : a0, 1);
-          const float other1 = __shfl_xor_sync(0xffffffffu, even ? b1 : a1, 1);
-          if (there && 2 * h < heads)
-            *reinterpret_cast<uint32_t*>(to + (2 * h) * head_stride) = even ? pack_bf16(a0, other0) : pack_bf16(other0, b0);
-          if (there && 2 * h + 1 < heads)
-            *reinterpret_cast<uint32_t*>(to + (2 * h + 1) * head_stride) = even ? pack_bf16(a1, other1) : pack_bf16(other1, b1);
+          for (int h = 0; h < HEADS / 2; ++h) {
+            float a0, a1, b0, b1;
+            split_pair(acc[i][h], a0, a1);
+            split_pair(acc[i + 1][h], b0, b1);
+            const float other0 = __shfl_xor_sync(0xffffffffu, even ? b0 : a0, 1);
+            const float other1 = __shfl_xor_sync(0xffffffffu, even ? b1 : a1, 1);
+            if (there && 2 * h < heads)
+              *reinterpret_cast<uint32_t*>(to + (2 * h) * head_stride) = even ? pack_bf16(a0, other0) : pack_bf16(other0, b0);
+            if (there && 2 * h + 1 < heads)
+              *reinterpret_cast<uint32_t*>(to + (2 * h + 1) * head_stride) = even ? pack_bf16(a1, other1) : pack_bf16(other1, b1);
+          }
         }
       }
     }
   }
-  copy_wait<0>();
+  __syncwarp();
   release(tmem, COLUMNS);
 }
 
@@ -455,13 +515,14 @@ mixed_values_tc_kernel(const bf16* __restrict__ mixed, bf16* __restrict__ out, c
   __shared__ uint32_t tmem_place;
   __shared__ __align__(8) uint64_t barriers[kSlabStages];
   QueryTile w;
-  if (!find_tile(first_tile + blockIdx.y, query_starts, context_lens, rows, window, chunk, w)) return;
+  const int local_tile = gridDim.y - 1 - blockIdx.y;             // (late tiles of a request see the most keys: they come first)
+  if (!find_tile(first_tile + local_tile, query_starts, context_lens, rows, window, chunk, w)) return;
   const uint32_t base = (smem_u32(dynamic) + 1023u) & ~1023u;
   const int head = blockIdx.x, kv_head = head / (heads / kv_heads);
   const int* table = block_table + (size_t)w.row * table_width;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int slabs = min((w.key_end - w.key_begin + kSlab - 1) / kSlab, key_columns / kSlab);
-  const bf16* const weights = mixed + ((size_t)blockIdx.y * heads + head) * kTile * key_columns;
+  const bf16* const weights = mixed + ((size_t)local_tile * heads + head) * kTile * key_columns;
   const uint32_t tmem = allocate(&tmem_place, 128, barriers, kSlabStages);
 
   auto fetch = [&](int s) {
@@ -473,14 +534,8 @@ mixed_values_tc_kernel(const bf16* __restrict__ mixed, bf16* __restrict__ out, c
         const bool there = r < w.here;
         copy16(a + r * 128 + ((piece ^ (r & 7)) << 4), there ? weights + (size_t)r * key_columns + s * kSlab + piece * 8 : weights, there);
       }
-      const int sub = threadIdx.x / 16, piece = threadIdx.x % 16;
-#pragma unroll
-      for (int i = 0; i < kSlab; i += 16) {
-        const int r = i + sub, key = w.key_begin + s * kSlab + r;
-        const int page = key < w.key_end ? table[key / page_size] : -1;
-        const bf16* from = page >= 0 ? v_pages + (((size_t)page * page_size + key % page_size) * kv_heads + kv_head) * kDim + piece * 8 : v_pages;
-        copy16(v + (piece >> 3) * (kSlab * 128) + r * 128 + (((piece & 7) ^ (r & 7)) << 4), from, page >= 0);
-      }
+      load_rows<kSlab, 8>(v, v_pages, kv_heads, kv_head,
+                          cache_row<kSlab, 8>(table, page_size, w.key_begin + s * kSlab, w.key_end, warp, lane), warp, lane);
     }
     copy_commit();
   };
@@ -583,7 +638,7 @@ MIR_EXPORT int mir_mixed_prefill_attention_tc_bf16(const void* q, long long q_st
   do {                                                                                                                   \
     const size_t smem = 2 * kOperand + (size_t)queries_for(H) * heads * 256 + 1024;                                      \
     if ((status = reserve((const void*)mixed_weights_tc_kernel<H>, smem, "mixed_weights_tc")) != MIR_OK) return status;  \
-    mixed_weights_tc_kernel<H><<<dim3(segments, here * (kTile / queries_for(H))), 256, smem, stream>>>(                  \
+    mixed_weights_tc_kernel<H><<<dim3(segments, here * (kTile / queries_for(H))), kMixers + kLoaders, smem, stream>>>(                  \
         qb, q_stride, kb, block_table, table_width, query_starts, context_lens, rows, page_size, heads, kv_heads, scale2, \
         window, chunk, mix, log_sums, tokens, from, segment_tiles, key_columns, (bf16*)mixed);                           \
   } while (0)
