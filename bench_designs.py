@@ -671,13 +671,14 @@ def pedotar_kernel_table(s, tools) -> dict:
         v_cache = [rand(cache_rows, kv_heads, dim, scale=0.5) for _ in range(banks)]
         qkv = rand(tokens, (heads + 2 * kv_heads) * dim, scale=0.3)
         mix = rand(heads, heads, dtype=f32, scale=0.3)
+        host_mix = mix.cpu()
         result = torch.empty(tokens, heads * dim, device=device, dtype=bf16)
         scale = dim ** -0.5
         if prompt:
             seen = sum(p % chunk + 1 for p in range(PROMPT))
             calls = [with_scratch(lambda k=k, v=v: kernels.mixed_prefill_attention(
                 qkv, result, k, v, block_table, starts, contexts, PAGE, heads, kv_heads, dim, dim, scale, mix, None, chunk, tokens,
-                context, alloc)) for k, v in zip(k_cache, v_cache)]
+                context, alloc, host_mix=host_mix)) for k, v in zip(k_cache, v_cache)]
             table[f"{label}_mixed_attention"] = timed(calls, seen * (4.0 * dim * heads + 2.0 * heads * heads), flops_peak)
             in_window = sum(min(p + 1, chunk // 2) for p in range(PROMPT))
             calls = [lambda k=k, v=v: kernels.prefill_attention(qkv, result, k, v, block_table, starts, contexts, PAGE, heads,

@@ -78,18 +78,23 @@ __device__ __forceinline__ int first_visible(int position, int window, int chunk
 struct QueryTile {
   int row, token0, here, position0, key_begin, key_end;          // key_begin is a multiple of 128
 };
+__device__ __forceinline__ QueryTile query_tile(int row, int tile, int begin, int count, int context, int window, int chunk) {
+  QueryTile w;
+  w.row = row;
+  w.token0 = begin + tile * kTile;
+  w.here = min(kTile, count - tile * kTile);
+  w.position0 = context - count + tile * kTile;
+  w.key_begin = first_visible(w.position0, window, chunk) / kTile * kTile;
+  w.key_end = w.position0 + w.here;
+  return w;
+}
 __device__ __forceinline__ bool find_tile(int index, const int* query_starts, const int* context_lens, int rows, int window,
                                           int chunk, QueryTile& w) {
   for (int r = 0; r < rows; ++r) {
     const int begin = query_starts[r], count = query_starts[r + 1] - begin;
     const int tiles = (count + kTile - 1) / kTile;
     if (index < tiles) {
-      w.row = r;
-      w.token0 = begin + index * kTile;
-      w.here = min(kTile, count - index * kTile);
-      w.position0 = context_lens[r] - count + index * kTile;
-      w.key_begin = first_visible(w.position0, window, chunk) / kTile * kTile;
-      w.key_end = w.position0 + w.here;
+      w = query_tile(r, index, begin, count, context_lens[r], window, chunk);
       return true;
     }
     index -= tiles;
@@ -283,53 +288,88 @@ __device__ __forceinline__ void tmem_request_wait(uint32_t (&r)[8]) {
 __host__ __device__ constexpr int queries_for(int padded_heads) { return padded_heads == 32 ? 16 : 32; }
 constexpr int kMixers = 256, kLoaders = 128;
 constexpr int kMixerRegisters = 216, kLoaderRegisters = 72;      // together what 384 threads are launched with (168 each)
+// The mixing matrix comes as a launch parameter: every thread uses the same number at the same time, and a parameter's
+// reach the multiply-adds through the constant cache; the same numbers from shared memory cost 512 bytes of register
+// writes per 16 of them and warp, which bound the kernel.
+struct MixMatrix { float of[32 * 32]; };                         // [head][result head], rows of 8, 16 or 32
 
 // Barriers of the mixing kernel: a stage's keys are there, its products are over, all scores of a tile are there.
 enum { KEYS_FULL = 0, KEYS_FREE = 2, SCORES_FULL = 4, WEIGHTS_BARRIERS = 5 };
 
-// grid (segments of the keys, 128 / Q x tiles of 128 queries), kMixers + kLoaders threads, Q queries and all heads.  Mixer:
-// key = its lane of the accumulators (four warps), half of the queries (two sets of four warps); the first of their warps
-// issues the products as keys arrive.  Loaders: the key tiles of one kv head after the other, two stages ahead.
+// What a CTA works on: Q queries and a segment of their tile's keys.  The items of a launch are counted from its last tile of
+// queries backwards (late tiles of a request see the most keys: they come first), a tile's segments one after the other and
+// within a segment its groups of Q queries; only items that exist are counted, so that a CTA which takes every n-th gets its
+// share.
+struct MixItem {
+  QueryTile w;
+  int sub, here, position0, token0, segment_begin, segment_end, seen_begin, seen_end;
+  // the walk over the tiles: tile `tile` of row `row` is the batch's tile `index`, has `subs` groups of queries and `items`
+  // items, and `passed` items lie behind it
+  int row, tile, index, subs, items, passed;
+};
+__device__ __forceinline__ void start_mix_items(const int* query_starts, int rows, MixItem& m) {
+  m.row = rows;
+  m.tile = m.index = m.items = m.passed = 0;
+  for (int r = 0; r < rows; ++r) m.index += (query_starts[r + 1] - query_starts[r] + kTile - 1) / kTile;
+}
+// Item `rank` of the launch (ranks ascend from call to call); false when there are no more.
+template <int Q>
+__device__ __forceinline__ bool mix_item(int rank, int first_tile, int slab_tiles, const int* query_starts,
+                                         const int* context_lens, int window, int chunk, int segment_tiles, int key_columns,
+                                         MixItem& m) {
+  int tiles = 0;
+  while (rank >= m.passed + m.items) {
+    m.passed += m.items;
+    m.items = 0;
+    while (m.tile == 0) {
+      if (m.row == 0) return false;
+      --m.row;
+      m.tile = (query_starts[m.row + 1] - query_starts[m.row] + kTile - 1) / kTile;
+    }
+    --m.tile;
+    --m.index;
+    if (m.index < first_tile) return false;
+    if (m.index >= first_tile + slab_tiles) continue;
+    const int begin = query_starts[m.row];
+    m.w = query_tile(m.row, m.tile, begin, query_starts[m.row + 1] - begin, context_lens[m.row], window, chunk);
+    tiles = min((m.w.key_end - m.w.key_begin + kTile - 1) / kTile, key_columns / kTile);
+    m.subs = (m.w.here + Q - 1) / Q;
+    m.items = m.subs * ((tiles + segment_tiles - 1) / segment_tiles);
+  }
+  tiles = min((m.w.key_end - m.w.key_begin + kTile - 1) / kTile, key_columns / kTile);
+  const int local = rank - m.passed;
+  m.sub = local % m.subs;
+  m.here = min(Q, m.w.here - m.sub * Q);
+  m.segment_begin = local / m.subs * segment_tiles;
+  m.segment_end = min(m.segment_begin + segment_tiles, tiles);
+  m.token0 = m.w.token0 + m.sub * Q;
+  m.position0 = m.w.position0 + m.sub * Q;
+  // the key tiles that one of these queries sees; the others of the segment are zeros
+  m.seen_begin = max(m.segment_begin, (first_visible(m.position0, window, chunk) - m.w.key_begin) / kTile);
+  m.seen_end = min(m.segment_end, (m.position0 + m.here - m.w.key_begin + kTile - 1) / kTile);
+  return true;
+}
+
+// One CTA per SM goes over the items (a unit of Q queries, a segment of the keys), kMixers + kLoaders threads.  Mixer: key =
+// its lane of the accumulators (four warps), half of the queries (two sets of four warps); the first of their warps
+// issues the products as keys arrive.  Loaders: the key tiles of one kv head after the other, two stages ahead.  Stages and
+// barrier phases run on across the items.
 template <int HEADS>
 __global__ void __launch_bounds__(kMixers + kLoaders, 1)
 mixed_weights_tc_kernel(const bf16* __restrict__ q, long long q_stride, const bf16* __restrict__ k_pages,
                         const int* __restrict__ block_table, int table_width, const int* __restrict__ query_starts,
                         const int* __restrict__ context_lens, int rows, int page_size, int heads, int kv_heads, float scale2,
-                        int window, int chunk, const float* __restrict__ mix, const float* __restrict__ log_sums, int tokens,
-                        int first_tile, int segment_tiles, int key_columns, bf16* __restrict__ mixed) {
-  constexpr int Q = queries_for(HEADS), SUBS = kTile / Q;
+                        int window, int chunk, const __grid_constant__ MixMatrix mix,
+                        const float* __restrict__ log_sums, int tokens, int first_tile, int slab_tiles,
+                        int segment_tiles, int key_columns, bf16* __restrict__ mixed) {
+  constexpr int Q = queries_for(HEADS), SET = Q / (kMixers / 128);
   constexpr int QB = HEADS == 32 ? 4 : 8;                        // queries a thread mixes at a time
-  constexpr int GB = HEADS == 32 ? 4 : 2;                        // heads whose scores it asks for at a time
+  constexpr int GB = HEADS == 32 ? 4 : 2;                                          // heads whose scores it asks for at a time
   constexpr uint32_t COLUMNS = HEADS * Q;
   extern __shared__ unsigned char dynamic[];
   __shared__ uint32_t tmem_place;
   __shared__ __align__(8) uint64_t barriers[WEIGHTS_BARRIERS];
-  __shared__ __align__(16) float mix_s[HEADS * HEADS];           // [head][result head]
   __shared__ __align__(16) float sums_s[HEADS * Q];              // [head][query]
-  QueryTile w;
-  const int index = gridDim.y - 1 - blockIdx.y;                  // (late tiles of a request see the most keys: they come first)
-  if (!find_tile(first_tile + index / SUBS, query_starts, context_lens, rows, window, chunk, w)) return;
-  const int sub = index % SUBS;
-  const int here = min(Q, w.here - sub * Q);
-  if (here <= 0) return;
-  const int tiles = min((w.key_end - w.key_begin + kTile - 1) / kTile, key_columns / kTile);
-  const int segment_begin = blockIdx.x * segment_tiles, segment_end = min(segment_begin + segment_tiles, tiles);
-  if (segment_begin >= segment_end) return;
-  const int token0 = w.token0 + sub * Q, position0 = w.position0 + sub * Q;
-  // the key tiles that one of these queries sees; the others of the segment are zeros
-  const int seen_begin = max(segment_begin, (first_visible(position0, window, chunk) - w.key_begin) / kTile);
-  const int seen_end = min(segment_end, (position0 + here - w.key_begin + kTile - 1) / kTile);
-  bf16* const result = mixed + ((size_t)(index / SUBS) * heads * kTile + sub * Q) * key_columns;
-  const size_t head_stride = (size_t)kTile * key_columns;
-  for (int kt = segment_begin; kt < segment_end; ++kt) {
-    if (kt >= seen_begin && kt < seen_end) continue;
-    for (int i = threadIdx.x; i < heads * here * 16; i += kMixers + kLoaders) {
-      const int row = i / 16, h = row / here, query = row - h * here;
-      *reinterpret_cast<uint4*>(result + h * head_stride + (size_t)query * key_columns + kt * kTile + i % 16 * 8) = make_uint4(0u, 0u, 0u, 0u);
-    }
-  }
-  if (seen_begin >= seen_end) return;
-
   const uint32_t base = (smem_u32(dynamic) + 1023u) & ~1023u;
   const uint32_t q_half = (uint32_t)(Q * heads) * 128u;          // bytes of a 64-element half of all the queries' rows
   const uint32_t k_at = base, q_at = base + 2 * kOperand;
@@ -339,158 +379,172 @@ mixed_weights_tc_kernel(const bf16* __restrict__ q, long long q_stride, const bf
   if (threadIdx.x == 0)
     for (int i = 0; i < WEIGHTS_BARRIERS; ++i) barrier_init(bar + i * 8, i < KEYS_FREE ? kLoaders : 1);
   const uint32_t tmem = allocate(&tmem_place, COLUMNS, nullptr, 0);
-  const int steps = (seen_end - seen_begin) * kv_heads;
   bool alive = true;
+  int step = 0;                                                  // key tiles (of one kv head) so far, over all items
+  MixItem m;
+  start_mix_items(query_starts, rows, m);
 
   if (threadIdx.x >= kMixers) {
     asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kLoaderRegisters));
-    const int* table = block_table + (size_t)w.row * table_width;
-    int mine = -1;
-    for (int step = 0; step < steps; ++step) {
-      const int stage = step & 1, kv_head = step % kv_heads;
-      if (kv_head == 0)
-        mine = cache_row<kTile, 4>(table, page_size, w.key_begin + (seen_begin + step / kv_heads) * kTile, w.key_end, warp - 8, lane);
-      if (step >= 2) wait_alive(bar + (KEYS_FREE + stage) * 8, ((step >> 1) - 1) & 1, alive, 2);
-      __syncwarp();
-      load_rows<kTile, 4>(k_at + stage * kOperand, k_pages, kv_heads, kv_head, mine, warp - 8, lane);
-      copy_commit();
-      if (step > 0) {                                            // the stage before: it has landed, and the tensor cores may see it
-        copy_wait<1>();
-        fence_for_tensor_cores();
-        barrier_arrive(bar + (KEYS_FULL + (stage ^ 1)) * 8);
+    const int loader = warp - kMixers / 32;
+    for (int rank = blockIdx.x; mix_item<Q>(rank, first_tile, slab_tiles, query_starts, context_lens, window, chunk,
+                                            segment_tiles, key_columns, m); rank += gridDim.x) {
+      const int* table = block_table + (size_t)m.w.row * table_width;
+      for (int kt = m.seen_begin; kt < m.seen_end; ++kt) {
+        const int mine = cache_row<kTile, kLoaders / 32>(table, page_size, m.w.key_begin + kt * kTile, m.w.key_end, loader, lane);
+        for (int kv_head = 0; kv_head < kv_heads; ++kv_head, ++step) {
+          const int stage = step & 1;
+          if (step >= 2) wait_alive(bar + (KEYS_FREE + stage) * 8, ((step >> 1) - 1) & 1, alive, 2);
+          __syncwarp();
+          load_rows<kTile, kLoaders / 32>(k_at + stage * kOperand, k_pages, kv_heads, kv_head, mine, loader, lane);
+          copy_commit();
+          if (step > 0) {                                        // the stage before: it has landed, and the tensor cores may see it
+            copy_wait<1>();
+            fence_for_tensor_cores();
+            barrier_arrive(bar + (KEYS_FULL + (stage ^ 1)) * 8);
+          }
+        }
       }
     }
-    copy_wait<0>();
-    fence_for_tensor_cores();
-    barrier_arrive(bar + (KEYS_FULL + ((steps - 1) & 1)) * 8);
+    if (step > 0) {
+      copy_wait<0>();
+      fence_for_tensor_cores();
+      barrier_arrive(bar + (KEYS_FULL + ((step - 1) & 1)) * 8);
+    }
   } else {
     asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(kMixerRegisters));
-    // row head * Q + query of the second operand
-    for (int i = threadIdx.x; i < heads * Q * 16; i += kMixers) {
-      const int row = i / 16, piece = i % 16, query = row % Q;
-      const bool there = query < here;
-      copy16(q_at + (piece >> 3) * q_half + row * 128 + (((piece & 7) ^ (row & 7)) << 4),
-             there ? q + (size_t)(token0 + query) * q_stride + (size_t)(row / Q) * kDim + piece * 8 : q, there);
-    }
-    copy_commit();
-    for (int i = threadIdx.x; i < HEADS * HEADS; i += kMixers) {
-      const int g = i / HEADS, h = i % HEADS;
-      mix_s[i] = g < heads && h < heads ? mix[h * heads + g] : 0.0f;
-    }
-    for (int i = threadIdx.x; i < HEADS * Q; i += kMixers) {
-      const int g = i / Q, query = i % Q;
-      sums_s[i] = g < heads && query < here ? log_sums[(size_t)g * tokens + token0 + query] : 0.0f;
-    }
-    copy_wait<0>();
-    fence_for_tensor_cores();
-    const int quarter = (warp & 3) * 32, half = warp >> 2;
+    const int quarter = (warp & 3) * 32, set = warp >> 2;
     const uint32_t lane_at = tmem + ((uint32_t)quarter << 16);
-    int step = 0;
-    for (int kt = seen_begin; kt < seen_end; ++kt) {
-      tensor_fence_before_sync();                                // (the last tile's scores have been read)
-      asm volatile("bar.sync 1, %0;" ::"n"(kMixers) : "memory");
-      if (warp == 0) {
-        tensor_fence_after_sync();
-        const uint32_t elected = elect_one();
-        for (int group = 0; group < kv_heads; ++group, ++step) {
-          const int stage = step & 1;
-          wait_alive(bar + (KEYS_FULL + stage) * 8, (step >> 1) & 1, alive, 2);
-          __syncwarp();
-          tensor_fence_after_sync();
-          const uint32_t a = operand_low(k_at + stage * kOperand);
-          for (int n0 = 0; n0 < per_group * Q; n0 += 256) {
-            const uint32_t idesc = instruction_descriptor(kTile, min(256, per_group * Q - n0));
-            const uint32_t b = operand_low(q_at + (uint32_t)(group * per_group * Q + n0) * 128u);
-#pragma unroll
-            for (int k = 0; k < 8; ++k)
-              mma_bf16_ss_halves(tmem + group * per_group * Q + n0, a + (k >> 2) * (kHalf >> 4) + (k & 3) * 2,
-                                 b + (k >> 2) * (q_half >> 4) + (k & 3) * 2, idesc, (uint32_t)(k > 0), elected);
-          }
-          mma_commit_elected(bar + (KEYS_FREE + stage) * 8, elected);
+    const size_t head_stride = (size_t)kTile * key_columns;
+    int tile_count = 0;                                          // tiles of keys so far, over all items
+    for (int rank = blockIdx.x; mix_item<Q>(rank, first_tile, slab_tiles, query_starts, context_lens, window, chunk,
+                                            segment_tiles, key_columns, m); rank += gridDim.x) {
+      bf16* const result = mixed + ((size_t)(m.index - first_tile) * heads * kTile + m.sub * Q) * key_columns;
+      for (int kt = m.segment_begin; kt < m.segment_end; ++kt) {
+        if (kt >= m.seen_begin && kt < m.seen_end) continue;
+        for (int i = threadIdx.x; i < heads * m.here * 16; i += kMixers) {
+          const int row = i / 16, h = row / m.here, query = row - h * m.here;
+          *reinterpret_cast<uint4*>(result + h * head_stride + (size_t)query * key_columns + kt * kTile + i % 16 * 8) = make_uint4(0u, 0u, 0u, 0u);
         }
-        mma_commit_elected(bar + SCORES_FULL * 8, elected);
       }
-      wait_alive(bar + SCORES_FULL * 8, (kt - seen_begin) & 1, alive, 2);
-      __syncwarp();
-      tensor_fence_after_sync();
-      const int key = w.key_begin + kt * kTile + quarter + lane;
-#pragma unroll 1
-      for (int q0 = half * (Q / 2); q0 < (half + 1) * (Q / 2); q0 += QB) {
-        bool seen[QB];
+      if (m.seen_begin >= m.seen_end) continue;
+      asm volatile("bar.sync 1, %0;" ::"n"(kMixers) : "memory");    // (the last item's sums and queries are used no more)
+      // row head * Q + query of the second operand
+      for (int i = threadIdx.x; i < heads * Q * 16; i += kMixers) {
+        const int row = i / 16, piece = i % 16, query = row % Q;
+        const bool there = query < m.here;
+        copy16(q_at + (piece >> 3) * q_half + row * 128 + (((piece & 7) ^ (row & 7)) << 4),
+               there ? q + (size_t)(m.token0 + query) * q_stride + (size_t)(row / Q) * kDim + piece * 8 : q, there);
+      }
+      copy_commit();
+      for (int i = threadIdx.x; i < HEADS * Q; i += kMixers) {
+        const int g = i / Q, query = i % Q;
+        sums_s[i] = g < heads && query < m.here ? log_sums[(size_t)g * tokens + m.token0 + query] : 0.0f;
+      }
+      copy_wait<0>();
+      fence_for_tensor_cores();
+      for (int kt = m.seen_begin; kt < m.seen_end; ++kt, ++tile_count) {
+        tensor_fence_before_sync();                              // (the last tile's scores have been read)
+        asm volatile("bar.sync 1, %0;" ::"n"(kMixers) : "memory");
+        if (warp == 0) {
+          tensor_fence_after_sync();
+          const uint32_t elected = elect_one();
+          for (int group = 0; group < kv_heads; ++group, ++step) {
+            const int stage = step & 1;
+            wait_alive(bar + (KEYS_FULL + stage) * 8, (step >> 1) & 1, alive, 2);
+            __syncwarp();
+            tensor_fence_after_sync();
+            const uint32_t a = operand_low(k_at + stage * kOperand);
+            for (int n0 = 0; n0 < per_group * Q; n0 += 256) {
+              const uint32_t idesc = instruction_descriptor(kTile, min(256, per_group * Q - n0));
+              const uint32_t b = operand_low(q_at + (uint32_t)(group * per_group * Q + n0) * 128u);
 #pragma unroll
-        for (int i = 0; i < QB; ++i) {
-          const int position = position0 + q0 + i;
-          seen[i] = q0 + i < here && key <= position && key >= first_visible(position, window, chunk);
-        }
-        pair32 acc[QB][HEADS / 2];
-#pragma unroll
-        for (int i = 0; i < QB; ++i)
-#pragma unroll
-          for (int h = 0; h < HEADS / 2; ++h) acc[i][h] = 0ull;
-        auto request = [&](int g, uint32_t (&scores)[GB][QB]) {  // (columns behind the last head: read, and not used)
-#pragma unroll
-          for (int e = 0; e < GB; ++e) tmem_request<QB>(lane_at + (g + e) * Q + q0, scores[e]);
-        };
-        auto add_heads = [&](int g, uint32_t (&scores)[GB][QB]) {
-#pragma unroll
-          for (int e = 0; e < GB; ++e)
-#pragma unroll
-            for (int i = 0; i < QB; ++i) {
-              const float v = fast_exp2(fmaf(__uint_as_float(scores[e][i]), scale2, -sums_s[(g + e) * Q + q0 + i]));
-              scores[e][i] = seen[i] && g + e < heads ? __float_as_uint(v) : 0u;
+              for (int k = 0; k < 8; ++k)
+                mma_bf16_ss_halves(tmem + group * per_group * Q + n0, a + (k >> 2) * (kHalf >> 4) + (k & 3) * 2,
+                                   b + (k >> 2) * (q_half >> 4) + (k & 3) * 2, idesc, (uint32_t)(k > 0), elected);
             }
+            mma_commit_elected(bar + (KEYS_FREE + stage) * 8, elected);
+          }
+          mma_commit_elected(bar + SCORES_FULL * 8, elected);
+        }
+        wait_alive(bar + SCORES_FULL * 8, tile_count & 1, alive, 2);
+        __syncwarp();
+        tensor_fence_after_sync();
+        const int key = m.w.key_begin + kt * kTile + quarter + lane;
+#pragma unroll 1
+        for (int q0 = set * SET; q0 < (set + 1) * SET; q0 += QB) {
+          bool seen[QB];
 #pragma unroll
-          for (int e = 0; e < GB; ++e) {
-            const ulonglong2* factors = reinterpret_cast<const ulonglong2*>(mix_s + (g + e) * HEADS);
-            pair32 weight[QB];
+          for (int i = 0; i < QB; ++i) {
+            const int position = m.position0 + q0 + i;
+            seen[i] = q0 + i < m.here && key <= position && key >= first_visible(position, window, chunk);
+          }
+          pair32 acc[QB][HEADS / 2];
 #pragma unroll
-            for (int i = 0; i < QB; ++i) weight[i] = make_pair(__uint_as_float(scores[e][i]), __uint_as_float(scores[e][i]));
+          for (int i = 0; i < QB; ++i)
 #pragma unroll
-            for (int h = 0; h < HEADS / 4; ++h) {
-              const ulonglong2 m = factors[h];
+            for (int h = 0; h < HEADS / 2; ++h) acc[i][h] = 0ull;
+          auto request = [&](int g, uint32_t (&scores)[GB][QB]) {  // (columns behind the last head: read, and not used)
+#pragma unroll
+            for (int e = 0; e < GB; ++e) tmem_request<QB>(lane_at + (g + e) * Q + q0, scores[e]);
+          };
+          auto add_heads = [&](int g, uint32_t (&scores)[GB][QB]) {
+#pragma unroll
+            for (int e = 0; e < GB; ++e)
 #pragma unroll
               for (int i = 0; i < QB; ++i) {
-                acc[i][2 * h] = fma_pair(m.x, weight[i], acc[i][2 * h]);
-                acc[i][2 * h + 1] = fma_pair(m.y, weight[i], acc[i][2 * h + 1]);
+                const float v = fast_exp2(fmaf(__uint_as_float(scores[e][i]), scale2, -sums_s[(g + e) * Q + q0 + i]));
+                scores[e][i] = seen[i] && g + e < heads ? __float_as_uint(v) : 0u;
+              }
+#pragma unroll
+            for (int e = 0; e < GB; ++e) {
+              pair32 weight[QB];
+#pragma unroll
+              for (int i = 0; i < QB; ++i) weight[i] = make_pair(__uint_as_float(scores[e][i]), __uint_as_float(scores[e][i]));
+#pragma unroll
+              for (int h = 0; h < HEADS / 2; ++h) {
+                const pair32 both = make_pair(mix.of[(g + e) * HEADS + 2 * h], mix.of[(g + e) * HEADS + 2 * h + 1]);
+#pragma unroll
+                for (int i = 0; i < QB; ++i) acc[i][h] = fma_pair(both, weight[i], acc[i][h]);
               }
             }
-          }
-        };
-        auto arrived = [&](uint32_t (&scores)[GB][QB]) {
+          };
+          auto arrived = [&](uint32_t (&scores)[GB][QB]) {
 #pragma unroll
-          for (int e = 0; e < GB; ++e) tmem_request_wait(scores[e]);
-        };
-        // some heads' scores are on their way while the heads before are added
-        uint32_t front[GB][QB], back[GB][QB];
-        request(0, front);
-        arrived(front);
+            for (int e = 0; e < GB; ++e) tmem_request_wait(scores[e]);
+          };
+          // some heads' scores are on their way while the heads before are added
+          uint32_t front[GB][QB], back[GB][QB];
+          request(0, front);
+          arrived(front);
 #pragma unroll 1
-        for (int g = 0; g < heads; g += 2 * GB) {
-          request(g + GB, back);
-          add_heads(g, front);
-          arrived(back);
-          if (g + 2 * GB < heads) request(g + 2 * GB, front);
-          add_heads(g + GB, back);
-          if (g + 2 * GB < heads) arrived(front);
-        }
-        // neighbouring lanes hold neighbouring keys: the even one stores both keys of a query, the odd one of the next query
-        const bool even = (lane & 1) == 0;
+          for (int g = 0; g < heads; g += 2 * GB) {
+            request(g + GB, back);
+            add_heads(g, front);
+            arrived(back);
+            if (g + 2 * GB < heads) request(g + 2 * GB, front);
+            add_heads(g + GB, back);
+            if (g + 2 * GB < heads) arrived(front);
+          }
+          // neighbouring lanes hold neighbouring keys: the even one stores both keys of a query, the odd one of the next query
+          const bool even = (lane & 1) == 0;
 #pragma unroll
-        for (int i = 0; i < QB; i += 2) {
-          const int query = q0 + i + (even ? 0 : 1);
-          bf16* to = result + (size_t)query * key_columns + kt * kTile + quarter + (lane & ~1);
-          const bool there = query < here;
+          for (int i = 0; i < QB; i += 2) {
+            const int query = q0 + i + (even ? 0 : 1);
+            bf16* to = result + (size_t)query * key_columns + kt * kTile + quarter + (lane & ~1);
+            const bool there = query < m.here;
 #pragma unroll
-          for (int h = 0; h < HEADS / 2; ++h) {
-            float a0, a1, b0, b1;
-            split_pair(acc[i][h], a0, a1);
-            split_pair(acc[i + 1][h], b0, b1);
-            const float other0 = __shfl_xor_sync(0xffffffffu, even ? b0 : a0, 1);
-            const float other1 = __shfl_xor_sync(0xffffffffu, even ? b1 : a1, 1);
-            if (there && 2 * h < heads)
-              *reinterpret_cast<uint32_t*>(to + (2 * h) * head_stride) = even ? pack_bf16(a0, other0) : pack_bf16(other0, b0);
-            if (there && 2 * h + 1 < heads)
-              *reinterpret_cast<uint32_t*>(to + (2 * h + 1) * head_stride) = even ? pack_bf16(a1, other1) : pack_bf16(other1, b1);
+            for (int h = 0; h < HEADS / 2; ++h) {
+              float a0, a1, b0, b1;
+              split_pair(acc[i][h], a0, a1);
+              split_pair(acc[i + 1][h], b0, b1);
+              const float other0 = __shfl_xor_sync(0xffffffffu, even ? b0 : a0, 1);
+              const float other1 = __shfl_xor_sync(0xffffffffu, even ? b1 : a1, 1);
+              if (there && 2 * h < heads)
+                *reinterpret_cast<uint32_t*>(to + (2 * h) * head_stride) = even ? pack_bf16(a0, other0) : pack_bf16(other0, b0);
+              if (there && 2 * h + 1 < heads)
+                *reinterpret_cast<uint32_t*>(to + (2 * h + 1) * head_stride) = even ? pack_bf16(a1, other1) : pack_bf16(other1, b1);
+            }
           }
         }
       }
@@ -603,7 +657,8 @@ MIR_EXPORT int mir_mixed_prefill_tc_takes(int heads, int dim, int value_dim) {
 // Portions: row r brings the tokens query_starts[r] .. query_starts[r + 1] of qkv and out and has context_lens[r] keys after
 // the step.  tiles: at least the number of tiles of 128 tokens over all rows; the mixed weights of slab_tiles of them at a
 // time pass through `mixed` (slab_tiles * heads * 128 * key_columns * 2 bytes), key_columns a multiple of 128: enough for the
-// keys from the multiple of 128 below the first one a tile sees to its last query.  scale is above zero.
+// keys from the multiple of 128 below the first one a tile sees to its last query.  scale is above zero.  mix is in host
+// memory.
 MIR_EXPORT int mir_mixed_prefill_attention_tc_bf16(const void* q, long long q_stride, void* out, const void* k_pages,
                                                    const void* v_pages, const int* block_table, int table_width,
                                                    const int* query_starts, const int* context_lens, int rows, int tokens,
@@ -636,11 +691,15 @@ MIR_EXPORT int mir_mixed_prefill_attention_tc_bf16(const void* q, long long q_st
     const int here = std::min(slab_tiles, tiles - from);
 #define MIR_WEIGHTS(H)                                                                                                   \
   do {                                                                                                                   \
+    MixMatrix matrix = {};                                                                                              \
+    for (int g = 0; g < heads; ++g)                                                                                     \
+      for (int h = 0; h < heads; ++h) matrix.of[g * H + h] = mix[h * heads + g];                                        \
     const size_t smem = 2 * kOperand + (size_t)queries_for(H) * heads * 256 + 1024;                                      \
     if ((status = reserve((const void*)mixed_weights_tc_kernel<H>, smem, "mixed_weights_tc")) != MIR_OK) return status;  \
-    mixed_weights_tc_kernel<H><<<dim3(segments, here * (kTile / queries_for(H))), kMixers + kLoaders, smem, stream>>>(                  \
+    mixed_weights_tc_kernel<H><<<dim3(std::min(mir_sm_count(), here * segments * (kTile / queries_for(H)))), kMixers + kLoaders, smem, stream>>>( \
         qb, q_stride, kb, block_table, table_width, query_starts, context_lens, rows, page_size, heads, kv_heads, scale2, \
-        window, chunk, mix, log_sums, tokens, from, segment_tiles, key_columns, (bf16*)mixed);                           \
+        window, chunk, matrix, log_sums, tokens, from, here, segment_tiles,                  \
+        key_columns, (bf16*)mixed);                           \
   } while (0)
     if (heads <= 8) MIR_WEIGHTS(8);
     else if (heads <= 16) MIR_WEIGHTS(16);

@@ -1470,12 +1470,14 @@ def mixed_prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
                             block_table: torch.Tensor, query_starts: torch.Tensor, context_lens: torch.Tensor,
                             page_size: int, heads: int, kv_heads: int, dim: int, value_dim: int, scale: float,
                             head_mix: torch.Tensor, window: Optional[int], chunk: Optional[int], portion_tokens: int,
-                            longest: int, alloc, tensor_cores: Optional[bool] = None) -> None:
+                            longest: int, alloc, tensor_cores: Optional[bool] = None,
+                            host_mix: Optional[torch.Tensor] = None) -> None:
     """paged_attention_mixed for any mix of portions (row r owns the tokens query_starts[r] .. query_starts[r + 1] of qkv
     and out; the rows may be a part of the batch, with portion_tokens tokens together and at most `longest` tokens each),
     bfloat16, on tensor cores: the rows' log-sums, the mixed weights, the products with the values.  `tensor_cores`: True
     runs the tcgen05 kernels (heads of 128 channels), False the mma.sync kernels, None chooses: tcgen05 where they take
-    the sizes and the portions average PREFILL_TENSOR_CORE_MIN_PORTION tokens."""
+    the sizes and the portions average PREFILL_TENSOR_CORE_MIN_PORTION tokens.  `host_mix`: the mixing matrix in host
+    memory, which the tcgen05 kernels take as a launch parameter (copied from the device if it is not given)."""
     _check_mixed("mixed_prefill_attention", qkv, out, k_pages, v_pages, block_table, head_mix, heads, kv_heads, dim, value_dim)
     rows, tokens = context_lens.numel(), out.shape[0]
     _require(out.dtype == torch.bfloat16 and query_starts.dtype == torch.int32 and context_lens.dtype == torch.int32
@@ -1487,6 +1489,10 @@ def mixed_prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
                         and bool(lib.mir_mixed_prefill_tc_takes(heads, dim, value_dim)))
     log_sums = alloc((heads, tokens), torch.float32)
     if tensor_cores:
+        if host_mix is None:
+            host_mix = head_mix.cpu()
+        _require(host_mix.dtype == torch.float32 and not host_mix.is_cuda and host_mix.is_contiguous()
+                 and host_mix.shape == (heads, heads), "mixed_prefill_attention: host_mix is float32 [heads, heads] on the host")
         tiles = portion_tokens // 128 + rows
         # keys of a tile of 128 queries, from the multiple of 128 at or below the first one that is seen
         key_columns = 128 * min(-(-(min(longest, span + 127) + 127) // 128), -(-longest // 128))
@@ -1496,7 +1502,7 @@ def mixed_prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
         _check(lib, lib.mir_mixed_prefill_attention_tc_bf16(
             qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
             block_table.shape[1], query_starts.data_ptr(), context_lens.data_ptr(), rows, tokens, page_size, heads, kv_heads,
-            dim, value_dim, scale, head_mix.data_ptr(), int(window or 0), int(chunk or 0), tiles, slab_tiles, key_columns,
+            dim, value_dim, scale, host_mix.data_ptr(), int(window or 0), int(chunk or 0), tiles, slab_tiles, key_columns,
             MIXED_TC_SEGMENT_TILES, log_sums.data_ptr(), mixed.data_ptr(), _stream()))
         return
     tiles = portion_tokens // 64 + rows              # (a row's last tile may be short)

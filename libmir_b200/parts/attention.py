@@ -64,7 +64,7 @@ class SoftmaxAttention(Mixer):
         if self.other_norm and not s.own_kv:
             raise ValueError("these q/k norms need keys of the mixer's own")
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = self.q_norm = self.k_norm = self.sinks = None
-        self.distance_bias = self.head_mix = None
+        self.distance_bias = self.head_mix = self.host_mix = None
         if s.head_mix and (s.keep_first or s.sinks or s.fixed_sink is not None or s.gate or s.softcap is not None
                            or s.distance_bias is not None):
             raise ValueError("mixed heads go with plain scores: no sinks, gate, cap, bias or kept first tokens")
@@ -154,6 +154,7 @@ class SoftmaxAttention(Mixer):
                                     device=self.w_o.device)
         if self.spec.head_mix:
             self.head_mix = tensors["head_mix"].contiguous()
+            self.host_mix = self.head_mix.cpu()
         if self.spec.distance_bias is not None:
             self.distance_bias = self.bias_by_distance(tensors["rel_bias"].float())
 
@@ -354,7 +355,8 @@ class SoftmaxAttention(Mixer):
             kernels.mixed_prefill_attention(qkv, out, cache.k_pages, cache.v_pages, group.block_table[singles:],
                                             ctx.query_starts[singles:], ctx.context_lens[singles:], cache.page_size,
                                             s.heads, s.kv_heads, s.head_dim, s.value_dim, s.scale, self.head_mix, s.window,
-                                            s.chunk, out.shape[0] - singles, ctx.max_context, ctx.alloc)
+                                            s.chunk, out.shape[0] - singles, ctx.max_context, ctx.alloc,
+                                            host_mix=self.host_mix)
             return
         if done == out.shape[0]:
             return
