@@ -1463,7 +1463,10 @@ def mixed_decode_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.
 
 MIXED_SLAB_BYTES = 256 << 20     # how much of the mixed weights of a prompt is in memory at a time
 MIXED_SEGMENT_TILES = 4          # tiles of 64 keys that a CTA of the mma.sync mixing kernel goes through
-MIXED_TC_SEGMENT_TILES = 3       # tiles of 128 keys that a CTA of the tcgen05 mixing kernel goes through
+# tiles of 128 keys that a CTA of the tcgen05 mixing kernel goes through with the same queries: few where an item is long
+# (more than 16 heads: 217 us for a 2,048-token prompt with one tile, 233 with three), more where its start weighs (120 us
+# with three tiles at 16 heads, 134 with one)
+MIXED_TC_SEGMENT_TILES = {True: 1, False: 3}
 
 
 def mixed_prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
@@ -1503,7 +1506,7 @@ def mixed_prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
             qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
             block_table.shape[1], query_starts.data_ptr(), context_lens.data_ptr(), rows, tokens, page_size, heads, kv_heads,
             dim, value_dim, scale, host_mix.data_ptr(), int(window or 0), int(chunk or 0), tiles, slab_tiles, key_columns,
-            MIXED_TC_SEGMENT_TILES, log_sums.data_ptr(), mixed.data_ptr(), _stream()))
+            MIXED_TC_SEGMENT_TILES[heads > 16], log_sums.data_ptr(), mixed.data_ptr(), _stream()))
         return
     tiles = portion_tokens // 64 + rows              # (a row's last tile may be short)
     # keys of a tile of 16 queries: what the first and the last of them see, from the multiple of 64 below on

@@ -559,7 +559,9 @@ def test_the_designs_kernels_run_in_bfloat16(tmp_path):
         order = [config["layers"][index] for index, _ in plain.layer_order(config)]
         runs = {kind: sum(layer["type"] == kind for layer in order) for kind in ("mamba1", "latent_attention", "attention")}
         steps = 3
-        assert counts["mixed_weights"] == counts["mixed_values"] == counts["mixed_row_sums"] == runs["attention"], counts
+        form = "_tc" if name == "D" else ""                     # heads of 128 channels: tcgen05, of 64: mma.sync
+        assert counts["mixed_weights" + form] == counts["mixed_values" + form] == counts["mixed_row_sums" + form] \
+            == runs["attention"], counts
         assert counts["mixed_decode_scores"] == counts["mixed_decode_values"] == 2 * runs["attention"], counts
         assert counts["selective_scan"] == steps * runs["mamba1"] and counts["latent_prepare"] == steps * runs["latent_attention"]
         assert counts["latent_attention"] == steps * runs["latent_attention"], counts
