@@ -52,7 +52,7 @@ PEDOTAR_B = {   # sizes that are 1 or equal, widths that are no multiples of 8, 
 }
 
 PEDOTAR_C = {   # heads of 64 channels (tensor cores in bfloat16), as many key heads as query heads; the loop at the end
-    "architecture": "Pedotar", "vocab": 151, "width": 104, "norm": {"eps": 1e-5}, "loop": {"start": 1, "stop": 3, "times": 3},
+    "architecture": "Pedotar", "vocab": 151, "width": 104, "norm": {"eps": 1e-5}, "loop": {"start": 1, "stop": 3, "times": 2},
     "layers": [
         _layer(scan(160, 12, 6, 4)),
         _layer(mixed(5, 5, 64, 64, 0.12, 50), 88),

@@ -58,7 +58,7 @@ def test_a_repeated_run_of_layers_adds_the_embedding_before_every_pass_but_the_f
     model = DecoderModel(spec, META)
     assert [model.pass_adds(entry) for entry in spec.schedule] == [False] * 4 + [True] + [False] * 3
     assert [entry.layer for entry in build_spec(PEDOTAR_B, None).schedule] == [0, 1, 2, 3, 4]
-    assert [entry.layer for entry in build_spec(PEDOTAR_C, None).schedule] == [0, 1, 2, 1, 2, 1, 2]
+    assert [entry.layer for entry in build_spec(PEDOTAR_C, None).schedule] == [0, 1, 2, 1, 2]
     assert [entry.layer for entry in build_spec(PEDOTAR_E, None).schedule] == [0, 1, 1, 1, 1]
     assert build_spec(PEDOTAR_B, None).loop is None
     empty = dict(PEDOTAR_A, loop={"start": 2, "stop": 2, "times": 3})

@@ -97,7 +97,7 @@ PORTIONS = ([1, 2], [2, 1], [1, 1], [3, 1], [1, 5], [40, 2], [7, 66], [1, 1], [2
 
 
 @pytest.mark.parametrize("dtype,tol", DTYPES)
-@pytest.mark.parametrize("taps,channels", [(1, 64), (2, 64), (3, 72), (4, 320), (5, 64), (4, 30), (2, 12)])
+@pytest.mark.parametrize("taps,channels", [(1, 64), (2, 64), (3, 72), (4, 272), (5, 64), (4, 30), (2, 12)])
 def test_short_convolution_with_a_bias_in_the_activations_type(dtype, tol, taps, channels):
     """Two requests in portions of 1, 2, 3 and more tokens, in state slots 2 and 0: 16-byte pieces up to four taps, the
     general kernel for other sizes; the same bits in 32-bit results of the two."""
@@ -137,7 +137,7 @@ def test_short_convolution_with_a_bias_in_the_activations_type(dtype, tol, taps,
 
 
 @pytest.mark.parametrize("dtype,tol", DTYPES)
-@pytest.mark.parametrize("channels,n", [(64, 16), (40, 1), (320, 24), (8, 7), (72, 4), (64, 33), (32, 64), (16, 100), (8, 256)])
+@pytest.mark.parametrize("channels,n", [(64, 16), (40, 1), (200, 24), (8, 7), (72, 4), (64, 33), (32, 64), (16, 100), (8, 256)])
 def test_selective_scan_carries_its_state_between_portions(dtype, tol, channels, n):
     """Two requests in portions, in state slots 2 and 0; step sizes from almost nothing to large ones (a state that
     stays, a state that is forgotten at once); the state after it in 32-bit, other slots untouched, and in 32-bit the
@@ -189,7 +189,7 @@ def test_selective_scan_carries_its_state_between_portions(dtype, tol, channels,
 
 # ------------------------------------------------------------------------------ latent attention
 @pytest.mark.parametrize("dtype,tol", DTYPES)
-@pytest.mark.parametrize("heads,dim,rot,rank", [(3, 16, 8, 48), (1, 5, 2, 10), (6, 32, 64, 128)])
+@pytest.mark.parametrize("heads,dim,rot,rank", [(3, 16, 8, 48), (1, 5, 2, 10), (5, 40, 64, 160)])
 def test_the_latent_is_normed_and_queries_and_shared_key_rotated_in_one_launch(dtype, tol, heads, dim, rot, rank):
     from libmir_b200 import kernels
     generator = torch.Generator().manual_seed(rank)
@@ -244,10 +244,10 @@ MIXED_CASES = [
     (torch.float32, 4, 2, 24, 40, 8, None, 37, "reference"),
     (torch.float32, 3, 1, 10, 6, 4, None, 50, "reference"),
     (torch.float32, 5, 5, 64, 16, 16, 29, None, "reference"),
-    (BF16, 6, 3, 32, 16, 16, None, 96, "split"),
+    (BF16, 6, 3, 32, 16, 16, None, 110, "split"),
     (BF16, 7, 7, 8, 200, 8, None, 130, "split"),
     (BF16, 9, 1, 256, 64, 16, None, None, "split"),
-    (BF16, 6, 6, 64, 64, 16, None, 96, "tiles"),
+    (BF16, 7, 7, 64, 64, 16, None, 90, "tiles"),
     (BF16, 1, 1, 64, 128, 4, None, 64, "tiles"),
     (BF16, 12, 3, 128, 128, 16, None, 50, "tiles"),
     (BF16, 32, 8, 128, 64, 32, None, 101, "tiles"),
