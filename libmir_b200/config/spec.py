@@ -187,6 +187,14 @@ class DistanceBiasSpec:
 
 
 @dataclass(frozen=True)
+class QueryTemperature:
+    """A factor on the queries (behind their norm) that grows with the position p: 1 + coef ln(floor((p + 1) / every) + 1)."""
+
+    coef: float
+    every: float
+
+
+@dataclass(frozen=True)
 class YarnScaling:
     """Frequencies stretched by `factor` where a pair turns fewer than `slow` times over `original` positions, kept
     where it turns more than `fast` times, blended linearly (by pair index) in between; cos and sin are multiplied by
@@ -255,6 +263,12 @@ class SoftmaxAttentionSpec(PartSpec):
     # sum_g head_mix[h, g] weights_g of all heads' softmax weights to the values of its own kv head.
     chunk: Optional[int] = None
     head_mix: bool = False
+    # values_from_keys: there is no value tensor, a token's value is its key as projected, before norm and rotation.
+    # slopes: one number per query head (or none): slopes[h] * (query position - key position) is taken off the score.
+    # temperature: what the queries are multiplied by.
+    values_from_keys: bool = False
+    slopes: tuple = ()
+    temperature: Optional[QueryTemperature] = None
     kind: str = field(init=False, default="softmax_attention")
 
     @property
@@ -348,9 +362,11 @@ class RoutedExpertsSpec(PartSpec):
 @dataclass(frozen=True)
 class RetentionSpec(PartSpec):
     """Linear attention with one fixed decay per head and no softmax (parts/retention.py): per head a matrix state
-    S <- decay_h S + k v^T, read out as S^T q, with k scaled by key_dim^-1/2 after the rotation; the read-out of each
-    head is divided by its root mean square and multiplied by silu of a projection of the mixer's input.  `decays`
-    holds one number per head."""
+    S <- decay_h S + k v^T, read out as S^T q, with k scaled by `key_scale` (None: key_dim^-1/2) after the rotation; the
+    read-out of each head is divided by its root mean square and multiplied by silu of a projection of the mixer's
+    input.  `decays` holds one number per head.  Other forms: `activated`, silu of q, k and v enters the recurrence;
+    `norm_span` "all", one root mean square over all heads' read-outs together; `norm_weight`, a stored weight (tensor
+    `norm`, one number per column of the heads) behind the norm; `gate` "sigmoid"."""
 
     hidden_size: int = 0
     heads: int = 0
@@ -359,6 +375,11 @@ class RetentionSpec(PartSpec):
     decays: tuple = ()
     norm_eps: float = 1e-5
     position: Optional[PartSpec] = None
+    key_scale: Optional[float] = None
+    activated: bool = False
+    norm_span: str = "head"
+    norm_weight: bool = False
+    gate: str = "silu"
     kind: str = field(init=False, default="retention")
 
 
@@ -399,13 +420,15 @@ class SelectiveScanSpec(PartSpec):
 @dataclass(frozen=True)
 class SideBySideSpec(PartSpec):
     """Several mixers that read the same input; the result is `scale` times the sum of their outputs, each first
-    RMS-normed over the model width with a plain weight `<branch name>.<out_tensor>`."""
+    RMS-normed over the model width with a plain weight `<branch name>.<out_tensor>`.  With `scales` (one number per
+    branch) there are no such norms and weights: the result is the sum of scales[b] times the output of branch b."""
 
     hidden_size: int = 0
     branches: tuple = ()                     # (name, PartSpec) pairs; a branch's tensors lie under "<name>."
     eps: float = 1e-5
     scale: float = 0.5
     out_tensor: str = "out"
+    scales: tuple = ()
     kind: str = field(init=False, default="side_by_side")
 
 
@@ -432,7 +455,8 @@ class LayerSpec:
     `feed_forward_norm` is None, else each through a norm of its own), "output_norm" (each branch reads the
     residual itself and its RESULT goes through the norm: x += residual_scale * norm(branch(x)), one after the other),
     "sandwich" (a norm before and a norm behind each branch: x += mixer_out_norm(mixer(mixer_norm(x))), then the same
-    with the feed-forward's two norms) and "streams" (the residual is ModelSpec.streams copies; each branch reads a mix of them through its norm and
+    with the feed-forward's two norms), "post_norm" (each branch reads the residual itself, and the norm stands behind
+    the sum: x = mixer_norm(residual_alpha * x + mixer(x)), then the same with the feed-forward) and "streams" (the residual is ModelSpec.streams copies; each branch reads a mix of them through its norm and
     writes into all of them as `mixer_streams` / `feed_forward_streams`, StreamMixSpec, say).
     """
 
@@ -443,6 +467,7 @@ class LayerSpec:
     feed_forward_norm: Optional[PartSpec]
     names: Mapping[str, str]
     arrangement: str = "pre_norm"
+    residual_alpha: float = 1.0           # what the residual is multiplied by ahead of the sum ("post_norm" only)
     residual_scale: float = 1.0           # what a branch's (normed) result is multiplied by ("output_norm" only)
     mixer_streams: Optional[PartSpec] = None          # ("streams" only) how the mixer reads and writes the streams
     feed_forward_streams: Optional[PartSpec] = None   # the same for the feed-forward

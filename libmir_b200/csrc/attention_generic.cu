@@ -23,6 +23,7 @@
 // softcap > 0: score <- softcap * tanh(score / softcap) after the scale.  rel_bias ([heads, rel_rows] 32-bit, or none):
 // the entry min(position - key, rel_rows - 1) of head h is added to the score after the cap (a bias by distance whose
 // buckets the host has spread out into one row per distance; from the last row on it no longer changes).
+// slopes ([heads] 32-bit, or none): slopes[h] * (position - key) is taken off the score after the cap.
 #include <cfloat>
 #include "common.cuh"
 
@@ -38,7 +39,7 @@ __global__ void paged_attention_generic_kernel(
     const int* __restrict__ row_of_token, const int* __restrict__ positions, int page_size, int heads, int kv_heads,
     int head_dim, int value_dim, int value_row_width, float scale, int window, int keep_first,
     const float* __restrict__ sinks, const T* __restrict__ gate, size_t gate_stride, int gate_per_head, float softcap,
-    const float* __restrict__ rel_bias, int rel_rows, int chunk_size) {
+    const float* __restrict__ rel_bias, int rel_rows, int chunk_size, const float* __restrict__ slopes) {
   __shared__ float q_shared[kWarpsPerBlock][kMaxHeadDim];
   const int lane = threadIdx.x;
   const int warp = threadIdx.y;
@@ -91,6 +92,7 @@ __global__ void paged_attention_generic_kernel(
       }
       score = dot * scale;
       if (softcap > 0.0f) score = softcap * tanhf(score / softcap);
+      if (slopes != nullptr) score = fmaf(-slopes[head], (float)(position - key), score);
       if (rel_bias != nullptr) score += rel_bias[(size_t)head * rel_rows + min(position - key, rel_rows - 1)];
     }
     const float next_max = fmaxf(running_max, warp_max(score));
@@ -144,7 +146,7 @@ MIR_EXPORT int mir_paged_attention_generic(int bf16, const void* q, long long q_
                                            float scale, int window, int keep_first, int value_row_width,
                                            const float* sinks, const void* gate, long long gate_stride,
                                            int gate_per_head, float softcap, const float* rel_bias, int rel_rows,
-                                           int chunk, cudaStream_t stream) {
+                                           int chunk, const float* slopes, cudaStream_t stream) {
   if (tokens == 0) return MIR_OK;
   if (tokens < 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || page_size <= 0 || table_width <= 0 ||
       window < 0 || keep_first < 0 || chunk < 0 || (chunk > 0 && keep_first > 0)) {
@@ -169,12 +171,12 @@ MIR_EXPORT int mir_paged_attention_generic(int bf16, const void* q, long long q_
         (const __nv_bfloat16*)q, (size_t)q_token_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_pages,
         (const __nv_bfloat16*)v_pages, block_table, table_width, row_of_token, positions, page_size, heads, kv_heads,
         head_dim, value_dim, value_row_width, scale, window, keep_first, sinks, (const __nv_bfloat16*)gate,
-        (size_t)gate_stride, gate_per_head, softcap, rel_bias, rel_rows, chunk);
+        (size_t)gate_stride, gate_per_head, softcap, rel_bias, rel_rows, chunk, slopes);
   else
     paged_attention_generic_kernel<<<grid, block, 0, stream>>>(
         (const float*)q, (size_t)q_token_stride, (float*)out, (const float*)k_pages, (const float*)v_pages,
         block_table, table_width, row_of_token, positions, page_size, heads, kv_heads, head_dim, value_dim,
         value_row_width, scale, window, keep_first, sinks, (const float*)gate, (size_t)gate_stride, gate_per_head, softcap,
-        rel_bias, rel_rows, chunk);
+        rel_bias, rel_rows, chunk, slopes);
   return mir_check_launch("paged_attention_generic");
 }

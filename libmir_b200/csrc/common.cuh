@@ -126,6 +126,10 @@ struct AttentionExtras {
   float softcap = 0.0f;
   const float* rel_bias = nullptr;
   int rel_rows = 0, rel_heads = 0;
+  // slopes [heads] 32-bit (or null): slopes[h] * (query position - key position) is taken off the score after the cap.
+  const float* slopes = nullptr;
+  // the width of a value head where it differs from a key head's (0: the same)
+  int value_dim = 0;
 };
 // The sink's share of a denominator whose terms are exp2(score * log2 e - reference).
 __device__ __forceinline__ float sink_term(const AttentionExtras& extras, int head, float reference) {
@@ -137,7 +141,7 @@ __device__ __forceinline__ float gate_factor(const AttentionExtras& extras, size
   return 1.0f / (1.0f + __expf(-__bfloat162float(extras.gate[token * (size_t)extras.gate_stride + column])));
 }
 __device__ __forceinline__ bool scores_modified(const AttentionExtras& extras) {
-  return extras.softcap > 0.0f || extras.rel_bias != nullptr;
+  return extras.softcap > 0.0f || extras.rel_bias != nullptr || extras.slopes != nullptr;
 }
 // A score that is already scaled and in units of log2 e (the tile kernels' form), capped and biased in 32-bit.
 __device__ __forceinline__ float modified_score(const AttentionExtras& extras, float score_log2, int distance, int head) {
@@ -145,6 +149,7 @@ __device__ __forceinline__ float modified_score(const AttentionExtras& extras, f
   if (extras.softcap > 0.0f) x = extras.softcap * tanhf(x / extras.softcap);
   if (extras.rel_bias != nullptr)
     x += extras.rel_bias[(size_t)min(head, extras.rel_heads - 1) * extras.rel_rows + min(max(distance, 0), extras.rel_rows - 1)];
+  if (extras.slopes != nullptr) x = fmaf(-extras.slopes[min(head, extras.rel_heads - 1)], (float)max(distance, 0), x);
   return x * 1.4426950408889634f;
 }
 

@@ -373,6 +373,28 @@ __global__ void gated_head_norm_kernel(const float* __restrict__ o, const TG* __
   }
 }
 
+// The same for wide rows (a norm over all heads at once): one CTA per (token, head), its sum by a fixed tree.
+template <typename T, typename TG>
+__global__ void gated_wide_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, long long ld_gate,
+                                       const float* __restrict__ weight, T* __restrict__ out, int heads, int value_dim,
+                                       float eps, int sigmoid_gate, int weight_per_head) {
+  __shared__ float scratch[32];
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int unit = blockIdx.x;                                  // token * heads + head
+  const float* src = o + (size_t)unit * value_dim;
+  float sum = 0.0f;
+  for (int d = threadIdx.x; d < value_dim; d += blockDim.x) sum = fmaf(src[d], src[d], sum);
+  const float inverse = rsqrtf(block_sum(sum, scratch) / (float)value_dim + eps);
+  const TG* gate_row = gate + (size_t)(unit / heads) * ld_gate + (size_t)(unit % heads) * value_dim;
+  const float* scale = weight + (weight_per_head ? (size_t)(unit % heads) * value_dim : 0);
+  for (int d = threadIdx.x; d < value_dim; d += blockDim.x) {
+    const float z = to_float(gate_row[d]);
+    out[(size_t)unit * value_dim + d] = from_float<T>(src[d] * inverse * scale[d] * (sigmoid_gate ? sigmoid(z) : silu(z)));
+  }
+}
+constexpr int kWideNormColumns = 512;                           // rows from this width on take a CTA each
+
 // How many lanes share a column of the state: 0 lets the launcher choose, 8 / 16 / 32 fix it (for measurements).
 int g_scan_lanes = 0;
 
@@ -515,6 +537,20 @@ MIR_EXPORT int mir_gated_head_norm(int bf16, int gate_f32, const float* o, const
   if (tokens == 0) return MIR_OK;
   if (tokens < 0 || heads <= 0 || value_dim <= 0) { mir_set_error("gated_head_norm: bad sizes"); return MIR_BAD_ARGUMENT; }
   const int units = tokens * heads;
+  if (value_dim >= kWideNormColumns) {
+    const dim3 threads(256);
+    if (bf16 && gate_f32)
+      return mir_launch("gated_head_norm", gated_wide_norm_kernel<__nv_bfloat16, float>, dim3(units), threads, 0, stream, 0,
+                        o, (const float*)gate, ld_gate, weight, (__nv_bfloat16*)out, heads, value_dim, eps, sigmoid_gate,
+                        weight_per_head);
+    if (bf16)
+      return mir_launch("gated_head_norm", gated_wide_norm_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(units), threads, 0,
+                        stream, 0, o, (const __nv_bfloat16*)gate, ld_gate, weight, (__nv_bfloat16*)out, heads, value_dim,
+                        eps, sigmoid_gate, weight_per_head);
+    return mir_launch("gated_head_norm", gated_wide_norm_kernel<float, float>, dim3(units), threads, 0, stream, 0, o,
+                      (const float*)gate, ld_gate, weight, (float*)out, heads, value_dim, eps, sigmoid_gate,
+                      weight_per_head);
+  }
   const dim3 grid((units + 3) / 4), block(32, 4);
   if (bf16 && gate_f32)
     return mir_launch("gated_head_norm", gated_head_norm_kernel<__nv_bfloat16, float>, grid, block, 0, stream, 0, o,

@@ -130,6 +130,95 @@ __global__ void add_normed_branches_vec4_kernel(NormedBranches branches, float* 
   }
 }
 
+// residual[r, :] = u * rsqrt(mean(u^2) + eps) * weight with u = alpha * residual[r, :] + sum over branches b of
+// scale_b * branch_b[r, :]: what stands behind a sublayer whose norm comes after the sum.  One CTA per row, which stays
+// in registers between the sum and the norm (V columns a thread and access, PIECES of them blockDim.x * V columns apart).
+// `rounded` (may be null): the new rows once more, rounded to bfloat16, for the product that reads them next.
+struct ScaledBranches {
+  const float* rows[4];
+  float scale[4];
+  int count;
+};
+template <int V, int PIECES>
+__global__ void __launch_bounds__(512) norm_scaled_sum_kernel(ScaledBranches branches, float* __restrict__ residual,
+                                                              const float* __restrict__ weight,
+                                                              __nv_bfloat16* __restrict__ rounded, int hidden, float alpha,
+                                                              float eps) {
+  __shared__ float scratch[32];
+  grid_launch_dependents();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
+  const size_t base = (size_t)blockIdx.x * hidden;
+  auto load = [](float (&v)[V], const float* from) {
+    if constexpr (V == 4) {
+      const float4 a = *reinterpret_cast<const float4*>(from);
+      v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    } else {
+      v[0] = *from;
+    }
+  };
+  float w[PIECES][V];                                // the weight is older than the kernel before this one
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * V;
+    if (c < hidden) load(w[p], weight + c);
+  }
+  grid_dependency_wait();
+  float u[PIECES][V];
+  float sum = 0.0f;
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * V;
+#pragma unroll
+    for (int v = 0; v < V; ++v) u[p][v] = 0.0f;
+    if (c >= hidden) continue;
+    load(u[p], residual + base + c);
+#pragma unroll
+    for (int v = 0; v < V; ++v) u[p][v] *= alpha;
+    for (int b = 0; b < branches.count; ++b) {
+      float piece[V];
+      load(piece, branches.rows[b] + base + c);
+#pragma unroll
+      for (int v = 0; v < V; ++v) u[p][v] = fmaf(branches.scale[b], piece[v], u[p][v]);
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) sum = fmaf(u[p][v], u[p][v], sum);
+  }
+  sum = warp_sum(sum);
+  if (lane == 0) scratch[warp] = sum;
+  __syncthreads();
+  float total = 0.0f;
+  for (int i = 0; i < warps; ++i) total += scratch[i];
+  const float inverse = rsqrtf(total / (float)hidden + eps);
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int c = (p * blockDim.x + threadIdx.x) * V;
+    if (c >= hidden) continue;
+#pragma unroll
+    for (int v = 0; v < V; ++v) u[p][v] *= inverse * w[p][v];
+    if constexpr (V == 4) {
+      *reinterpret_cast<float4*>(residual + base + c) = make_float4(u[p][0], u[p][1], u[p][2], u[p][3]);
+      if (rounded) {
+        uint2 packed;
+        *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(u[p][0], u[p][1]);
+        *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(u[p][2], u[p][3]);
+        *reinterpret_cast<uint2*>(rounded + base + c) = packed;
+      }
+    } else {
+      residual[base + c] = u[p][0];
+      if (rounded) rounded[base + c] = __float2bfloat16(u[p][0]);
+    }
+  }
+}
+
+// out[i] (+)= sum over branches b of scale_b * branch_b[i].
+__global__ void scaled_sum_kernel(ScaledBranches branches, float* __restrict__ out, size_t total, int accumulate) {
+  const size_t index = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (index >= total) return;
+  float sum = accumulate ? out[index] : 0.0f;
+  for (int b = 0; b < branches.count; ++b) sum = fmaf(branches.scale[b], branches.rows[b][index], sum);
+  out[index] = sum;
+}
+
 // gelu_tanh on eight bfloat16 values per thread (16-byte accesses).
 __global__ void gelu_tanh_bf16x8_kernel(__nv_bfloat16* __restrict__ x, size_t total8) {
   const size_t index = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -361,6 +450,54 @@ MIR_EXPORT int mir_add_normed_branches(const float* const* branch_rows, const fl
   const int threads = hidden >= 2048 ? 512 : 256;
   return mir_launch("add_normed_branches", add_normed_branches_kernel, dim3(rows), dim3(threads), 0, stream, 0, branches,
                     residual, (__nv_bfloat16*)rounded, hidden, eps, scale);
+}
+
+// branch_rows: `count` (1 to 4) pointers to 32-bit [rows, hidden]; scales: as many numbers; the rest as
+// norm_scaled_sum_kernel says.
+MIR_EXPORT int mir_norm_scaled_sum(const float* const* branch_rows, const float* scales, int count, float* residual,
+                                   const float* weight, void* rounded, int rows, int hidden, float alpha, float eps,
+                                   cudaStream_t stream) {
+  if (rows == 0) return MIR_OK;
+  if (rows < 0 || hidden <= 0 || count < 1 || count > 4) { mir_set_error("norm_scaled_sum: bad sizes"); return MIR_BAD_ARGUMENT; }
+  ScaledBranches branches = {};
+  branches.count = count;
+  bool aligned = (hidden & 3) == 0 && ((uintptr_t)residual & 15) == 0 && ((uintptr_t)weight & 15) == 0 &&
+                 ((uintptr_t)rounded & 7) == 0;
+  for (int b = 0; b < count; ++b) {
+    branches.rows[b] = branch_rows[b];
+    branches.scale[b] = scales[b];
+    aligned = aligned && ((uintptr_t)branch_rows[b] & 15) == 0;
+  }
+#define MIR_NORM_SUM(V, P)                                                                                              \
+  return mir_launch("norm_scaled_sum", norm_scaled_sum_kernel<V, P>, dim3(rows), dim3(threads), 0, stream, 0, branches, \
+                    residual, weight, (__nv_bfloat16*)rounded, hidden, alpha, eps)
+  const int per_thread = aligned ? 4 : 1;
+  const int places = (hidden + per_thread - 1) / per_thread;
+  const int threads = places >= 512 ? 512 : (places + 31) / 32 * 32;
+  const int pieces = (places + threads - 1) / threads;
+  if (per_thread == 4) {
+    if (pieces <= 1) MIR_NORM_SUM(4, 1);
+    if (pieces <= 2) MIR_NORM_SUM(4, 2);
+    if (pieces <= 4) MIR_NORM_SUM(4, 4);
+    if (pieces <= 8) MIR_NORM_SUM(4, 8);
+  } else {
+    if (pieces <= 2) MIR_NORM_SUM(1, 2);
+    if (pieces <= 8) MIR_NORM_SUM(1, 8);
+    if (pieces <= 32) MIR_NORM_SUM(1, 32);
+  }
+#undef MIR_NORM_SUM
+  mir_set_error("norm_scaled_sum: rows of %d numbers are wider than the kernel takes", hidden);
+  return MIR_BAD_ARGUMENT;
+}
+
+MIR_EXPORT int mir_scaled_sum(const float* const* branch_rows, const float* scales, int count, float* out, size_t total,
+                              int accumulate, cudaStream_t stream) {
+  if (count < 1 || count > 4) { mir_set_error("scaled_sum: one to four branches"); return MIR_BAD_ARGUMENT; }
+  ScaledBranches branches = {};
+  branches.count = count;
+  for (int b = 0; b < count; ++b) { branches.rows[b] = branch_rows[b]; branches.scale[b] = scales[b]; }
+  LAUNCH_1D(scaled_sum_kernel, total, branches, out, total, accumulate);
+  return mir_check_launch("scaled_sum");
 }
 
 MIR_EXPORT int mir_rms_norm(int bf16, const float* x, const float* weight, void* out, const int* rows, int n_rows,

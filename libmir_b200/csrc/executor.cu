@@ -201,7 +201,7 @@ struct Run {
                                        group.block_table, group.table_width, step.row_of_token, step.positions,
                                        step.tokens, layer.page_size, layer.heads, layer.kv_heads, layer.head_dim,
                                        layer.head_dim, layer.scale, layer.window, 0, 0, nullptr, nullptr, 0, 0, 0.0f,
-                                       nullptr, 0, 0, step.stream);
+                                       nullptr, 0, 0, nullptr, step.stream);
   }
 
   int feed_forward(const MirLayerDesc& layer, const MirNormDesc* upcoming) {

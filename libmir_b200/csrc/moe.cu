@@ -70,7 +70,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
   for (int e = lane; e < experts; e += 32) {
     const float s = softmax_scores ? expf(z[e] - softmax_top) * softmax_inverse : sigmoid_of(z[e]);
     score[e] = s;
-    choice[e] = correction != nullptr ? s + correction[e] : s;
+    // (plain softmax scores are in the logits' order: the choice then looks at the logits, which do not underflow)
+    choice[e] = correction != nullptr ? s + correction[e] : (softmax_scores && keep >= groups ? z[e] : s);
   }
   if (has_gate && lane == 0) shared_gate[token] = sigmoid_of(z[experts]);
   __syncwarp();

@@ -5,6 +5,8 @@
 //   q and k are the projections' results rotated by the token's position (half-split pairs i, i + r/2 of the first r
 //   channels; angle = position * inv_freq[i], a 32-bit product), k also times key_scale, both in 32-bit while a chunk
 //   of tokens is staged in shared memory: nothing rotated is ever rounded to the storage type.
+//   With `activated` the recurrence's inputs are silu of the projections' results (of q and k before the rotation, and of
+//   v), also in 32-bit while they are staged.
 // The decay, the rotation, the state and every sum are 32-bit; T is the storage type of the projections' results.
 // One lane count and one order of sums for every shape of step: a request's 32-bit results do not depend on how it was
 // cut into steps.  A row of a captured decode batch whose position is negative is padding: nothing is read or written.
@@ -29,6 +31,11 @@ struct TokenInputs {
   float position;
 };
 
+// What enters the recurrence of a projection's element: the element, or its silu.
+__device__ __forceinline__ float entering(float z, int activated) {
+  return activated ? z / (1.0f + expf(-z)) : z;
+}
+
 template <typename T, int PER_LANE>
 __device__ __forceinline__ void load_token(TokenInputs<T, PER_LANE>& in, const T* __restrict__ q,
                                            const T* __restrict__ k, size_t source, bool live, float position, int lane,
@@ -50,17 +57,17 @@ __device__ __forceinline__ void load_token(TokenInputs<T, PER_LANE>& in, const T
 
 template <typename T, int PER_LANE>
 __device__ __forceinline__ void stage_token(const TokenInputs<T, PER_LANE>& in, const float* frequency, float key_scale,
-                                            int lane, int half, int rotary_dim, float* row) {
+                                            int lane, int half, int rotary_dim, int activated, float* row) {
   constexpr int PADDED = 32 * PER_LANE;
   float sum = 0.0f;
 #pragma unroll
   for (int e = 0; e < PER_LANE; ++e) {
     const int i = lane + 32 * e;
     if (32 * e >= half && 32 * e + 32 <= rotary_dim) continue;   // a warp of partners: their owners write them
-    const float qi = to_float(in.q[e]), ki = to_float(in.k[e]);
+    const float qi = entering(to_float(in.q[e]), activated), ki = entering(to_float(in.k[e]), activated);
     if (e < TokenInputs<T, PER_LANE>::PAIRED && i < half) {
       // the first of a pair becomes u cos - v sin, the second v cos + u sin
-      const float qp = to_float(in.partner_q[e]), kp = to_float(in.partner_k[e]);
+      const float qp = entering(to_float(in.partner_q[e]), activated), kp = entering(to_float(in.partner_k[e]), activated);
       float sine, cosine;
       sincosf(__fmul_rn(in.position, frequency[e]), &sine, &cosine);
       const float q_first = fmaf(qi, cosine, -__fmul_rn(qp, sine)), q_second = fmaf(qp, cosine, __fmul_rn(qi, sine));
@@ -92,7 +99,7 @@ retention_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T*
                       const float* __restrict__ inv_freq, int rotary_dim, const float* __restrict__ decays,
                       float key_scale, float* __restrict__ state, const int* __restrict__ query_starts,
                       const int* __restrict__ state_slots, const int* __restrict__ positions, float* __restrict__ out,
-                      int heads, int dim, int value_dim) {
+                      int heads, int dim, int value_dim, int activated) {
   constexpr int COLUMNS = 32 / kLanes;
   constexpr int BLOCK_COLUMNS = COLUMNS * kWarps;
   constexpr int PADDED = kLanes * PER;
@@ -164,13 +171,13 @@ retention_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T*
     for (int tt = 0; tt < TOKENS_PER_WARP; ++tt) {
       const int t = warp + tt * kWarps;
       if (t >= count) continue;                                  // (the same for the whole warp)
-      stage_token(next[tt], frequency, key_scale, lane, half, rotary_dim, staged + t * ROW);
+      stage_token(next[tt], frequency, key_scale, lane, half, rotary_dim, activated, staged + t * ROW);
     }
 #pragma unroll
     for (int j = 0; j < VALUES_PER_THREAD; ++j) {
       const int index = thread + j * kWarps * 32;
       const int t = index / BLOCK_COLUMNS, c = index - t * BLOCK_COLUMNS;
-      if (t < CHUNK) staged[t * ROW + 2 * PADDED + 4 + c] = to_float(next_v[j]);
+      if (t < CHUNK) staged[t * ROW + 2 * PADDED + 4 + c] = entering(to_float(next_v[j]), activated);
     }
   };
   fetch(start);
@@ -228,7 +235,8 @@ template <typename T, int PER_LANE>
 __global__ void __launch_bounds__(kWarps * 32)
 retention_prepare_kernel(const T* __restrict__ q, const T* __restrict__ k, long long ld,
                          const float* __restrict__ inv_freq, int rotary_dim, float key_scale,
-                         const int* __restrict__ positions, float* __restrict__ prepared, int tokens, int heads, int dim) {
+                         const int* __restrict__ positions, float* __restrict__ prepared, int tokens, int heads, int dim,
+                         int activated) {
   constexpr int PADDED = 32 * PER_LANE;
   using Inputs = TokenInputs<T, PER_LANE>;
   grid_launch_dependents();
@@ -245,7 +253,7 @@ retention_prepare_kernel(const T* __restrict__ q, const T* __restrict__ k, long 
   for (int e = 0; e < Inputs::PAIRED; ++e) frequency[e] = lane + 32 * e < half ? inv_freq[lane + 32 * e] : 0.0f;
   Inputs in;
   load_token(in, q, k, (size_t)token * ld + (size_t)head * dim, true, (float)position, lane, dim, half, rotary_dim);
-  stage_token(in, frequency, key_scale, lane, half, rotary_dim, prepared + (size_t)unit * (2 * PADDED + 4));
+  stage_token(in, frequency, key_scale, lane, half, rotary_dim, activated, prepared + (size_t)unit * (2 * PADDED + 4));
 }
 
 // The walk over prepared rows: as retention_scan_kernel, but a chunk's q, k and q . k arrive by 16-byte asynchronous
@@ -257,7 +265,7 @@ retention_scan_prepared_kernel(const float* __restrict__ prepared, const T* __re
                                const float* __restrict__ decays, float* __restrict__ state,
                                const int* __restrict__ query_starts, const int* __restrict__ state_slots,
                                const int* __restrict__ positions, float* __restrict__ out, int heads, int dim,
-                               int value_dim) {
+                               int value_dim, int activated) {
   constexpr int COLUMNS = 32 / kLanes;
   constexpr int BLOCK_COLUMNS = COLUMNS * kWarps;
   constexpr int PADDED = kLanes * PER;
@@ -325,7 +333,7 @@ retention_scan_prepared_kernel(const float* __restrict__ prepared, const T* __re
     for (int j = 0; j < VALUES_PER_THREAD; ++j) {
       const int index = thread + j * kWarps * 32;
       const int t = index / BLOCK_COLUMNS, c = index - t * BLOCK_COLUMNS;
-      if (t < CHUNK) staged[stage][t * ROW + PREPARED + c] = to_float(next_v[j]);
+      if (t < CHUNK) staged[stage][t * ROW + PREPARED + c] = entering(to_float(next_v[j]), activated);
     }
     __syncthreads();                   // this chunk is whole, and every thread has left the chunk before
     if (from + CHUNK < end) issue(from + CHUNK, stage ^ 1);
@@ -389,45 +397,47 @@ template <typename T, int PER, int kLanes>
 int launch_prepared(cudaStream_t stream, const void* q, const void* k, const void* v, long long ld, const float* inv_freq,
                     int rotary_dim, const float* decays, float key_scale, float* state, const int* query_starts,
                     const int* state_slots, const int* positions, float* out, float* prepared, int tokens, int rows,
-                    int heads, int dim, int value_dim) {
+                    int heads, int dim, int value_dim, int activated) {
   constexpr int columns = kWarps * (32 / kLanes);
   const long long units = (long long)tokens * heads;
   int status = mir_launch("retention_prepare", retention_prepare_kernel<T, kLanes * PER / 32>,
                           dim3((unsigned)((units + kWarps - 1) / kWarps)), dim3(32, kWarps), 0, stream, 0, (const T*)q,
-                          (const T*)k, ld, inv_freq, rotary_dim, key_scale, positions, prepared, tokens, heads, dim);
+                          (const T*)k, ld, inv_freq, rotary_dim, key_scale, positions, prepared, tokens, heads, dim,
+                          activated);
   if (status != MIR_OK) return status;
   return mir_launch("retention_scan", retention_scan_prepared_kernel<T, PER, kLanes>,
                     dim3(rows, heads, (value_dim + columns - 1) / columns), dim3(32, kWarps), 0, stream, 0,
                     (const float*)prepared, (const T*)v, ld, decays, state, query_starts, state_slots, positions, out,
-                    heads, dim, value_dim);
+                    heads, dim, value_dim, activated);
 }
 
 template <typename T, int PER, int kLanes, bool SHORT>
 int launch_scan(cudaStream_t stream, const void* q, const void* k, const void* v, long long ld, const float* inv_freq,
                 int rotary_dim, const float* decays, float key_scale, float* state, const int* query_starts,
-                const int* state_slots, const int* positions, float* out, int rows, int heads, int dim, int value_dim) {
+                const int* state_slots, const int* positions, float* out, int rows, int heads, int dim, int value_dim,
+                int activated) {
   constexpr int columns = kWarps * (32 / kLanes);
   return mir_launch("retention_scan", retention_scan_kernel<T, PER, kLanes, SHORT>,
                     dim3(rows, heads, (value_dim + columns - 1) / columns), dim3(32, kWarps), 0, stream, 0, (const T*)q,
                     (const T*)k, (const T*)v, ld, inv_freq, rotary_dim, decays, key_scale, state, query_starts,
-                    state_slots, positions, out, heads, dim, value_dim);
+                    state_slots, positions, out, heads, dim, value_dim, activated);
 }
 
 template <typename T>
 int launch_scan_for(cudaStream_t stream, const void* q, const void* k, const void* v, long long ld,
                     const float* inv_freq, int rotary_dim, const float* decays, float key_scale, float* state,
                     const int* query_starts, const int* state_slots, const int* positions, float* out, int rows,
-                    int heads, int dim, int value_dim, bool single_tokens, float* prepared, int tokens) {
+                    int heads, int dim, int value_dim, bool single_tokens, float* prepared, int tokens, int activated) {
 #define MIR_RETENTION(P, L)                                                                                         \
   if (prepared && !single_tokens)                                                                                   \
     return launch_prepared<T, P, L>(stream, q, k, v, ld, inv_freq, rotary_dim, decays, key_scale, state,           \
                                     query_starts, state_slots, positions, out, prepared, tokens, rows, heads, dim,  \
-                                    value_dim);                                                                     \
+                                    value_dim, activated);                                                          \
   if (single_tokens)                                                                                                \
     return launch_scan<T, P, L, true>(stream, q, k, v, ld, inv_freq, rotary_dim, decays, key_scale, state,         \
-                                      query_starts, state_slots, positions, out, rows, heads, dim, value_dim);     \
+                                      query_starts, state_slots, positions, out, rows, heads, dim, value_dim, activated); \
   return launch_scan<T, P, L, false>(stream, q, k, v, ld, inv_freq, rotary_dim, decays, key_scale, state,          \
-                                     query_starts, state_slots, positions, out, rows, heads, dim, value_dim);
+                                     query_starts, state_slots, positions, out, rows, heads, dim, value_dim, activated);
   if (dim <= 32) { MIR_RETENTION(4, 8) }
   if (dim <= 64) { MIR_RETENTION(4, 16) }
   if (dim <= 128) { MIR_RETENTION(8, 16) }
@@ -445,11 +455,12 @@ int launch_scan_for(cudaStream_t stream, const void* q, const void* k, const voi
 // state [slots, heads, value_dim, dim] 32-bit; out [tokens, heads * value_dim] 32-bit: o before the head norm.
 // prepared: null, or 32-bit scratch of tokens * heads * (2 * padded + 4) numbers, padded = the key width rounded up to
 // 32, 64, 128, 192 or 256: a step that brings more than single tokens then rotates in a kernel of its own first.
+// activated: silu on q, k and v as they enter.
 MIR_EXPORT int mir_retention_scan(int bf16, const void* q, const void* k, const void* v, long long ld,
                                   const float* inv_freq, int rotary_dim, const float* decays, float key_scale,
                                   float* state, const int* query_starts, const int* state_slots, const int* positions,
                                   float* out, float* prepared, int tokens, int rows, int heads, int dim, int value_dim,
-                                  cudaStream_t stream) {
+                                  int activated, cudaStream_t stream) {
   if (tokens == 0 || rows == 0) return MIR_OK;
   if (tokens < 0 || rows < 0 || heads <= 0 || dim <= 0 || value_dim <= 0 || heads > 65535 || rotary_dim < 0 ||
       rotary_dim > dim || (rotary_dim & 1) || (rotary_dim > 0 && inv_freq == nullptr)) {
@@ -461,7 +472,8 @@ MIR_EXPORT int mir_retention_scan(int bf16, const void* q, const void* k, const 
   if (bf16)
     return launch_scan_for<__nv_bfloat16>(stream, q, k, v, ld, inv_freq, rotary_dim, decays, key_scale, state,
                                           query_starts, state_slots, positions, out, rows, heads, dim, value_dim,
-                                          single_tokens, prepared, tokens);
+                                          single_tokens, prepared, tokens, activated);
   return launch_scan_for<float>(stream, q, k, v, ld, inv_freq, rotary_dim, decays, key_scale, state, query_starts,
-                                state_slots, positions, out, rows, heads, dim, value_dim, single_tokens, prepared, tokens);
+                                state_slots, positions, out, rows, heads, dim, value_dim, single_tokens, prepared, tokens,
+                                activated);
 }

@@ -31,10 +31,16 @@ _SIGNATURES = {
         "mir_cast": [c_int, c_void_p, c_void_p, c_size_t, c_void_p],
         "mir_qk_rope_store": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                               c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_longlong, c_int, c_void_p],
+        "mir_qk_rope_store_forms": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                    c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_longlong, c_int,
+                                    c_float, c_float, c_float, c_int, c_void_p],
+        "mir_norm_scaled_sum": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float,
+                                c_void_p],
+        "mir_scaled_sum": [c_void_p, c_void_p, c_int, c_void_p, c_size_t, c_int, c_void_p],
         "mir_paged_attention_generic": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
                                         c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_float, c_void_p, c_int,
-                                        c_int, c_void_p],
+                                        c_int, c_void_p, c_void_p],
         "mir_paged_attention_mixed": [c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                       c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int,
                                       c_void_p],
@@ -83,7 +89,7 @@ _SIGNATURES = {
                         c_int, c_int, c_int, c_int, c_void_p],
         "mir_retention_scan": [c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_float,
                                c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                               c_int, c_void_p],
+                               c_int, c_int, c_void_p],
         "mir_wkv_scan": [c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "mir_moe_route": [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -460,6 +466,37 @@ def add_normed_branches(branches, weights, residual: torch.Tensor, eps: float, s
     lib = library("core")
     _check(lib, lib.mir_add_normed_branches(pointers, weight_pointers, len(branches), residual.data_ptr(), _ptr(rounded),
                                             rows, hidden, eps, scale, _stream()))
+
+
+def _scaled_branches(what: str, branches, scales, like: torch.Tensor):
+    _require(1 <= len(branches) <= 4 and len(scales) == len(branches) and like.dtype == torch.float32
+             and like.is_contiguous() and all(b.dtype == torch.float32 and b.shape == like.shape and b.is_contiguous()
+                                              for b in branches), f"{what}: one to four 32-bit branches of one shape")
+    return (c_void_p * len(branches))(*[b.data_ptr() for b in branches]), (c_float * len(scales))(*[float(s) for s in scales])
+
+
+def norm_scaled_sum(branches, scales, residual: torch.Tensor, weight: torch.Tensor, alpha: float, eps: float,
+                    rounded: Optional[torch.Tensor] = None) -> None:
+    """residual <- rmsnorm(alpha * residual + sum_b scales[b] * branches[b]) * weight, every tensor 32-bit, branches and
+    residual [rows, hidden].  `rounded` (bfloat16 [rows, hidden], contiguous) also receives the new residual."""
+    _cuda(residual, weight, rounded, *branches)
+    pointers, factors = _scaled_branches("norm_scaled_sum", branches, scales, residual)
+    rows, hidden = residual.shape
+    _require(weight.dtype == torch.float32 and weight.numel() == hidden and weight.is_contiguous()
+             and (rounded is None or (rounded.dtype == torch.bfloat16 and rounded.shape == residual.shape
+                                      and rounded.is_contiguous())),
+             "norm_scaled_sum: the weight is float32 [hidden], rounded bfloat16 [rows, hidden]")
+    lib = library("core")
+    _check(lib, lib.mir_norm_scaled_sum(pointers, factors, len(branches), residual.data_ptr(), weight.data_ptr(),
+                                        _ptr(rounded), rows, hidden, float(alpha), float(eps), _stream()))
+
+
+def scaled_sum(branches, scales, out: torch.Tensor, accumulate: bool = False) -> None:
+    """out = sum_b scales[b] * branches[b], or out += it with `accumulate`; every tensor 32-bit of one shape."""
+    _cuda(out, *branches)
+    pointers, factors = _scaled_branches("scaled_sum", branches, scales, out)
+    lib = library("core")
+    _check(lib, lib.mir_scaled_sum(pointers, factors, len(branches), out.data_ptr(), out.numel(), int(accumulate), _stream()))
 
 
 def short_conv_silu(x: torch.Tensor, weight: torch.Tensor, tail: torch.Tensor, row_of_token: torch.Tensor,
@@ -891,14 +928,15 @@ def retention_prepared_floats(tokens: int, heads: int, dim: int) -> int:
 def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, inv_freq: Optional[torch.Tensor],
                    decays: torch.Tensor, key_scale: float, state: torch.Tensor, query_starts: torch.Tensor,
                    state_slots: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, heads: int, dim: int,
-                   value_dim: int, prepared: Optional[torch.Tensor] = None) -> None:
+                   value_dim: int, prepared: Optional[torch.Tensor] = None, activated: bool = False) -> None:
     """The retention recurrence over the tokens of each request row, from and into state [slots, heads, value_dim, dim]
     (32-bit): per head S <- decay_h S + k v^T, o = S^T q, with q and k rotated by the token's position (half-split pairs
     of the first 2 * len(inv_freq) channels, 32-bit angles) and k times `key_scale` after the rotation.  q, k [tokens,
     heads * dim] and v [tokens, heads * value_dim]: views with one row stride in the activations' dtype; decays 32-bit
     [heads]; out 32-bit [tokens, heads * value_dim].  With `prepared` (32-bit scratch of retention_prepared_floats
     numbers) a step that brings more than single tokens rotates in a kernel of its own, once per token and head, and
-    the walk copies what that left; the results are the same bits either way."""
+    the walk copies what that left; the results are the same bits either way.  `activated`: silu of q, k (ahead of the
+    rotation) and v enter instead of the projections' results."""
     _cuda(q, k, v, inv_freq, decays, state, query_starts, state_slots, positions, out, prepared)
     _require(prepared is None or (prepared.dtype == torch.float32 and prepared.is_contiguous()
                                   and prepared.numel() >= retention_prepared_floats(q.shape[0], heads, dim)),
@@ -920,7 +958,8 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, inv_freq: 
     _check(lib, lib.mir_retention_scan(_is_bf16(q), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0),
                                        _ptr(inv_freq), rotary, decays.data_ptr(), float(key_scale), state.data_ptr(),
                                        query_starts.data_ptr(), state_slots.data_ptr(), positions.data_ptr(),
-                                       out.data_ptr(), _ptr(prepared), tokens, rows, heads, dim, value_dim, _stream()))
+                                       out.data_ptr(), _ptr(prepared), tokens, rows, heads, dim, value_dim, int(activated),
+                                       _stream()))
 
 
 # --------------------------------------------------------------------------- routed experts
@@ -1264,16 +1303,21 @@ def qk_rope_store(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opti
                   k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], heads: int, kv_heads: int,
                   head_dim: int, rotary_dim: int, eps: float, write_kv: bool = True,
                   keys_in_place: bool = False, value_dim: Optional[int] = None, interleaved: bool = False,
-                  queries_only: bool = False) -> None:
+                  queries_only: bool = False, magnitude: float = 1.0, temperature: Optional[tuple] = None,
+                  values_from_keys: bool = False) -> None:
     """q/k-norm + rotary on the packed qkv rows in place for q, k and v into their pages.  `keys_in_place`:
     the keys are normed and rotated in place like the queries and nothing is written to the pages.  `interleaved`:
     the rotation pairs dims 2i and 2i + 1.  The rows may be wider than q, k and v (what lies behind them is left
-    alone); `queries_only`: they start with the query heads and hold no keys or values."""
+    alone); `queries_only`: they start with the query heads and hold no keys or values.  `magnitude` multiplies cos and
+    sin; `temperature` (coef, every): a query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1);
+    `values_from_keys`: the rows hold no values, a token's value is its key as projected (before norm and rotation)."""
     write_kv = write_kv and not keys_in_place and not queries_only
     _cuda(qkv, positions, slot_mapping, inv_freq, q_norm, k_norm, k_pages, v_pages)
     tokens = qkv.shape[0]
     value_dim = head_dim if value_dim is None else value_dim
-    packed = heads * head_dim if queries_only else (heads + kv_heads) * head_dim + kv_heads * value_dim
+    _require(not values_from_keys or value_dim == head_dim, "qk_rope_store: values that are the keys have their width")
+    packed = heads * head_dim if queries_only else (heads + kv_heads) * head_dim + (0 if values_from_keys
+                                                                                    else kv_heads * value_dim)
     _require(qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] >= packed and qkv.stride(0) >= qkv.shape[1]
              and not (keys_in_place and queries_only), "qk_rope_store: bad qkv")
     _require(positions.dtype == torch.int32 and positions.numel() >= tokens, "qk_rope_store: bad positions")
@@ -1288,11 +1332,13 @@ def qk_rope_store(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opti
                  and v_pages is not None and k_pages.dtype == qkv.dtype and v_pages.dtype == qkv.dtype,
                  "qk_rope_store: cache pages of the activations' dtype and a slot mapping are needed")
     lib = library("core")
-    _check(lib, lib.mir_qk_rope_store(_is_bf16(qkv), qkv.data_ptr(), positions.data_ptr(), _ptr(slot_mapping),
-                                      _ptr(inv_freq), _ptr(q_norm), _ptr(k_norm), _ptr(k_pages), _ptr(v_pages),
-                                      tokens, heads, kv_heads, head_dim, value_dim, rotary_dim, eps,
-                                      2 if keys_in_place else int(write_kv), int(interleaved), qkv.stride(0),
-                                      int(queries_only), _stream()))
+    coef, every = temperature if temperature is not None else (0.0, 0.0)
+    _check(lib, lib.mir_qk_rope_store_forms(_is_bf16(qkv), qkv.data_ptr(), positions.data_ptr(), _ptr(slot_mapping),
+                                            _ptr(inv_freq), _ptr(q_norm), _ptr(k_norm), _ptr(k_pages), _ptr(v_pages),
+                                            tokens, heads, kv_heads, head_dim, value_dim, rotary_dim, eps,
+                                            2 if keys_in_place else int(write_kv), int(interleaved), qkv.stride(0),
+                                            int(queries_only), float(magnitude), float(coef), float(every),
+                                            int(values_from_keys), _stream()))
 
 
 QK_NORM_SPANS = {None: 0, "head": 1, "projection": 2}
@@ -1350,7 +1396,7 @@ def paged_attention_generic(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
                             values_in_keys: bool = False, sinks: Optional[torch.Tensor] = None,
                             gate: Optional[torch.Tensor] = None, gate_per_head: bool = False,
                             softcap: Optional[float] = None, distance_bias: Optional[torch.Tensor] = None,
-                            chunk: Optional[int] = None) -> None:
+                            chunk: Optional[int] = None, slopes: Optional[torch.Tensor] = None) -> None:
     """out[t, h] = softmax over the visible cached keys of token t's request; q is read from the packed qkv rows.
     `value_dim`: width of a value head (head_dim if None); `keep_first`: with a window, the request's first keys
     that stay visible to every query; `values_in_keys`: a value is the first value_dim elements of its key (a cached
@@ -1359,10 +1405,13 @@ def paged_attention_generic(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
     result is multiplied by its sigmoid; with `gate_per_head` it is [tokens, heads], one number per head.  `softcap`:
     score <- softcap * tanh(score / softcap) after the scale.  `distance_bias` (float32 [heads, rows]): row
     min(query position - key position, rows - 1) is added to the scores after the cap.  `chunk`: positions are cut into
-    runs of that many, and a query sees the keys of its own run only."""
+    runs of that many, and a query sees the keys of its own run only.  `slopes` (float32 [heads]): slopes[h] * (query
+    position - key position) is taken off the scores after the cap."""
+    _require(slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == heads and slopes.is_contiguous()),
+             "paged_attention: slopes are float32 [heads]")
     if values_in_keys:
         v_pages = k_pages
-    _cuda(qkv, out, k_pages, v_pages, block_table, row_of_token, positions, sinks, gate, distance_bias)
+    _cuda(qkv, out, k_pages, v_pages, block_table, row_of_token, positions, sinks, gate, distance_bias, slopes)
     _require(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads and sinks.is_contiguous()),
              "paged_attention: sinks are float32 [heads]")
     _require(gate is None or (gate.dtype == out.dtype and gate.stride(1) == 1
@@ -1385,7 +1434,7 @@ def paged_attention_generic(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
         page_size, heads, kv_heads, head_dim, value_dim, scale, int(window or 0), int(keep_first or 0),
         head_dim if values_in_keys else 0, _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0,
         int(gate_per_head), float(softcap or 0.0), _ptr(distance_bias),
-        distance_bias.shape[1] if distance_bias is not None else 0, int(chunk or 0), _stream()))
+        distance_bias.shape[1] if distance_bias is not None else 0, int(chunk or 0), _ptr(slopes), _stream()))
 
 
 MIXED_TENSOR_CORES = True        # False: attention with mixed heads always runs the reference kernel

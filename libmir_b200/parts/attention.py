@@ -16,7 +16,10 @@ capped by softcap * tanh(score / softcap), and a stored bias by the bucket of th
 table is spread out to one row per distance when the weights are bound).  Positions cut into runs (`chunk`): a query
 sees the keys of its own run only.  Mixed heads (head_mix, a stored matrix M over the query heads): head h applies
 sum_g M[h, g] weights_g, the combination of all heads' softmax weights, to the values of its own kv head
-(csrc/attention_mixed.cu, csrc/attention_mixed_mma.cu).
+(csrc/attention_mixed.cu, csrc/attention_mixed_mma.cu).  No value tensor (values_from_keys): a token's value is its key as
+projected, which the kernel that norms and rotates the key writes to the value pages on the way.  A factor on the
+queries that grows with the position (temperature, in the same kernel), and a bias that falls linearly with the
+distance, slopes[h] per position (in every attention kernel, in 32-bit).
 """
 
 from __future__ import annotations
@@ -41,7 +44,7 @@ class SoftmaxAttention(Mixer):
             raise ValueError("heads must be divisible by kv_heads")
         self.q_width = s.heads * s.head_dim
         self.kv_width = s.kv_heads * s.head_dim
-        self.v_width = s.kv_heads * s.value_dim
+        self.v_width = 0 if s.values_from_keys else s.kv_heads * s.value_dim
         self.out_width = s.heads * s.value_dim
         self.stored = dict(s.names)              # local name -> the name the checkpoint uses
         self.position = build_part(s.position, env) if s.position is not None else None
@@ -68,6 +71,15 @@ class SoftmaxAttention(Mixer):
         if s.head_mix and (s.keep_first or s.sinks or s.fixed_sink is not None or s.gate or s.softcap is not None
                            or s.distance_bias is not None):
             raise ValueError("mixed heads go with plain scores: no sinks, gate, cap, bias or kept first tokens")
+        if s.values_from_keys and (s.value_dim != s.head_dim or not s.own_kv or self.other_norm):
+            raise ValueError("values that are the keys have their width, are the mixer's own, and go with the per-head norm "
+                             "ahead of the rotation")
+        if s.slopes and (len(s.slopes) != s.heads or s.head_mix or (s.keep_first and s.window is not None)):
+            raise ValueError("one slope per query head, without mixed heads and kept first tokens")
+        if s.temperature is not None and (self.other_norm or s.temperature.every <= 0):
+            raise ValueError("a temperature on the queries goes with the per-head norm ahead of the rotation")
+        self.slopes = torch.tensor([float(v) for v in s.slopes], dtype=torch.float32, device=env.device) if s.slopes else None
+        self.temperature = (s.temperature.coef, s.temperature.every) if s.temperature is not None else None
         if s.chunk is not None and s.keep_first:
             raise ValueError("runs of positions do not go with kept first tokens")
         if s.fixed_sink is not None:
@@ -76,6 +88,15 @@ class SoftmaxAttention(Mixer):
     @property
     def graph_safe(self):
         return self.position is None or self.position.graph_safe
+
+    @property
+    def plain(self):
+        """Whether this is what the native layer executor knows: no option beyond q/k-norm with weights, biases, a window."""
+        s = self.spec
+        return not (s.sinks or s.gate or not s.own_kv or s.fixed_sink is not None or self.other_norm or s.softcap is not None
+                    or s.distance_bias is not None or s.chunk is not None or s.head_mix or s.values_from_keys or s.slopes
+                    or s.temperature is not None or s.value_dim != s.head_dim
+                    or (s.window is not None and s.keep_first))
 
     def cache_requirement(self):
         s = self.spec
@@ -99,6 +120,8 @@ class SoftmaxAttention(Mixer):
 
         if not s.own_kv:                         # queries alone: keys and values are another entry's
             ranges = {"q_proj": ranges["q_proj"]}
+        if s.values_from_keys:
+            ranges.pop("v_proj")
         table = {f"{projection}.weight": ParamSpec((end - begin, s.hidden_size), sources=fused(projection, "weight"))
                  for projection, (begin, end) in ranges.items()}
         table["o_proj.weight"] = ParamSpec((s.hidden_size, self.out_width))
@@ -127,6 +150,8 @@ class SoftmaxAttention(Mixer):
         local_of = {stored: local for local, stored in self.stored.items()}
         tensors = {local_of.get(name, name): tensor for name, tensor in tensors.items()}
         projections = ("q_proj", "k_proj", "v_proj") if self.spec.own_kv else ("q_proj",)
+        if self.spec.values_from_keys:
+            projections = projections[:2]
         weights = [tensors[f"{name}.weight"] for name in projections]
         if self.spec.gate:
             weights.append(tensors["g_proj.weight"])
@@ -194,18 +219,20 @@ class SoftmaxAttention(Mixer):
         qkv = ctx.alloc((tokens, self.packed_width), self.env.dtype)
         group = ctx.groups[cache.group]
         rotation = self.position.rotation() if self.position is not None else (None, 0)
-        interleaved = False
-        if rotation is None and getattr(self.position, "interleaved", False) and self.position.magnitude == 1.0:
-            # the other pairing of the same rotation: the kernel that norms q and k and writes the cache knows it too
-            rotation, interleaved = (self.position.table, self.position.rotary_dim), True
-        if self.other_norm and (rotation is None or interleaved):
+        interleaved, magnitude = False, 1.0
+        if rotation is None and hasattr(self.position, "table"):
+            # the other pairing of the same rotation, or cos and sin with a factor: the kernel that norms q and k and
+            # writes the cache knows them too
+            rotation = (self.position.table, self.position.rotary_dim)
+            interleaved, magnitude = self.position.interleaved, self.position.magnitude
+        if self.other_norm and (rotation is None or interleaved or magnitude != 1.0):
             raise ValueError("these q/k norms go with the half-split rotation or none")
         if self.other_norm:
             self.project_with_other_norm(ctx, cache, group, x, qkv, *rotation)
         elif rotation is None:
             self.project_with_other_position(ctx, cache, group, x, qkv)
         else:
-            self.project(ctx, cache, group, x, qkv, *rotation, interleaved=interleaved)
+            self.project(ctx, cache, group, x, qkv, *rotation, interleaved=interleaved, magnitude=magnitude)
         mixed = ctx.alloc((tokens, self.out_width), self.env.dtype)
         self.attend(ctx, group, cache, qkv, mixed)
         if overwrite:
@@ -213,14 +240,15 @@ class SoftmaxAttention(Mixer):
         else:
             ctx.accumulate(mixed, self.w_o, residual, self.b_o)      # may also prepare the norm that follows
 
-    def project(self, ctx, cache, group, x, qkv, table, rotary_dim, interleaved=False):
+    def project(self, ctx, cache, group, x, qkv, table, rotary_dim, interleaved=False, magnitude=1.0):
         """Projection, then per-head norm, rotation and cache write in one kernel."""
         s = self.spec
         kernels.linear(x, self.w_qkv, qkv, self.b_qkv, alloc=ctx.alloc)
         kernels.qk_rope_store(qkv, ctx.positions, group.slot_mapping, table, self.q_norm, self.k_norm,
                               cache.k_pages, cache.v_pages, s.heads, s.kv_heads, s.head_dim, rotary_dim,
                               s.qk_norm_eps, write_kv=cache.writes and s.own_kv, value_dim=s.value_dim,
-                              interleaved=interleaved, queries_only=not s.own_kv)
+                              interleaved=interleaved, queries_only=not s.own_kv, magnitude=magnitude,
+                              temperature=self.temperature, values_from_keys=s.values_from_keys)
 
     def project_with_other_norm(self, ctx, cache, group, x, qkv, table, rotary_dim):
         """Projection, then the kernel that knows the norm over a whole projection, the norm without weights and the
@@ -237,6 +265,8 @@ class SoftmaxAttention(Mixer):
         s = self.spec
         if not s.own_kv:
             raise ValueError("a position encoding of another kind needs keys of the mixer's own")
+        if s.values_from_keys or s.temperature is not None:
+            raise ValueError("a position encoding of another kind goes with values of their own and no temperature")
         kernels.linear(x, self.w_qkv, qkv, self.b_qkv, alloc=ctx.alloc)
         if s.qk_norm:
             kernels.qk_rope_store(qkv, ctx.positions, None, None, self.q_norm, self.k_norm, None, None, s.heads,
@@ -261,9 +291,9 @@ class SoftmaxAttention(Mixer):
         kept = s.keep_first if s.window is not None else 0
         first = self.q_width + self.kv_columns
         gate = qkv[:, first:first + self.gate_width] if s.gate else None        # [tokens, heads * value_dim] or [tokens, heads]
-        scored = s.softcap is not None or self.distance_bias is not None or s.gate_per_head
+        scored = s.softcap is not None or self.distance_bias is not None or s.gate_per_head or self.slopes is not None
         fast = self.env.dtype == torch.bfloat16 and s.head_dim in kernels.FAST_HEAD_DIMS and s.value_dim == s.head_dim \
-            and s.chunk is None                  # (runs of positions without mixed heads: the reference kernel)
+            and s.chunk is None and self.slopes is None                  # (runs of positions without mixed heads: the reference kernel)
         if fast and scored and not kept:
             # capped or biased scores, or a gate per head: single tokens split over the keys, portions as tiles of
             # queries, each on the tcgen05 or the mma.sync kernel by size
@@ -331,7 +361,7 @@ class SoftmaxAttention(Mixer):
                                         s.window, value_dim=s.value_dim,
                                         keep_first=s.keep_first if s.window is not None else 0, sinks=self.sinks,
                                         gate=gate, gate_per_head=s.gate_per_head, softcap=s.softcap,
-                                        distance_bias=self.distance_bias, chunk=s.chunk)
+                                        distance_bias=self.distance_bias, chunk=s.chunk, slopes=self.slopes)
 
     def attend_mixed(self, ctx, group, cache, qkv, out):
         """Attention whose heads' weights are mixed: a key's weight in one head needs its weight in all of them, so the

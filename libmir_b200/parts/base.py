@@ -187,6 +187,12 @@ class Mixer(Part):
     def forward(self, ctx, cache, x: torch.Tensor, residual: torch.Tensor) -> None:
         raise NotImplementedError
 
+    def results(self, ctx, cache, x: torch.Tensor, shape) -> list:
+        """[(32-bit tensor of `shape`, factor), ...]: the mixer's result as a sum that the caller's next kernel forms."""
+        out = ctx.alloc(shape, torch.float32)
+        self.forward(ctx, cache, x, out, overwrite=True)
+        return [(out, 1.0)]
+
 
 class Position(Part):
     def rotation(self):

@@ -22,6 +22,11 @@ A norm before and a norm behind each branch.  The branch writes its result into 
 layer norms one kernel norms that buffer, adds it to the residual and, in the same pass over a token, norms the new
 residual for whoever reads it next (this block's feed-forward or the next block's mixer).
 
+post_norm:  x = norm_1(alpha x + mixer(x));  x = norm_2(alpha x + feed_forward(x))
+Each branch reads the residual itself (cast to the engine's dtype), and the norm stands behind the sum.  The branch leaves
+its result in a 32-bit buffer (or several with a factor each, for a mixer made of branches); one kernel forms the sum,
+norms it, and writes the new residual in 32-bit and, for whoever reads it next, in the engine's dtype.
+
 streams:  the residual is S copies x_1 .. x_S per token (hyper-connections).  For each of the two sublayers, with its
 stored mixing tensors in [S], mix [S, S] and out [S]:  u = sum_s in[s] x_s;  y = sublayer(norm(u));  then all streams
 at once from the old ones, x_t <- sum_s mix[s, t] x_s + out[t] y.  Everything outside the sublayer is 32-bit: the
@@ -68,12 +73,10 @@ class PreNormBlock(Block):
         from .norm import RmsNorm
         mixer, ff = self.mixer, self.feed_forward
         if type(mixer) is not SoftmaxAttention or type(self.mixer_norm) is not RmsNorm or cache is None \
-                or cache.k_pages is None or mixer.w_qkv is None:
+                or cache.k_pages is None or mixer.w_qkv is None or not mixer.plain:
             return None
         if ff is not None and (type(ff) is not SwiGlu or type(self.feed_forward_norm) is not RmsNorm):
             return None
-        if mixer.spec.value_dim != mixer.spec.head_dim or (mixer.spec.window is not None and mixer.spec.keep_first):
-            return None                      # the executor knows neither a value width of its own nor kept first tokens
         rotation = mixer.position.rotation() if mixer.position is not None else (None, 0)
         if rotation is None or self.env.dtype not in (torch.bfloat16, torch.float32):
             return None
@@ -301,6 +304,53 @@ class SandwichBlock(Block):
         return reader.forward(ctx, residual, out=out) if reader is not None else None
 
 
+class PostNormBlock(Block):
+    """x = norm_1(alpha x + mixer(x)), then x = norm_2(alpha x + feed_forward(x)): the norms stand behind the sums."""
+
+    reads_residual_itself = True
+
+    SLOTS = ("mixer_norm", "mixer", "feed_forward_norm", "feed_forward")
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        from .norm import RmsNorm
+        for slot in self.SLOTS:
+            setattr(self, slot, build_part(getattr(spec, slot), env))
+        for norm, branch in ((self.mixer_norm, self.mixer), (self.feed_forward_norm, self.feed_forward)):
+            if branch is not None and type(norm) is not RmsNorm:
+                raise ValueError("the post_norm arrangement takes an RMS norm behind every branch")
+        self.alpha = float(spec.residual_alpha)
+
+    def parts(self):
+        return [(slot, getattr(self, slot)) for slot in self.SLOTS if getattr(self, slot) is not None]
+
+    def cache_requirement(self):
+        return self.mixer.cache_requirement()
+
+    def forward(self, ctx, cache, residual):
+        ctx.upcoming_norm = None             # the products' results go through a sum and its norm, not into the residual
+        ctx.residual_stats = None
+        hand_on = ctx.next_reads_residual
+        shape = tuple(residual.shape)
+        results = self.mixer.results(ctx, cache, ctx.take_rounded(residual), shape)
+        rounded = self._close(ctx, residual, results, self.mixer_norm, self.feed_forward is not None or hand_on)
+        if self.feed_forward is not None:
+            x = rounded if rounded is not None else ctx.cast_residual(residual)
+            result = ctx.alloc(shape, torch.float32)
+            self.feed_forward.forward(ctx, x, result, overwrite=True)
+            rounded = self._close(ctx, residual, [(result, 1.0)], self.feed_forward_norm, hand_on)
+        ctx.rounded_residual = rounded if hand_on else None
+        ctx.residual_stats = None
+
+    def _close(self, ctx, residual, results, norm, read_next):
+        """residual <- norm(alpha * residual + sum of the results); returns its copy in the engine dtype, if there is one."""
+        from .. import kernels
+        rounded = ctx.rounded_buffer(residual) if read_next else None
+        kernels.norm_scaled_sum([tensor for tensor, _ in results], [factor for _, factor in results], residual,
+                                norm.weight, self.alpha, norm.spec.eps, rounded=rounded)
+        return rounded
+
+
 class StreamMix(Part):
     """The three small tensors by which one sublayer reads and writes a residual of several streams."""
 
@@ -389,7 +439,7 @@ class StreamsBlock(Block):
 
 
 ARRANGEMENTS = {"pre_norm": PreNormBlock, "parallel": ParallelBlock, "output_norm": OutputNormBlock,
-                "sandwich": SandwichBlock, "streams": StreamsBlock}
+                "sandwich": SandwichBlock, "post_norm": PostNormBlock, "streams": StreamsBlock}
 
 
 def build_block(layer_spec, env):

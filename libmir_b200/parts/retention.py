@@ -7,6 +7,9 @@ With h the mixer's input, H heads, key width D and value width V:
     o_t     = S_t^T q_t
     y       = o / rms(o) per head * silu(W_g h)   no weight in the norm
     out     = W_o y
+Other forms from the spec: silu of q, k and v enters the recurrence (activated); another factor on k (key_scale); one
+root mean square over all heads together (norm_span "all"); a stored weight behind the norm (norm_weight); a sigmoid
+gate.  These make the mixer known as lightning attention.
 Per request the mixer keeps S of every head (32-bit) in the request's state slot.  The rotation, the decay, the state
 and the recurrence are 32-bit (csrc/retention.cu rotates while it stages the projections' results, or for prompts'
 portions in a kernel of its own into 32-bit scratch, so nothing rotated is rounded to the engine's dtype); the
@@ -38,6 +41,8 @@ class Retention(Mixer):
         s = spec
         if min(s.heads, s.key_dim, s.value_dim) <= 0 or len(s.decays) != s.heads:
             raise ValueError("retention needs heads, key_dim and value_dim above zero and one decay per head")
+        if s.norm_span not in ("head", "all") or s.gate not in ("silu", "sigmoid"):
+            raise ValueError(f"unknown norm span {s.norm_span!r} or gate {s.gate!r}")
         if s.key_dim > 256:
             raise ValueError("the recurrence kernel takes key heads up to 256 wide")
         self.qk_width = s.heads * s.key_dim
@@ -54,7 +59,10 @@ class Retention(Mixer):
             cursor = _pad8(cursor + width)
         self.packed_width = cursor
         self.decays = torch.tensor(list(s.decays), dtype=torch.float32, device=env.device)
-        self.ones = torch.ones(s.value_dim, dtype=torch.float32, device=env.device)
+        # the norm's units: one per head, or all heads as one
+        self.norm_units, self.norm_width = (s.heads, s.value_dim) if s.norm_span == "head" else (1, self.v_width)
+        self.norm = torch.ones(self.norm_width, dtype=torch.float32, device=env.device)
+        self.key_scale = float(s.key_dim) ** -0.5 if s.key_scale is None else float(s.key_scale)
         self.w_in = self.w_o = None
 
     def cache_requirement(self):
@@ -64,7 +72,8 @@ class Retention(Mixer):
     def parameters(self):
         s = self.spec
         matrix = lambda rows, columns: ParamSpec((rows, columns), accept_transposed=False)
-        return {"q": matrix(self.qk_width, s.hidden_size), "k": matrix(self.qk_width, s.hidden_size),
+        table = {"norm": ParamSpec((self.v_width,), init="ones", store="float32")} if s.norm_weight else {}
+        return {**table, "q": matrix(self.qk_width, s.hidden_size), "k": matrix(self.qk_width, s.hidden_size),
                 "v": matrix(self.v_width, s.hidden_size), "g": matrix(self.v_width, s.hidden_size),
                 "o": matrix(s.hidden_size, self.v_width)}
 
@@ -76,9 +85,11 @@ class Retention(Mixer):
             w_in[first:first + tensors[name].shape[0]] = tensors[name]
         self.w_in = w_in
         self.w_o = tensors["o"].contiguous()
+        if s.norm_weight:
+            self.norm = tensors["norm"].contiguous()
 
     def weight_bytes(self):
-        return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o))
+        return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o, self.norm))
 
     def forward(self, ctx, cache, x, residual, overwrite=False):
         """residual += W_o y (or residual = W_o y with `overwrite`, for an arrangement that norms the result)."""
@@ -94,10 +105,11 @@ class Retention(Mixer):
             (kernels.retention_prepared_floats(tokens, s.heads, s.key_dim),), torch.float32)
         kernels.retention_scan(view("q", self.qk_width), view("k", self.qk_width), view("v", self.v_width),
                                self.position.table if self.position is not None else None, self.decays,
-                               float(s.key_dim) ** -0.5, state, ctx.query_starts, ctx.state_slots, ctx.positions, read,
-                               s.heads, s.key_dim, s.value_dim, prepared=prepared)
+                               self.key_scale, state, ctx.query_starts, ctx.state_slots, ctx.positions, read,
+                               s.heads, s.key_dim, s.value_dim, prepared=prepared, activated=s.activated)
         mixed = ctx.alloc((tokens, self.v_width), self.env.dtype)
-        kernels.gated_head_norm(read, view("g", self.v_width), self.ones, mixed, s.heads, s.value_dim, s.norm_eps, False)
+        kernels.gated_head_norm(read, view("g", self.v_width), self.norm, mixed, self.norm_units, self.norm_width,
+                                s.norm_eps, s.gate == "sigmoid")
         if overwrite:
             kernels.linear(mixed, self.w_o, residual, alloc=ctx.alloc)
         else:
