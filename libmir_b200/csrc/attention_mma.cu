@@ -83,7 +83,7 @@ __device__ __forceinline__ float quad_sum(float v) {
 // instruction are GROUP consecutive keys; when the page size is a multiple of GROUP they lie in one page
 // and the block table is read once for all of them (the same address for every lane).
 template <int D, int ROWS, int THREADS>
-__device__ __forceinline__ void load_tile(bf16* k_dst, bf16* v_dst, const bf16* __restrict__ k_pages,
+__device__ __forceinline__ void load_tile_of_equal_widths(bf16* k_dst, bf16* v_dst, const bf16* __restrict__ k_pages,
                                           const bf16* __restrict__ v_pages, const int* __restrict__ table,
                                           int page_size, int kv_heads, int kv_head, int first_key, int limit,
                                           int thread) {
@@ -126,6 +126,66 @@ __device__ __forceinline__ void load_tile(bf16* k_dst, bf16* v_dst, const bf16* 
     }
     cp_async16(smem_u32(k_dst + r * STRIDE + piece * 8), k_pages + offset, valid);
     cp_async16(smem_u32(v_dst + r * STRIDE + piece * 8), v_pages + offset, valid);
+  }
+}
+
+// One of the two tensors alone, its heads D wide.
+template <int D, int ROWS, int THREADS>
+__device__ __forceinline__ void load_rows(bf16* dst, const bf16* __restrict__ pages, const int* __restrict__ table,
+                                          int page_size, int kv_heads, int kv_head, int first_key, int limit,
+                                          int thread) {
+  constexpr int STRIDE = D + 8;
+  constexpr int CHUNKS = D / 8;                    // 16-byte pieces per row
+  constexpr int GROUP = THREADS / CHUNKS;          // rows per instruction
+  static_assert(ROWS % GROUP == 0, "tile rows must be a multiple of the rows one instruction copies");
+  const int sub = thread / CHUNKS, piece = thread % CHUNKS;
+  if (page_size % ROWS == 0 && first_key % ROWS == 0) {
+    // the whole tile lies in one page: one table read, then constant strides
+    const int block = first_key / page_size;
+    const int entry = first_key < limit ? table[block] : -1;
+    const int page = entry < 0 ? 0 : entry;
+    const size_t row_stride = (size_t)kv_heads * D;
+    const size_t base = ((size_t)page * page_size + (first_key - block * page_size)) * row_stride + (size_t)kv_head * D +
+                        piece * 8;
+#pragma unroll
+    for (int i = 0; i < ROWS / GROUP; ++i) {
+      const int r = i * GROUP + sub;
+      const bool valid = entry >= 0 && first_key + r < limit;
+      const size_t offset = valid ? base + r * row_stride : 0;
+      cp_async16(smem_u32(dst + r * STRIDE + piece * 8), pages + offset, valid);
+    }
+    return;
+  }
+  const bool one_page = page_size % GROUP == 0 && first_key % GROUP == 0;
+#pragma unroll
+  for (int i = 0; i < ROWS / GROUP; ++i) {
+    const int r = i * GROUP + sub;
+    const int key = first_key + r;
+    bool valid = key < limit;
+    size_t offset = 0;
+    if (valid) {
+      const int lookup_key = one_page ? first_key + i * GROUP : key;
+      const int block = lookup_key / page_size;
+      const int page = table[block];
+      valid = page >= 0;
+      if (valid) offset = (((size_t)page * page_size + (key - block * page_size)) * kv_heads + kv_head) * D + piece * 8;
+    }
+    cp_async16(smem_u32(dst + r * STRIDE + piece * 8), pages + offset, valid);
+  }
+}
+
+// Keys D and values DV wide.
+template <int D, int DV, int ROWS, int THREADS>
+__device__ __forceinline__ void load_tile(bf16* k_dst, bf16* v_dst, const bf16* __restrict__ k_pages,
+                                          const bf16* __restrict__ v_pages, const int* __restrict__ table,
+                                          int page_size, int kv_heads, int kv_head, int first_key, int limit,
+                                          int thread) {
+  if constexpr (D == DV) {
+    load_tile_of_equal_widths<D, ROWS, THREADS>(k_dst, v_dst, k_pages, v_pages, table, page_size, kv_heads, kv_head,
+                                                first_key, limit, thread);
+  } else {
+    load_rows<D, ROWS, THREADS>(k_dst, k_pages, table, page_size, kv_heads, kv_head, first_key, limit, thread);
+    load_rows<DV, ROWS, THREADS>(v_dst, v_pages, table, page_size, kv_heads, kv_head, first_key, limit, thread);
   }
 }
 
@@ -226,9 +286,9 @@ constexpr int kDecodeMaxTiles = kDecodeMaxPartition / (kDecodeWarps * kDecodeTil
 
 // One CTA: one request, one kv head (up to 8 of its query heads), one partition of the keys.
 // Per 16-key tile a warp computes S = Q K^T (heads on the M side, 8 real rows), the softmax update of its
-// 8 heads, and O^T += V^T P^T (head_dim on the M side, heads on the N side: the padding rows cost nothing
+// 8 heads, and O^T += V^T P^T (the value's width DV on the M side, heads on the N side: the padding rows cost nothing
 // here, and P^T in the layout the product wants is exactly the layout S came out in).
-template <int D, int kDecodeStages, bool SCORED>
+template <int D, int DV, int kDecodeStages, bool SCORED>
 __global__ void __launch_bounds__(kDecodeWarps * 32)
 decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16* __restrict__ k_pages,
                         const bf16* __restrict__ v_pages, const int* __restrict__ block_table, int table_width,
@@ -236,8 +296,8 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
                         int window, int partition, int num_partitions, int part_slow, float* __restrict__ partial_o,
                         float* __restrict__ partial_ml, bf16* __restrict__ out, int keep_first,
                         int* __restrict__ virtual_positions, AttentionExtras extras) {
-  constexpr int STRIDE = D + 8;
-  constexpr int TILE_ELEMS = kDecodeTile * STRIDE;
+  constexpr int V_STRIDE = DV + 8;
+  constexpr int K_ELEMS = kDecodeTile * (D + 8), STAGE_ELEMS = K_ELEMS + kDecodeTile * V_STRIDE;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int quad = lane & 3, group_row = lane >> 2;
@@ -284,8 +344,8 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
   auto true_key = [&](int n) { return n < kept_tiles_end ? n : n + shift; };
   auto true_limit = [&](int n) { return n < kept_tiles_end ? kept_end : min(context, part_end + shift); };
 
-  // this warp's buffers: [stage][K | V][16 rows][STRIDE]
-  bf16* stage_base = reinterpret_cast<bf16*>(smem_raw) + (size_t)warp * kDecodeStages * 2 * TILE_ELEMS;
+  // this warp's buffers: [stage][16 rows of K, 16 rows of V]
+  bf16* stage_base = reinterpret_cast<bf16*>(smem_raw) + (size_t)warp * kDecodeStages * STAGE_ELEMS;
   const int* table = block_table + (size_t)row * table_width;
   const int stride_keys = kDecodeWarps * kDecodeTile;
   const int my_begin = begin + warp * kDecodeTile;
@@ -298,8 +358,8 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
 #pragma unroll
   for (int j = 0; j < kDecodeStages - 1; ++j) {
     if (j < my_tiles) {
-      bf16* dst = stage_base + j * 2 * TILE_ELEMS;
-      load_tile<D, kDecodeTile, 32>(dst, dst + TILE_ELEMS, k_pages, v_pages, table, page_size, kv_heads, kv_head,
+      bf16* dst = stage_base + j * STAGE_ELEMS;
+      load_tile<D, DV, kDecodeTile, 32>(dst, dst + K_ELEMS, k_pages, v_pages, table, page_size, kv_heads, kv_head,
                                     true_key(my_begin + j * stride_keys), true_limit(my_begin + j * stride_keys), lane);
     }
     cp_async_commit();
@@ -321,9 +381,9 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
     }
   }
 
-  float ot[D / 16][4];                                         // O^T: [d = mt*16 + lane/4 (+8)][head = quad*2 (+1)]
+  float ot[DV / 16][4];                                        // O^T: [d = mt*16 + lane/4 (+8)][head = quad*2 (+1)]
 #pragma unroll
-  for (int mt = 0; mt < D / 16; ++mt) ot[mt][0] = ot[mt][1] = ot[mt][2] = ot[mt][3] = 0.0f;
+  for (int mt = 0; mt < DV / 16; ++mt) ot[mt][0] = ot[mt][1] = ot[mt][2] = ot[mt][3] = 0.0f;
   float m = -INFINITY, l = 0.0f;                               // of head lane/4 (l: this lane's share)
 
 #pragma unroll
@@ -331,8 +391,8 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
     if (j >= my_tiles) break;
     constexpr int kAhead = kDecodeStages - 1;
     if (j + kAhead < my_tiles) {
-      bf16* dst = stage_base + ((j + kAhead) % kDecodeStages) * 2 * TILE_ELEMS;
-      load_tile<D, kDecodeTile, 32>(dst, dst + TILE_ELEMS, k_pages, v_pages, table, page_size, kv_heads, kv_head,
+      bf16* dst = stage_base + ((j + kAhead) % kDecodeStages) * STAGE_ELEMS;
+      load_tile<D, DV, kDecodeTile, 32>(dst, dst + K_ELEMS, k_pages, v_pages, table, page_size, kv_heads, kv_head,
                                     true_key(my_begin + (j + kAhead) * stride_keys),
                                     true_limit(my_begin + (j + kAhead) * stride_keys), lane);
     }
@@ -341,8 +401,8 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
     __syncwarp();
     const int tile = true_key(my_begin + j * stride_keys);     // true keys from here on
     const bool kept_tile = my_begin + j * stride_keys < kept_tiles_end;
-    const bf16* k_tile = stage_base + (j % kDecodeStages) * 2 * TILE_ELEMS;
-    const bf16* v_tile = k_tile + TILE_ELEMS;
+    const bf16* k_tile = stage_base + (j % kDecodeStages) * STAGE_ELEMS;
+    const bf16* v_tile = k_tile + K_ELEMS;
     float s[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
     scores<D, 2>(s, qa, k_tile, lane);
     float v00 = s[0][0] * scale_log2, v01 = s[0][1] * scale_log2, v10 = s[1][0] * scale_log2, v11 = s[1][1] * scale_log2;
@@ -381,7 +441,7 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
       const float corr_a = __shfl_sync(0xffffffffu, corr, quad * 8);        // head quad*2   lives in lanes 8*quad..
       const float corr_b = __shfl_sync(0xffffffffu, corr, quad * 8 + 4);    // head quad*2+1
 #pragma unroll
-      for (int mt = 0; mt < D / 16; ++mt) {
+      for (int mt = 0; mt < DV / 16; ++mt) {
         ot[mt][0] *= corr_a;
         ot[mt][1] *= corr_b;
         ot[mt][2] *= corr_a;
@@ -391,9 +451,9 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
     const uint32_t pb0 = pack_bf16(v00, v01), pb1 = pack_bf16(v10, v11);   // P^T: keys 0..7 and 8..15 of the tile
     {
       const int mat = lane >> 3, rowin = lane & 7;
-      const bf16* base = v_tile + ((mat >> 1) * 8 + rowin) * STRIDE + (mat & 1) * 8;
+      const bf16* base = v_tile + ((mat >> 1) * 8 + rowin) * V_STRIDE + (mat & 1) * 8;
 #pragma unroll
-      for (int mt = 0; mt < D / 16; ++mt) {
+      for (int mt = 0; mt < DV / 16; ++mt) {
         uint32_t a[4];
         ldmatrix_x4_trans(a, smem_u32(base + mt * 16));
         mma_bf16(ot[mt], a, pb0, pb1);
@@ -406,19 +466,19 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
   __syncthreads();                                            // every warp is done with its pipeline buffers
 
   // combine the 4 warps through shared memory
-  float* o_sm = reinterpret_cast<float*>(smem_raw);           // [warps][8 heads][D]
-  float* m_sm = o_sm + kDecodeWarps * kDecodeHeads * D;       // [warps][8]
+  float* o_sm = reinterpret_cast<float*>(smem_raw);           // [warps][8 heads][DV]
+  float* m_sm = o_sm + kDecodeWarps * kDecodeHeads * DV;       // [warps][8]
   float* l_sm = m_sm + kDecodeWarps * kDecodeHeads;
   {
-    float* mine = o_sm + (size_t)warp * kDecodeHeads * D;
+    float* mine = o_sm + (size_t)warp * kDecodeHeads * DV;
     const int head_a = quad * 2, head_b = head_a + 1;
 #pragma unroll
-    for (int mt = 0; mt < D / 16; ++mt) {
+    for (int mt = 0; mt < DV / 16; ++mt) {
       const int d = mt * 16 + group_row;
-      mine[head_a * D + d] = ot[mt][0];
-      mine[head_b * D + d] = ot[mt][1];
-      mine[head_a * D + d + 8] = ot[mt][2];
-      mine[head_b * D + d + 8] = ot[mt][3];
+      mine[head_a * DV + d] = ot[mt][0];
+      mine[head_b * DV + d] = ot[mt][1];
+      mine[head_a * DV + d + 8] = ot[mt][2];
+      mine[head_b * DV + d + 8] = ot[mt][3];
     }
     if (quad == 0) {
       m_sm[warp * kDecodeHeads + group_row] = m;
@@ -426,8 +486,8 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
     }
   }
   __syncthreads();
-  for (int index = threadIdx.x; index < valid_rows * D; index += kDecodeWarps * 32) {
-    const int r = index / D, d = index % D;
+  for (int index = threadIdx.x; index < valid_rows * DV; index += kDecodeWarps * 32) {
+    const int r = index / DV, d = index % DV;
     float top = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kDecodeWarps; ++w) top = fmaxf(top, m_sm[w * kDecodeHeads + r]);
@@ -436,17 +496,17 @@ decode_attention_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16*
 #pragma unroll
       for (int w = 0; w < kDecodeWarps; ++w) {
         const float weight = exp2f(m_sm[w * kDecodeHeads + r] - top);
-        acc += o_sm[((size_t)w * kDecodeHeads + r) * D + d] * weight;
+        acc += o_sm[((size_t)w * kDecodeHeads + r) * DV + d] * weight;
         denom += l_sm[w * kDecodeHeads + r] * weight;
       }
     }
     const size_t head = (size_t)row * heads + head0 + r;
     if (num_partitions == 1) {
       if (denom > 0.0f) denom += sink_term(extras, head0 + r, top);
-      out[head * D + d] = __float2bfloat16_rn(
-          denom > 0.0f ? acc / denom * gate_factor(extras, row, (size_t)(head0 + r) * D + d) : 0.0f);
+      out[head * DV + d] = __float2bfloat16_rn(
+          denom > 0.0f ? acc / denom * gate_factor(extras, row, (size_t)(head0 + r) * DV + d) : 0.0f);
     } else {
-      partial_o[(head * num_partitions + part) * D + d] = acc;
+      partial_o[(head * num_partitions + part) * DV + d] = acc;
       if (d == 0) {
         partial_ml[(head * num_partitions + part) * 2] = top;
         partial_ml[(head * num_partitions + part) * 2 + 1] = denom;
@@ -543,7 +603,7 @@ __global__ void __launch_bounds__(kMergeWarps * 32)
 decode_merge_few_kernel(const float* __restrict__ partial_o, const float* __restrict__ partial_ml,
                         const int* __restrict__ positions, int heads, int window, int partition, int num_partitions,
                         bf16* __restrict__ out, AttentionExtras extras) {
-  constexpr int PER = D / 32;                                  // elements per lane: 4 or 2
+  constexpr int PER = D / 32;                                  // elements per lane: 4, 2 or 1
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.x * kMergeWarps + warp, row = blockIdx.y;
   grid_launch_dependents();
@@ -579,10 +639,12 @@ decode_merge_few_kernel(const float* __restrict__ partial_o, const float* __rest
     if (live) {
       if (PER == 4) {
         const float4 v = *reinterpret_cast<const float4*>(o + (size_t)p * D);
-        piece[i][0] = v.x; piece[i][1] = v.y; piece[i][2] = v.z; piece[i][PER - 1] = v.w;
-      } else {
+        piece[i][0] = v.x; piece[i][PER / 4] = v.y; piece[i][PER / 2] = v.z; piece[i][PER - 1] = v.w;
+      } else if (PER == 2) {
         const float2 v = *reinterpret_cast<const float2*>(o + (size_t)p * D);
-        piece[i][0] = v.x; piece[i][1] = v.y;
+        piece[i][0] = v.x; piece[i][PER - 1] = v.y;
+      } else {
+        piece[i][0] = o[(size_t)p * D];
       }
     }
   }
@@ -603,9 +665,13 @@ decode_merge_few_kernel(const float* __restrict__ partial_o, const float* __rest
 #pragma unroll
   for (int j = 0; j < PER; ++j)
     acc[j] = denom > 0.0f ? acc[j] / denom * gate_factor(extras, row, (size_t)head * D + PER * lane + j) : 0.0f;
+  if (PER == 1) {
+    dst[0] = __float2bfloat16_rn(acc[0]);
+  } else {
 #pragma unroll
-  for (int j = 0; j < PER; j += 2)
-    *reinterpret_cast<__nv_bfloat162*>(dst + j) = __floats2bfloat162_rn(acc[j], acc[j + 1]);
+    for (int j = 0; j < PER; j += 2)
+      *reinterpret_cast<__nv_bfloat162*>(dst + j) = __floats2bfloat162_rn(acc[j], acc[j + PER / 2 - (PER == 4)]);
+  }
   if (threadIdx.x == 0) MIR_TRACE_POINT(merge, 2);
 }
 
@@ -614,17 +680,16 @@ constexpr int kPrefillWarps = 4;
 constexpr int kQueryTile = kPrefillWarps * 16;     // 64 tokens per CTA
 constexpr int kKeyTile = 64;
 
-template <int D, bool SCORED>
+template <int D, int DV, bool SCORED>
 __global__ void __launch_bounds__(kPrefillWarps * 32, 3)
 prefill_attention_kernel(const bf16* __restrict__ q, size_t q_stride, bf16* __restrict__ out,
                          const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                          const int* __restrict__ block_table, int table_width, const int* __restrict__ query_starts,
                          const int* __restrict__ context_lens, int num_rows, int page_size, int heads, int kv_heads,
                          float scale_log2, int window, int keep_first, AttentionExtras extras) {
-  constexpr int STRIDE = D + 8;
-  constexpr int TILE_ELEMS = kKeyTile * STRIDE;
+  constexpr int K_ELEMS = kKeyTile * (D + 8), STAGE_ELEMS = K_ELEMS + kKeyTile * (DV + 8);
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  bf16* buffers = reinterpret_cast<bf16*>(smem_raw);          // [stage][K | V][64][STRIDE]
+  bf16* buffers = reinterpret_cast<bf16*>(smem_raw);          // [stage][64 rows of K, 64 rows of V]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.x;                                // the fast index: all heads of the longest tile start first
   const int kv_head = head / (heads / kv_heads);
@@ -668,9 +733,9 @@ prefill_attention_kernel(const bf16* __restrict__ q, size_t q_stride, bf16* __re
       qa[ks][3] = valid1 ? *reinterpret_cast<const uint32_t*>(q_row1 + ks * 16 + 8 + c) : 0u;
     }
   }
-  float o[D / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int nt = 0; nt < D / 8; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.0f;
+  for (int nt = 0; nt < DV / 8; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.0f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
 
   const int first_key = (window > 0 && first_position + 1 > window) ? first_position + 1 - window : 0;
@@ -688,7 +753,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, size_t q_stride, bf16* __re
   auto tile_key = [&](int i) { return i < kept_tiles ? i * kKeyTile : key_begin + (i - kept_tiles) * kKeyTile; };
   auto tile_limit = [&](int i) { return i < kept_tiles ? kept_keys : key_end; };
 
-  load_tile<D, kKeyTile, kPrefillWarps * 32>(buffers, buffers + TILE_ELEMS, k_pages, v_pages, table, page_size, kv_heads, kv_head,
+  load_tile<D, DV, kKeyTile, kPrefillWarps * 32>(buffers, buffers + K_ELEMS, k_pages, v_pages, table, page_size, kv_heads, kv_head,
                          tile_key(0), tile_limit(0), threadIdx.x);
   cp_async_commit();
   int stage = 0;
@@ -696,15 +761,15 @@ prefill_attention_kernel(const bf16* __restrict__ q, size_t q_stride, bf16* __re
     const int key0 = tile_key(tile);
     const bool kept_tile = tile < kept_tiles;
     if (tile + 1 < total_tiles) {
-      bf16* dst = buffers + (stage ^ 1) * 2 * TILE_ELEMS;
-      load_tile<D, kKeyTile, kPrefillWarps * 32>(dst, dst + TILE_ELEMS, k_pages, v_pages, table, page_size, kv_heads, kv_head,
+      bf16* dst = buffers + (stage ^ 1) * STAGE_ELEMS;
+      load_tile<D, DV, kKeyTile, kPrefillWarps * 32>(dst, dst + K_ELEMS, k_pages, v_pages, table, page_size, kv_heads, kv_head,
                              tile_key(tile + 1), tile_limit(tile + 1), threadIdx.x);
     }
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
-    const bf16* k_tile = buffers + stage * 2 * TILE_ELEMS;
-    const bf16* v_tile = k_tile + TILE_ELEMS;
+    const bf16* k_tile = buffers + stage * STAGE_ELEMS;
+    const bf16* v_tile = k_tile + K_ELEMS;
     // this warp needs the tile only if some key of it is visible to some of its rows
     // (a tile of the window's run may also hold kept keys that lie before this warp's own windows)
     const bool holds_kept = kept_tile || (window > 0 && key0 < keep_first);
@@ -732,8 +797,8 @@ prefill_attention_kernel(const bf16* __restrict__ q, size_t q_stride, bf16* __re
           s[nt][e] = visible ? value : -INFINITY;
         }
       uint32_t pa[NT / 2][4];
-      softmax<D, NT>(s, m, l, o, pa);
-      values<D, NT>(o, pa, v_tile, lane);
+      softmax<DV, NT>(s, m, l, o, pa);
+      values<DV, NT>(o, pa, v_tile, lane);
     }
     __syncthreads();
   }
@@ -746,18 +811,18 @@ prefill_attention_kernel(const bf16* __restrict__ q, size_t q_stride, bf16* __re
   }
   const float inv0 = l[0] > 0.0f ? 1.0f / l[0] : 0.0f, inv1 = l[1] > 0.0f ? 1.0f / l[1] : 0.0f;
   const size_t token0 = (size_t)(q_begin + local0 + local_r0), token1 = (size_t)(q_begin + local0 + local_r1);
-  bf16* out0 = out + (token0 * heads + head) * D;
-  bf16* out1 = out + (token1 * heads + head) * D;
+  bf16* out0 = out + (token0 * heads + head) * DV;
+  bf16* out1 = out + (token1 * heads + head) * DV;
   if (extras.gate != nullptr) {
 #pragma unroll
-    for (int nt = 0; nt < D / 8; ++nt) {
-      const size_t column = (size_t)head * D + nt * 8 + c;
+    for (int nt = 0; nt < DV / 8; ++nt) {
+      const size_t column = (size_t)head * DV + nt * 8 + c;
       if (valid0) { o[nt][0] *= gate_factor(extras, token0, column); o[nt][1] *= gate_factor(extras, token0, column + 1); }
       if (valid1) { o[nt][2] *= gate_factor(extras, token1, column); o[nt][3] *= gate_factor(extras, token1, column + 1); }
     }
   }
 #pragma unroll
-  for (int nt = 0; nt < D / 8; ++nt) {
+  for (int nt = 0; nt < DV / 8; ++nt) {
     if (valid0) *reinterpret_cast<uint32_t*>(out0 + nt * 8 + c) = pack_bf16(o[nt][0] * inv0, o[nt][1] * inv0);
     if (valid1) *reinterpret_cast<uint32_t*>(out1 + nt * 8 + c) = pack_bf16(o[nt][2] * inv1, o[nt][3] * inv1);
   }
@@ -788,45 +853,47 @@ int launch_merge(const float* partial_o, const float* partial_ml, const int* pos
                     partial_o, partial_ml, positions, heads, window, partition, num_partitions, out, extras);
 }
 
-template <int D, int STAGES>
+template <int D, int DV, int STAGES>
 int launch_decode_staged(const bf16* q, size_t q_stride, bf16* out, const bf16* k_pages, const bf16* v_pages,
                          const int* block_table, int table_width, const int* positions, int rows, int page_size,
                          int heads, int kv_heads, float scale, int window, int partition, int num_partitions,
                          float* partial_o, float* partial_ml, cudaStream_t stream, int keep_first = 0,
                          int* virtual_positions = nullptr, AttentionExtras extras = {}) {
-  const size_t pipeline = (size_t)kDecodeWarps * STAGES * 2 * kDecodeTile * (D + 8) * sizeof(bf16);
-  const size_t combine = (size_t)kDecodeWarps * kDecodeHeads * (D + 2) * sizeof(float);
+  const size_t pipeline = (size_t)kDecodeWarps * STAGES * kDecodeTile * (D + DV + 16) * sizeof(bf16);
+  const size_t combine = (size_t)kDecodeWarps * kDecodeHeads * (DV + 2) * sizeof(float);
   const size_t smem = pipeline > combine ? pipeline : combine;
   static bool smem_set = false;                               // per head size and depth: this function is a template
   static bool smem_set_scored = false;
-  const bool scored = extras.softcap > 0.0f || extras.rel_bias != nullptr;
-  int status = scored ? set_smem(decode_attention_kernel<D, STAGES, true>, smem, "decode_attention", smem_set_scored)
-                      : set_smem(decode_attention_kernel<D, STAGES, false>, smem, "decode_attention", smem_set);
+  // (value heads of a width of their own run the form with modified scores, which a plain score passes unchanged)
+  constexpr bool kOnlyScored = D != DV;
+  const bool scored = kOnlyScored || scores_modified(extras);
+  int status = scored ? set_smem(decode_attention_kernel<D, DV, STAGES, true>, smem, "decode_attention", smem_set_scored)
+                      : set_smem(decode_attention_kernel<D, DV, STAGES, kOnlyScored>, smem, "decode_attention", smem_set);
   if (status != MIR_OK) return status;
   const int group = heads / kv_heads;
   const int units = kv_heads * ((group + kDecodeHeads - 1) / kDecodeHeads);
   const dim3 grid = rows <= 4 ? dim3(rows, units, num_partitions) : dim3(num_partitions, units, rows);
   status = scored
-      ? mir_launch_with(mir_pdl_for_streaming(), "decode_attention", decode_attention_kernel<D, STAGES, true>, grid,
+      ? mir_launch_with(mir_pdl_for_streaming(), "decode_attention", decode_attention_kernel<D, DV, STAGES, true>, grid,
                         dim3(kDecodeWarps * 32), smem, stream, 0, q, q_stride, k_pages, v_pages, block_table,
                         table_width, positions, page_size, heads, kv_heads, scale * 1.4426950408889634f, window,
                         partition, num_partitions, rows <= 4 ? 1 : 0, partial_o, partial_ml, out, keep_first,
                         virtual_positions, extras)
-      : mir_launch_with(mir_pdl_for_streaming(), "decode_attention", decode_attention_kernel<D, STAGES, false>, grid,
+      : mir_launch_with(mir_pdl_for_streaming(), "decode_attention", decode_attention_kernel<D, DV, STAGES, kOnlyScored>, grid,
                         dim3(kDecodeWarps * 32), smem, stream, 0, q, q_stride, k_pages, v_pages, block_table,
                         table_width, positions, page_size, heads, kv_heads, scale * 1.4426950408889634f, window,
                         partition, num_partitions, rows <= 4 ? 1 : 0, partial_o, partial_ml, out, keep_first,
                         virtual_positions, extras);
   if (status != MIR_OK || num_partitions == 1) return status;
   if (keep_first > 0 && window > 0)      // the partitions were counted in the kernel's own numbering of the visible keys
-    return launch_merge<D>(partial_o, partial_ml, virtual_positions, rows, heads, 0, partition, num_partitions, out, stream,
+    return launch_merge<DV>(partial_o, partial_ml, virtual_positions, rows, heads, 0, partition, num_partitions, out, stream,
                            extras);
-  return launch_merge<D>(partial_o, partial_ml, positions, rows, heads, window, partition, num_partitions, out, stream,
+  return launch_merge<DV>(partial_o, partial_ml, positions, rows, heads, window, partition, num_partitions, out, stream,
                          extras);
 }
 
 long long g_deep_ring_ctas = 1536;                              // up to this many CTAs run three tiles in flight per warp
-template <int D>
+template <int D, int DV>
 int launch_decode(const bf16* q, size_t q_stride, bf16* out, const bf16* k_pages, const bf16* v_pages,
                   const int* block_table, int table_width, const int* positions, int rows, int page_size, int heads,
                   int kv_heads, float scale, int window, int partition, int num_partitions, float* partial_o,
@@ -835,25 +902,26 @@ int launch_decode(const bf16* q, size_t q_stride, bf16* out, const bf16* k_pages
   const int group = heads / kv_heads;
   const long long ctas = (long long)num_partitions * kv_heads * ((group + kDecodeHeads - 1) / kDecodeHeads) * rows;
   if (ctas <= g_deep_ring_ctas)
-    return launch_decode_staged<D, 3>(q, q_stride, out, k_pages, v_pages, block_table, table_width, positions, rows,
+    return launch_decode_staged<D, DV, 3>(q, q_stride, out, k_pages, v_pages, block_table, table_width, positions, rows,
                                       page_size, heads, kv_heads, scale, window, partition, num_partitions, partial_o,
                                       partial_ml, stream, keep_first, virtual_positions, extras);
-  return launch_decode_staged<D, 2>(q, q_stride, out, k_pages, v_pages, block_table, table_width, positions, rows,
+  return launch_decode_staged<D, DV, 2>(q, q_stride, out, k_pages, v_pages, block_table, table_width, positions, rows,
                                     page_size, heads, kv_heads, scale, window, partition, num_partitions, partial_o,
                                     partial_ml, stream, keep_first, virtual_positions, extras);
 }
 
-template <int D>
+template <int D, int DV>
 int launch_prefill(const bf16* q, size_t q_stride, bf16* out, const bf16* k_pages, const bf16* v_pages,
                    const int* block_table, int table_width, const int* query_starts, const int* context_lens,
                    int num_rows, int tokens, int page_size, int heads, int kv_heads, float scale, int window,
                    int keep_first, cudaStream_t stream, AttentionExtras extras = {}) {
-  const size_t smem = (size_t)2 * 2 * kKeyTile * (D + 8) * sizeof(bf16);
+  const size_t smem = (size_t)2 * kKeyTile * (D + DV + 16) * sizeof(bf16);
   static bool smem_set = false;
   static bool smem_set_scored = false;
-  const bool scored = extras.softcap > 0.0f || extras.rel_bias != nullptr;
-  int status = scored ? set_smem(prefill_attention_kernel<D, true>, smem, "prefill_attention", smem_set_scored)
-                      : set_smem(prefill_attention_kernel<D, false>, smem, "prefill_attention", smem_set);
+  constexpr bool kOnlyScored = D != DV;
+  const bool scored = kOnlyScored || scores_modified(extras);
+  int status = scored ? set_smem(prefill_attention_kernel<D, DV, true>, smem, "prefill_attention", smem_set_scored)
+                      : set_smem(prefill_attention_kernel<D, DV, kOnlyScored>, smem, "prefill_attention", smem_set);
   if (status != MIR_OK) return status;
   const int tiles = (tokens + kQueryTile - 1) / kQueryTile + num_rows;   // an upper bound; spare CTAs return
   if (tiles > 65535) {
@@ -861,15 +929,28 @@ int launch_prefill(const bf16* q, size_t q_stride, bf16* out, const bf16* k_page
     return MIR_BAD_ARGUMENT;
   }
   if (scored)
-    return mir_launch("prefill_attention", prefill_attention_kernel<D, true>, dim3(heads, tiles), dim3(kPrefillWarps * 32),
+    return mir_launch("prefill_attention", prefill_attention_kernel<D, DV, true>, dim3(heads, tiles), dim3(kPrefillWarps * 32),
                       smem, stream, 0, q, q_stride, out, k_pages, v_pages, block_table, table_width, query_starts,
                       context_lens, num_rows, page_size, heads, kv_heads, scale * 1.4426950408889634f, window,
                       keep_first, extras);
-  return mir_launch("prefill_attention", prefill_attention_kernel<D, false>, dim3(heads, tiles), dim3(kPrefillWarps * 32),
+  return mir_launch("prefill_attention", prefill_attention_kernel<D, DV, kOnlyScored>, dim3(heads, tiles), dim3(kPrefillWarps * 32),
                     smem, stream, 0, q, q_stride, out, k_pages, v_pages, block_table, table_width, query_starts,
                     context_lens, num_rows, page_size, heads, kv_heads, scale * 1.4426950408889634f, window,
                     keep_first, extras);
 }
+
+// The value's width of a call (0: the key's).
+int value_width(const AttentionExtras& extras, int head_dim) { return extras.value_dim > 0 ? extras.value_dim : head_dim; }
+bool bad_value_width(const char* what, int value_dim) {
+  if (value_dim == 32 || value_dim == 64 || value_dim == 128) return false;
+  mir_set_error("%s: value heads of %d are not one of 32, 64, 128 (the reference kernel takes the other sizes)", what, value_dim);
+  return true;
+}
+// CALL(D, DV) for the sizes that the tile kernels take.
+#define MIR_FOR_WIDTHS(head_dim, value_dim, CALL)                                  \
+  if ((head_dim) == 64)                                                            \
+    return (value_dim) == 32 ? CALL(64, 32) : ((value_dim) == 64 ? CALL(64, 64) : CALL(64, 128)); \
+  return (value_dim) == 32 ? CALL(128, 32) : ((value_dim) == 64 ? CALL(128, 64) : CALL(128, 128));
 
 bool bad_common(const char* what, int heads, int kv_heads, int head_dim, int page_size, int table_width, int window) {
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || page_size <= 0 || table_width <= 0 || window < 0) {
@@ -908,11 +989,14 @@ MIR_EXPORT int mir_decode_merge_gated_bf16(const float* partial_o, const float* 
                                            const void* gate, long long gate_stride, int gate_head_width) {
   const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_head_width};
   if (rows <= 0 || rows > 65535 || heads <= 0 || partition <= 0 || num_partitions <= 0 || window < 0 ||
-      (head_dim != 64 && head_dim != 128) || partial_o == nullptr || partial_ml == nullptr) {
+      (head_dim != 32 && head_dim != 64 && head_dim != 128) || partial_o == nullptr || partial_ml == nullptr) {
     mir_set_error("decode_merge: bad sizes (rows %d, heads %d, head_dim %d, partition %d, partitions %d)", rows, heads,
                   head_dim, partition, num_partitions);
     return MIR_BAD_ARGUMENT;
   }
+  if (head_dim == 32)
+    return launch_merge<32>(partial_o, partial_ml, positions, rows, heads, window, partition, num_partitions, (bf16*)out,
+                            stream, extras);
   if (head_dim == 64)
     return launch_merge<64>(partial_o, partial_ml, positions, rows, heads, window, partition, num_partitions, (bf16*)out,
                             stream, extras);
@@ -957,10 +1041,10 @@ MIR_EXPORT int mir_decode_attention_bf16(const void* q, long long q_stride, void
   float* partial_o = scratch;
   float* partial_ml = scratch ? scratch + (size_t)rows * heads * num_partitions * head_dim : nullptr;
   if (head_dim == 64)
-    return launch_decode<64>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,
+    return launch_decode<64, 64>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,
                              block_table, table_width, positions, rows, page_size, heads, kv_heads, scale, window,
                              partition, num_partitions, partial_o, partial_ml, stream);
-  return launch_decode<128>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,
+  return launch_decode<128, 128>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,
                             block_table, table_width, positions, rows, page_size, heads, kv_heads, scale, window,
                             partition, num_partitions, partial_o, partial_ml, stream);
 }
@@ -986,22 +1070,21 @@ static int decode_attention_with(const void* q, long long q_stride, void* out, c
     mir_set_error("decode_attention: bad rows %d, partition %d or partition count %d", rows, partition, num_partitions);
     return MIR_BAD_ARGUMENT;
   }
-  const long long need = mir_decode_attention_scratch_floats(rows, heads, head_dim, num_partitions);
+  const int value_dim = value_width(extras, head_dim);
+  if (bad_value_width("decode_attention", value_dim)) return MIR_BAD_ARGUMENT;
+  const long long need = mir_decode_attention_scratch_floats(rows, heads, value_dim, num_partitions);
   if (need < 0 || (need > 0 && (scratch == nullptr || scratch_floats < need))) {
     mir_set_error("decode_attention: scratch of %lld floats is needed, got %lld", need, scratch_floats);
     return MIR_BAD_ARGUMENT;
   }
   float* partial_o = scratch;
-  float* partial_ml = scratch ? scratch + (size_t)rows * heads * num_partitions * head_dim : nullptr;
-  if (head_dim == 64)
-    return launch_decode<64>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,
-                             block_table, table_width, positions, rows, page_size, heads, kv_heads, scale, window,
-                             partition, num_partitions, partial_o, partial_ml, stream, keep_first, virtual_positions,
-                             extras);
-  return launch_decode<128>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,
-                            block_table, table_width, positions, rows, page_size, heads, kv_heads, scale, window,
-                            partition, num_partitions, partial_o, partial_ml, stream, keep_first, virtual_positions,
-                            extras);
+  float* partial_ml = scratch ? scratch + (size_t)rows * heads * num_partitions * value_dim : nullptr;
+#define MIR_DECODE(D, DV)                                                                                             \
+  launch_decode<D, DV>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,      \
+                       block_table, table_width, positions, rows, page_size, heads, kv_heads, scale, window, partition, \
+                       num_partitions, partial_o, partial_ml, stream, keep_first, virtual_positions, extras)
+  MIR_FOR_WIDTHS(head_dim, value_dim, MIR_DECODE)
+#undef MIR_DECODE
 }
 
 MIR_EXPORT int mir_decode_attention_extra_bf16(const void* q, long long q_stride, void* out, const void* k_pages,
@@ -1026,10 +1109,10 @@ MIR_EXPORT int mir_decode_attention_scored_bf16(const void* q, long long q_strid
                                                 int num_partitions, float* scratch, long long scratch_floats,
                                                 cudaStream_t stream, const float* sinks, const void* gate,
                                                 long long gate_stride, int gate_per_head, float softcap,
-                                                const float* rel_bias, int rel_rows) {
+                                                const float* rel_bias, int rel_rows, const float* slopes, int value_dim) {
   if (rel_bias != nullptr && rel_rows <= 0) { mir_set_error("decode_attention: a bias by distance needs rows"); return MIR_BAD_ARGUMENT; }
-  const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_per_head ? head_dim : 0, softcap, rel_bias,
-                               rel_rows, heads};
+  const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_per_head ? (value_dim > 0 ? value_dim : head_dim) : 0, softcap, rel_bias,
+                               rel_rows, heads, slopes, value_dim};
   return decode_attention_with(q, q_stride, out, k_pages, v_pages, block_table, table_width, positions, rows, page_size,
                                heads, kv_heads, head_dim, scale, window, partition, num_partitions, scratch,
                                scratch_floats, stream, 0, nullptr, extras);
@@ -1065,13 +1148,14 @@ static int prefill_attention_with(const void* q, long long q_stride, void* out, 
     mir_set_error("prefill_attention: bad tokens %d, rows %d or heads %d", tokens, num_rows, heads);
     return MIR_BAD_ARGUMENT;
   }
-  if (head_dim == 64)
-    return launch_prefill<64>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,
-                              block_table, table_width, query_starts, context_lens, num_rows, tokens, page_size, heads,
-                              kv_heads, scale, window, keep_first, stream, extras);
-  return launch_prefill<128>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,
-                             block_table, table_width, query_starts, context_lens, num_rows, tokens, page_size, heads,
-                             kv_heads, scale, window, keep_first, stream, extras);
+  const int value_dim = value_width(extras, head_dim);
+  if (bad_value_width("prefill_attention", value_dim)) return MIR_BAD_ARGUMENT;
+#define MIR_PREFILL(D, DV)                                                                                            \
+  launch_prefill<D, DV>((const bf16*)q, (size_t)q_stride, (bf16*)out, (const bf16*)k_pages, (const bf16*)v_pages,     \
+                        block_table, table_width, query_starts, context_lens, num_rows, tokens, page_size, heads,     \
+                        kv_heads, scale, window, keep_first, stream, extras)
+  MIR_FOR_WIDTHS(head_dim, value_dim, MIR_PREFILL)
+#undef MIR_PREFILL
 }
 
 MIR_EXPORT int mir_prefill_attention_extra_bf16(const void* q, long long q_stride, void* out, const void* k_pages,
@@ -1093,10 +1177,10 @@ MIR_EXPORT int mir_prefill_attention_scored_bf16(const void* q, long long q_stri
                                                  int tokens, int page_size, int heads, int kv_heads, int head_dim,
                                                  float scale, int window, cudaStream_t stream, const float* sinks,
                                                  const void* gate, long long gate_stride, int gate_per_head,
-                                                 float softcap, const float* rel_bias, int rel_rows) {
+                                                 float softcap, const float* rel_bias, int rel_rows, const float* slopes, int value_dim) {
   if (rel_bias != nullptr && rel_rows <= 0) { mir_set_error("prefill_attention: a bias by distance needs rows"); return MIR_BAD_ARGUMENT; }
-  const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_per_head ? head_dim : 0, softcap, rel_bias,
-                               rel_rows, heads};
+  const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_per_head ? (value_dim > 0 ? value_dim : head_dim) : 0, softcap, rel_bias,
+                               rel_rows, heads, slopes, value_dim};
   return prefill_attention_with(q, q_stride, out, k_pages, v_pages, block_table, table_width, query_starts, context_lens,
                                 num_rows, tokens, page_size, heads, kv_heads, head_dim, scale, window, 0, stream, extras);
 }

@@ -166,13 +166,14 @@ struct Handoff {
 };
 // SCORED: the scaled score is capped (softcap * tanh(score / softcap)) and gets the head's bias by distance (`bias`,
 // one entry per distance up to bias_last; `distance` is that of this thread's first column, the next column's is one
-// less), in 32-bit; from there on the scores are final and in units of log2 e.
+// less), or `slope` times the distance is taken off it, in 32-bit; from there on the scores are final and in units of log2 e.
 template <bool MASKED, bool SHARED, bool SCORED>
 __device__ __forceinline__ float softmax_tile(uint32_t scores, int first, int low, int high, float scale_log2,
                                               float& reference, float& factor, bool& grow,
                                               uint32_t (&packed)[kCols / 2], float* shared_max, int part, int team,
                                               int stamp_tile, const Handoff& handoff, float& own_factor, bool& alive,
-                                              float softcap, const float* __restrict__ bias, int bias_last, int distance) {
+                                              float softcap, const float* __restrict__ bias, int bias_last, int distance,
+                                              float slope) {
   float v[kCols];
 #pragma unroll
   for (int c0 = 0; c0 < kCols; c0 += 32) tmem_load_32_nowait(scores + first + c0, v + c0);
@@ -190,7 +191,15 @@ __device__ __forceinline__ float softmax_tile(uint32_t scores, int first, int lo
     const float drop = -2.0f * softcap * kLog2e, base = capped ? softcap * kLog2e : 0.0f;
     // the bias: most tiles lie wholly beyond the table's last entry (one value for all columns) or wholly inside it
     const int nearest = distance - (kCols - 1);
-    if (bias == nullptr || nearest >= bias_last) {
+    if (slope != 0.0f) {                                     // a bias that falls linearly: slope * (distance - c) off
+      const float fall = slope * kLog2e;
+      const float lift0 = fmaf(-fall, (float)distance, base);
+#pragma unroll
+      for (int c = 0; c < kCols; ++c) {
+        const float lift = fmaf(fall, (float)c, lift0);
+        v[c] = capped ? fmaf(drop, fast_reciprocal(1.0f + fast_exp2(v[c] * k)), lift) : fmaf(v[c], k, lift);
+      }
+    } else if (bias == nullptr || nearest >= bias_last) {
       const float lift = base + (bias != nullptr ? __ldg(bias + bias_last) * kLog2e : 0.0f);
 #pragma unroll
       for (int c = 0; c < kCols; ++c)
@@ -261,6 +270,9 @@ __device__ __forceinline__ float softmax_tile(uint32_t scores, int first, int lo
   return (sums[0] + sums[1]) + (sums[2] + sums[3]);
 }
 
+__device__ __forceinline__ void tmem_load_piece(uint32_t address, float (&v)[32]) { tmem_load_32(address, v); }
+__device__ __forceinline__ void tmem_load_piece(uint32_t address, float (&v)[16]) { tmem_load_16(address, v); }
+
 // What one work item is: which queries, which keys.
 struct Work {
   bool valid;
@@ -326,7 +338,9 @@ __device__ __forceinline__ int item_of(int k, int cta, int ctas, int items) {
   return k * ctas + ((k & 1) ? ctas - 1 - cta : cta);
 }
 
-template <int kStreams, bool kShared, bool kScored = false>
+// kValueDim: width of a value head, 128 or 64 (then one 64-wide half of the value tiles is loaded and the products with V
+// and the output accumulator are 64 columns wide).
+template <int kStreams, bool kShared, bool kScored = false, int kValueDim = kDim>
 __global__ void __launch_bounds__(threads_for(kStreams), 1)
 tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                             const __grid_constant__ CUtensorMap v_map, const __grid_constant__ CUtensorMap k_tile_map,
@@ -408,7 +422,8 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     const uint32_t box_bytes = (uint32_t)page_size * 128u;
     // lane l loads half (l & 1) of page slot (l >> 1): at most 16 pages of 8 keys, so one round of 32 lanes
     const int slot = lane >> 1, half = lane & 1;
-    const bool loads = lane < 2 * pages_per_tile;
+    const int halves = which ? kValueDim / 64 : 2, width = which ? kValueDim : kDim;
+    const bool loads = lane < 2 * pages_per_tile && half < halves;
     const uint32_t lane_dst = smem_base + (which ? kOffV : kOffK) + (uint32_t)half * kHalf +
                               (uint32_t)(slot * page_size) * 128u;
     const CUtensorMap* map = which ? &v_map : &k_map;
@@ -432,7 +447,7 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
           tma_load_2d(smem_base + kOffQ + kHalf, &q_map, bar(Q_FULL), w.head * kDim + 64, w.q_row0);
         }
       }
-      const int x = w.kv_head * kDim + half * 64;
+      const int x = w.kv_head * width + half * 64;
       const int tiles = w.tiles, key_end = w.key_end, first_visible = w.first_key - page_size;
       auto page_of = [&](int t) {                              // this lane's page of tile t, -1 if nothing of it is seen
         if (!loads || t >= tiles) return -1;
@@ -459,11 +474,11 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         const int first_page = __shfl_sync(0xffffffffu, page, 0);
         const bool in_a_row = first_page >= 0 && __all_sync(0xffffffffu, !loads || page == first_page + slot);
         if (in_a_row) {
-          if (lane == 0) barrier_expect_bytes(full, kTile);
+          if (lane == 0) barrier_expect_bytes(full, (uint32_t)(halves * kHalf));
           __syncwarp();
-          if (lane < 2)
+          if (lane < halves)
             tma_load_2d(tile_dst + (uint32_t)lane * kHalf + (uint32_t)stage * kTile, tile_map, full,
-                        w.kv_head * kDim + lane * 64, first_page << page_shift);
+                        w.kv_head * width + lane * 64, first_page << page_shift);
         } else {
           const unsigned valid = __ballot_sync(0xffffffffu, page >= 0);
           if (lane == 0) barrier_expect_bytes(full, (uint32_t)__popc(valid) * box_bytes);
@@ -483,7 +498,7 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     // ------------------------------------------------------------------ issuer: the whole warp stays converged, the
     // products are predicated on the elected lane (see tcgen05.cuh on issuing from a whole warp)
     constexpr uint32_t idesc_qk = instruction_descriptor(kRows, kKeys, false);
-    constexpr uint32_t idesc_pv = instruction_descriptor(kRows, kDim, true);
+    constexpr uint32_t idesc_pv = instruction_descriptor(kRows, kValueDim, true);
     const uint32_t elected = elect_one();
     const uint32_t q_low = operand_low(smem_base + kOffQ), k_low = operand_low(smem_base + kOffK);
     const uint32_t v_low = operand_low_mn_major(smem_base + kOffV, kHalf);
@@ -623,15 +638,16 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         float own_factor;
         const float* bias = (kScored && extras.rel_bias != nullptr)
                                 ? extras.rel_bias + (size_t)min(w.head, extras.rel_heads - 1) * extras.rel_rows : nullptr;
+        const float slope = (kScored && extras.slopes != nullptr) ? extras.slopes[w.head] : 0.0f;
         const int distance = position - key0 - first;         // of this thread's first column
         const float sum = every ? softmax_tile<false, kShared, kScored>(scores, first, low, high, scale_log2, reference, factor,
                                                                         grow, packed, shared_max, part, team, stamp_tile,
                                                                         handoff, own_factor, alive, extras.softcap, bias,
-                                                                        extras.rel_rows - 1, distance)
+                                                                        extras.rel_rows - 1, distance, slope)
                                 : softmax_tile<true, kShared, kScored>(scores, first, low, high, scale_log2, reference, factor,
                                                                        grow, packed, shared_max, part, team, stamp_tile,
                                                                        handoff, own_factor, alive, extras.softcap, bias,
-                                                                       extras.rel_rows - 1, distance);
+                                                                       extras.rel_rows - 1, distance, slope);
         ATT_STAMP(stamp_tile, 9);
         denominator = denominator * own_factor + sum;
         // Split keys: this stream's previous product (tile t - kStreams) is over: S(t) was issued behind it, and the
@@ -648,12 +664,13 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         }
         if (rescale) {
 #pragma unroll 1
-          for (int c0 = 0; c0 < kDim / kParts; c0 += 32) {
+          for (int c0 = 0; c0 < kValueDim / kParts; c0 += 32) {
+            constexpr int kPart = kValueDim / kParts;
             float o[32];
-            tmem_load_32(my_o + first + c0, o);
+            tmem_load_32(my_o + part * kPart + c0, o);
 #pragma unroll
             for (int i = 0; i < 32; ++i) o[i] *= factor;
-            tmem_store_32(my_o + first + c0, o);
+            tmem_store_32(my_o + part * kPart + c0, o);
           }
         }
         // P as the A operand of the product with V, in tensor memory over the scores it came from: this row's lane,
@@ -692,33 +709,34 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
       tensor_fence_after_sync();
       ATT_STAMP(stamp_item, 2);
       {
-        // this thread's columns of the output: the row's 128 are shared out over all its softmax threads
-        constexpr int kOut = kDim / (kParts * kStreams);
+        // this thread's columns of the output: the row's are shared out over all its softmax threads
+        constexpr int kOut = kValueDim / (kParts * kStreams);
+        constexpr int kPiece = kOut < 32 ? kOut : 32;          // columns it handles at a time
         const int column = (stream * kParts + part) * kOut;
         const float inverse = total > 0.0f ? 1.0f / total : 0.0f;
-        bf16* dst = out + ((size_t)(w.q_row0 + r) * heads + w.head) * kDim + column;
+        bf16* dst = out + ((size_t)(w.q_row0 + r) * heads + w.head) * kValueDim + column;
 #pragma unroll 1
-        for (int c0 = 0; c0 < kOut; c0 += 32) {
-          float o[32];
+        for (int c0 = 0; c0 < kOut; c0 += kPiece) {
+          float o[kPiece];
 #pragma unroll
-          for (int i = 0; i < 32; ++i) o[i] = 0.0f;
+          for (int i = 0; i < kPiece; ++i) o[i] = 0.0f;
 #pragma unroll
           for (int other = 0; other < (kShared ? 1 : kStreams); ++other) {
             if (kShared) {
               // one accumulator, scaled to the last tile's reference, which is the largest
-              float theirs[32];
-              tmem_load_32(tmem_o + lane_bits + column + c0, theirs);
+              float theirs[kPiece];
+              tmem_load_piece(tmem_o + lane_bits + column + c0, theirs);
 #pragma unroll
-              for (int i = 0; i < 32; ++i) o[i] = inverse > 0.0f ? theirs[i] * inverse : 0.0f;
+              for (int i = 0; i < kPiece; ++i) o[i] = inverse > 0.0f ? theirs[i] * inverse : 0.0f;
             } else if (other < w.tiles) {                     // a stream without a tile never wrote its O
-              float theirs[32];
-              tmem_load_32(tmem_o + (uint32_t)other * 128u + lane_bits + column + c0, theirs);
+              float theirs[kPiece];
+              tmem_load_piece(tmem_o + (uint32_t)other * 128u + lane_bits + column + c0, theirs);
               const float share = weight[other] * inverse;
 #pragma unroll
-              for (int i = 0; i < 32; ++i) o[i] += share > 0.0f ? theirs[i] * share : 0.0f;
+              for (int i = 0; i < kPiece; ++i) o[i] += share > 0.0f ? theirs[i] * share : 0.0f;
             }
           }
-          if (c0 + 32 >= kOut) {
+          if (c0 + kPiece >= kOut) {
             // the accumulators are read out: the next item's products may overwrite them
             tensor_fence_before_sync();
             barrier_arrive(bar(O_FREE));
@@ -729,13 +747,13 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
             const float g = __bfloat162float(extras.gate[(size_t)(w.q_row0 + r) * (size_t)extras.gate_stride + w.head]);
             const float share = 1.0f / (1.0f + __expf(-g));
 #pragma unroll
-            for (int i = 0; i < 32; ++i) o[i] *= share;
+            for (int i = 0; i < kPiece; ++i) o[i] *= share;
           } else if (valid_row && alive && extras.gate != nullptr) {
-            // the gate's 32 elements of this token and head (16-byte pieces: the entry point checks the alignment)
+            // the gate's elements of this token and head (16-byte pieces: the entry point checks the alignment)
             const bf16* gate = extras.gate + (size_t)(w.q_row0 + r) * (size_t)extras.gate_stride +
-                               (size_t)w.head * kDim + column + c0;
+                               (size_t)w.head * kValueDim + column + c0;
 #pragma unroll
-            for (int i = 0; i < 32; i += 8) {
+            for (int i = 0; i < kPiece; i += 8) {
               float g[8];
               load8(gate + i, g);
 #pragma unroll
@@ -744,7 +762,7 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
           }
           if (valid_row && alive) {
 #pragma unroll
-            for (int i = 0; i < 32; i += 8) {
+            for (int i = 0; i < kPiece; i += 8) {
               uint4 packed_out;
               __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&packed_out);
 #pragma unroll
@@ -789,6 +807,9 @@ MIR_EXPORT int mir_prefill_attention_tc_error() {
   return flag;
 }
 
+// The widths of a value head that it takes beside keys of 128 (64: with modified scores only).
+MIR_EXPORT int mir_prefill_attention_tc_takes_values(int value_dim) { return value_dim == kDim || value_dim == 64; }
+
 // Whether the tcgen05 kernel takes these sizes (head_dim 128, pages of 8 to 128 keys that divide 128).
 MIR_EXPORT int mir_prefill_attention_tc_takes(int head_dim, int page_size) {
   return head_dim == kDim && page_size >= 8 && page_size <= kKeys && kKeys % page_size == 0 && page_size % 8 == 0;
@@ -822,16 +843,24 @@ static int prefill_attention_tc_with(const void* q, long long q_stride, void* ou
                   heads, kv_heads);
     return MIR_BAD_ARGUMENT;
   }
+  const int value_dim = extras.value_dim > 0 ? extras.value_dim : head_dim;
+  const bool scored = scores_modified(extras);
+  if (!mir_prefill_attention_tc_takes_values(value_dim) || (value_dim != kDim && !scored) ||
+      (extras.slopes != nullptr && extras.rel_bias != nullptr)) {
+    mir_set_error("prefill_attention_tc: value heads of %d (64 goes with modified scores), and one kind of bias at a time",
+                  value_dim);
+    return MIR_BAD_ARGUMENT;
+  }
   CUtensorMap q_map, k_map, v_map, k_tile_map, v_tile_map;
   int status = tensor_map_for(q, tokens, (int)q_stride, (int)q_stride, kRows, &q_map);
   if (status != MIR_OK) return status;
   status = tensor_map_for(k_pages, (int)cache_rows, kv_heads * kDim, kv_heads * kDim, page_size, &k_map);
   if (status != MIR_OK) return status;
-  status = tensor_map_for(v_pages, (int)cache_rows, kv_heads * kDim, kv_heads * kDim, page_size, &v_map);
+  status = tensor_map_for(v_pages, (int)cache_rows, kv_heads * value_dim, kv_heads * value_dim, page_size, &v_map);
   if (status != MIR_OK) return status;
   status = tensor_map_for(k_pages, (int)cache_rows, kv_heads * kDim, kv_heads * kDim, kKeys, &k_tile_map);
   if (status != MIR_OK) return status;
-  status = tensor_map_for(v_pages, (int)cache_rows, kv_heads * kDim, kv_heads * kDim, kKeys, &v_tile_map);
+  status = tensor_map_for(v_pages, (int)cache_rows, kv_heads * value_dim, kv_heads * value_dim, kKeys, &v_tile_map);
   if (status != MIR_OK) return status;
   static bool configured = false;
   if (!configured) {
@@ -846,6 +875,9 @@ static int prefill_attention_tc_with(const void* q, long long q_stride, void* ou
     if (err == cudaSuccess)
       err = cudaFuncSetAttribute(tc_prefill_attention_kernel<2, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  kSmemBytes);
+    if (err == cudaSuccess)
+      err = cudaFuncSetAttribute(tc_prefill_attention_kernel<2, true, true, 64>,
+                                 cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
     if (err != cudaSuccess) {
       mir_set_error("prefill_attention_tc: cannot reserve %d bytes of shared memory: %s", kSmemBytes,
                     cudaGetErrorString(err));
@@ -866,7 +898,12 @@ static int prefill_attention_tc_with(const void* q, long long q_stride, void* ou
     if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess || sms <= 0) sms = 148;
   }
   const int ctas = (int)std::min<long long>(items, g_ctas > 0 ? g_ctas : sms);
-  if (extras.softcap > 0.0f || extras.rel_bias != nullptr)   // capped or biased scores: two streams, a shared reference
+  if (value_dim == 64)
+    return mir_launch("prefill_attention_tc", tc_prefill_attention_kernel<2, true, true, 64>, dim3(ctas), dim3(threads_for(2)),
+                      (size_t)kSmemBytes, stream, 0, q_map, k_map, v_map, k_tile_map, v_tile_map, (bf16*)out, block_table, table_width,
+                      query_starts, context_lens, num_rows, page_size, heads, kv_heads,
+                      scale * 1.4426950408889634f, window, tile_slots, window > 0 ? keep_first : 0, extras);
+  if (scored)                                                // capped or biased scores: two streams, a shared reference
     return mir_launch("prefill_attention_tc", tc_prefill_attention_kernel<2, true, true>, dim3(ctas), dim3(threads_for(2)),
                       (size_t)kSmemBytes, stream, 0, q_map, k_map, v_map, k_tile_map, v_tile_map, (bf16*)out, block_table, table_width,
                       query_starts, context_lens, num_rows, page_size, heads, kv_heads,
@@ -908,10 +945,10 @@ MIR_EXPORT int mir_prefill_attention_tc_scored_bf16(const void* q, long long q_s
                                                     int num_rows, int tokens, int page_size, int heads, int kv_heads,
                                                     int head_dim, float scale, int window, cudaStream_t stream,
                                                     const float* sinks, const void* gate, long long gate_stride,
-                                                    int gate_per_head, float softcap, const float* rel_bias, int rel_rows) {
+                                                    int gate_per_head, float softcap, const float* rel_bias, int rel_rows, const float* slopes, int value_dim) {
   if (rel_bias != nullptr && rel_rows <= 0) { mir_set_error("prefill_attention_tc: a bias by distance needs entries"); return MIR_BAD_ARGUMENT; }
-  const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_per_head ? head_dim : 0, softcap, rel_bias,
-                               rel_rows, heads};
+  const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_per_head ? (value_dim > 0 ? value_dim : head_dim) : 0, softcap, rel_bias,
+                               rel_rows, heads, slopes, value_dim};
   return prefill_attention_tc_with(q, q_stride, out, k_pages, v_pages, cache_rows, block_table, table_width, query_starts,
                                    context_lens, num_rows, tokens, page_size, heads, kv_heads, head_dim, scale, window, 0,
                                    stream, extras);

@@ -125,7 +125,9 @@ __device__ __forceinline__ uint32_t small_operand_offset(int row, int column) {
 }
 
 // G: how many columns of the accumulators the softmax threads touch (the group's heads rounded up to 4, 8 or 16).
-template <int G>
+// DV: width of a value head, 128 or 64.  With 64 the second half of the value tile is zeros from the start and never
+// loaded: the product keeps its 128 rows, of which the lower 64 are the head's elements.
+template <int G, int DV>
 __global__ void __launch_bounds__(kThreads)
 tc_decode_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                            const __grid_constant__ CUtensorMap k_tile_map,
@@ -170,6 +172,11 @@ tc_decode_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __gr
     for (int i = 0; i < BARRIERS; ++i)
       barrier_init(bar(i), (i == P_READY || i == Q_READY) ? (uint32_t)kSoftmaxThreads : 1u);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (DV == 64) {
+    for (int i = threadIdx.x; i < kHalf / 16; i += kThreads)
+      *reinterpret_cast<uint4*>(smem + kOffV + kHalf + (size_t)i * 16) = make_uint4(0u, 0u, 0u, 0u);
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
   }
   if (warp == 5) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_slot)),
@@ -226,15 +233,16 @@ tc_decode_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __gr
         if (lane == 0) ok = wait_barrier(free_bar, parity ^ 1u) ? 1 : 0;
         ok = __shfl_sync(0xffffffffu, ok, 0);
         if (!ok) { if (lane == 0) g_tc_decode_error = 1; alive = false; break; }
-        if (lane == 0) barrier_expect_bytes(full, (uint32_t)kTile);
+        const int halves = which ? DV / 64 : 2, width = which ? DV : kDim;
+        if (lane == 0) barrier_expect_bytes(full, (uint32_t)(halves * kHalf));
         __syncwarp();
         if (in_a_row) {
-          if (lane < 2)
+          if (lane < halves)
             tma_load_2d(smem_base + (which ? kOffV : kOffK) + (uint32_t)lane * kHalf, which ? &v_tile_map : &k_tile_map,
-                        full, kv_head * kDim + lane * 64, first_row);
-        } else if (loads) {
+                        full, kv_head * width + lane * 64, first_row);
+        } else if (loads && half < halves) {
           tma_load_2d(smem_base + (which ? kOffV : kOffK) + (uint32_t)half * kHalf + (uint32_t)(slot * page_size) * 128u,
-                      which ? &v_map : &k_map, full, kv_head * kDim + half * 64, cache_row);
+                      which ? &v_map : &k_map, full, kv_head * width + half * 64, cache_row);
         }
       }
       cache_row = next_row;
@@ -377,7 +385,7 @@ tc_decode_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __gr
     tensor_fence_after_sync();
     float o[G];
     tmem_load<G>(tmem_o + lane_bits, o);
-    if (alive) {
+    if (alive && r < DV) {
 #pragma unroll
       for (int g = 0; g < G; ++g) {
         if (g >= valid_heads) break;
@@ -385,10 +393,10 @@ tc_decode_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __gr
         const size_t head = (size_t)row * heads + head0 + g;
         if (num_partitions == 1) {
           if (denom > 0.0f) denom += sink_term(extras, head0 + g, reference[g]);
-          out[head * kDim + r] = __float2bfloat16_rn(
-              denom > 0.0f ? o[g] / denom * gate_factor(extras, row, (size_t)(head0 + g) * kDim + r) : 0.0f);
+          out[head * DV + r] = __float2bfloat16_rn(
+              denom > 0.0f ? o[g] / denom * gate_factor(extras, row, (size_t)(head0 + g) * DV + r) : 0.0f);
         } else {
-          partial_o[(head * num_partitions + part) * kDim + r] = denom > 0.0f ? o[g] : 0.0f;
+          partial_o[(head * num_partitions + part) * DV + r] = denom > 0.0f ? o[g] : 0.0f;
           if (r == 0) {
             partial_ml[(head * num_partitions + part) * 2] = reference[g];
             partial_ml[(head * num_partitions + part) * 2 + 1] = denom;
@@ -407,7 +415,7 @@ tc_decode_attention_kernel(const __grid_constant__ CUtensorMap k_map, const __gr
   if (threadIdx.x == 0) MIR_TRACE_POINT(decode, 12);
 }
 
-template <int G>
+template <int G, int DV>
 int launch(const CUtensorMap& k_map, const CUtensorMap& v_map, const CUtensorMap& k_tile_map,
            const CUtensorMap& v_tile_map, const bf16* q, size_t q_stride, const int* block_table,
            int table_width, const int* positions, int rows, int page_size, int heads, int kv_heads, float scale,
@@ -415,7 +423,7 @@ int launch(const CUtensorMap& k_map, const CUtensorMap& v_map, const CUtensorMap
            cudaStream_t stream, AttentionExtras extras) {
   static bool configured = false;
   if (!configured) {
-    const cudaError_t err = cudaFuncSetAttribute(tc_decode_attention_kernel<G>,
+    const cudaError_t err = cudaFuncSetAttribute(tc_decode_attention_kernel<G, DV>,
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
     if (err != cudaSuccess) {
       mir_set_error("decode_attention_tc: cannot reserve %d bytes of shared memory: %s", kSmemBytes,
@@ -429,7 +437,7 @@ int launch(const CUtensorMap& k_map, const CUtensorMap& v_map, const CUtensorMap
   // the partition is the fast index (a request's CTAs start together), except for a handful of rows, where
   // partitions beyond the contexts (dead CTAs of a captured batch) are dispatched last
   const dim3 grid = rows <= 4 ? dim3(rows, units, num_partitions) : dim3(num_partitions, units, rows);
-  return mir_launch_with(mir_pdl_for_streaming(), "decode_attention_tc", tc_decode_attention_kernel<G>, grid,
+  return mir_launch_with(mir_pdl_for_streaming(), "decode_attention_tc", tc_decode_attention_kernel<G, DV>, grid,
                          dim3(kThreads), (size_t)kSmemBytes, stream, 0, k_map, v_map, k_tile_map, v_tile_map, q, q_stride,
                          block_table,
                          table_width, positions, page_size, heads, kv_heads, scale * 1.4426950408889634f, window,
@@ -453,6 +461,9 @@ MIR_EXPORT int mir_decode_attention_tc_takes(int head_dim, int page_size, int pa
          page_size % 8 == 0 && partition > 0 && partition % kKeys == 0;
 }
 
+// The widths of a value head that it takes beside keys of 128.
+MIR_EXPORT int mir_decode_attention_tc_takes_values(int value_dim) { return value_dim == kDim || value_dim == 64; }
+
 // One token per row, as mir_decode_attention_bf16; k_pages and v_pages are [cache_rows, kv_heads, 128].  sinks, gate,
 // gate_stride: what AttentionExtras describes (null for none).
 static int decode_attention_tc_with(const void* q, long long q_stride, void* out, const void* k_pages,
@@ -473,7 +484,12 @@ static int decode_attention_tc_with(const void* q, long long q_stride, void* out
                   head_dim, page_size, partition, heads, kv_heads, rows, num_partitions);
     return MIR_BAD_ARGUMENT;
   }
-  const long long need = mir_decode_attention_scratch_floats(rows, heads, head_dim, num_partitions);
+  const int value_dim = extras.value_dim > 0 ? extras.value_dim : head_dim;
+  if (!mir_decode_attention_tc_takes_values(value_dim)) {
+    mir_set_error("decode_attention_tc: value heads of %d are neither 64 nor 128", value_dim);
+    return MIR_BAD_ARGUMENT;
+  }
+  const long long need = mir_decode_attention_scratch_floats(rows, heads, value_dim, num_partitions);
   if (need < 0 || (need > 0 && (scratch == nullptr || scratch_floats < need))) {
     mir_set_error("decode_attention_tc: scratch of %lld floats is needed, got %lld", need, scratch_floats);
     return MIR_BAD_ARGUMENT;
@@ -481,23 +497,26 @@ static int decode_attention_tc_with(const void* q, long long q_stride, void* out
   CUtensorMap k_map, v_map, k_tile_map, v_tile_map;
   int status = tensor_map_for(k_pages, (int)cache_rows, kv_heads * kDim, kv_heads * kDim, page_size, &k_map);
   if (status != MIR_OK) return status;
-  status = tensor_map_for(v_pages, (int)cache_rows, kv_heads * kDim, kv_heads * kDim, page_size, &v_map);
+  status = tensor_map_for(v_pages, (int)cache_rows, kv_heads * value_dim, kv_heads * value_dim, page_size, &v_map);
   if (status != MIR_OK) return status;
   status = tensor_map_for(k_pages, (int)cache_rows, kv_heads * kDim, kv_heads * kDim, kKeys, &k_tile_map);
   if (status != MIR_OK) return status;
-  status = tensor_map_for(v_pages, (int)cache_rows, kv_heads * kDim, kv_heads * kDim, kKeys, &v_tile_map);
+  status = tensor_map_for(v_pages, (int)cache_rows, kv_heads * value_dim, kv_heads * value_dim, kKeys, &v_tile_map);
   if (status != MIR_OK) return status;
   const int group = heads / kv_heads;
   const int columns = std::min(group, kHeads);
   float* partial_o = scratch;
-  float* partial_ml = scratch ? scratch + (size_t)rows * heads * num_partitions * head_dim : nullptr;
+  float* partial_ml = scratch ? scratch + (size_t)rows * heads * num_partitions * value_dim : nullptr;
 #define MIR_SPLIT(G)                                                                                                 \
-  launch<G>(k_map, v_map, k_tile_map, v_tile_map, (const bf16*)q, (size_t)q_stride, block_table, table_width, positions, rows, page_size, heads, \
+  (value_dim == 64 ? MIR_SPLIT_AS(G, 64) : MIR_SPLIT_AS(G, kDim))
+#define MIR_SPLIT_AS(G, DV)                                                                                          \
+  launch<G, DV>(k_map, v_map, k_tile_map, v_tile_map, (const bf16*)q, (size_t)q_stride, block_table, table_width, positions, rows, page_size, heads, \
             kv_heads, scale, window, partition, num_partitions, partial_o, partial_ml, (bf16*)out, stream, extras)
   status = columns <= 4 ? MIR_SPLIT(4) : (columns <= 8 ? MIR_SPLIT(8) : MIR_SPLIT(16));
 #undef MIR_SPLIT
+#undef MIR_SPLIT_AS
   if (status != MIR_OK || num_partitions == 1) return status;
-  return mir_decode_merge_gated_bf16(partial_o, partial_ml, positions, rows, heads, head_dim, window, partition,
+  return mir_decode_merge_gated_bf16(partial_o, partial_ml, positions, rows, heads, value_dim, window, partition,
                                      num_partitions, out, stream, extras.sinks, extras.gate, extras.gate_stride,
                                      extras.gate_head_width);
 }
@@ -524,10 +543,10 @@ MIR_EXPORT int mir_decode_attention_tc_scored_bf16(const void* q, long long q_st
                                                    int partition, int num_partitions, float* scratch,
                                                    long long scratch_floats, cudaStream_t stream, const float* sinks,
                                                    const void* gate, long long gate_stride, int gate_per_head,
-                                                   float softcap, const float* rel_bias, int rel_rows) {
+                                                   float softcap, const float* rel_bias, int rel_rows, const float* slopes, int value_dim) {
   if (rel_bias != nullptr && rel_rows <= 0) { mir_set_error("decode_attention_tc: a bias by distance needs entries"); return MIR_BAD_ARGUMENT; }
-  const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_per_head ? head_dim : 0, softcap, rel_bias,
-                               rel_rows, heads};
+  const AttentionExtras extras{sinks, (const bf16*)gate, gate_stride, gate_per_head ? (value_dim > 0 ? value_dim : head_dim) : 0, softcap, rel_bias,
+                               rel_rows, heads, slopes, value_dim};
   return decode_attention_tc_with(q, q_stride, out, k_pages, v_pages, cache_rows, block_table, table_width, positions,
                                   rows, page_size, heads, kv_heads, head_dim, scale, window, partition, num_partitions,
                                   scratch, scratch_floats, stream, extras);

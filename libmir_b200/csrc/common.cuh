@@ -140,7 +140,7 @@ __device__ __forceinline__ float gate_factor(const AttentionExtras& extras, size
   if (extras.gate_head_width > 0) column /= (size_t)extras.gate_head_width;
   return 1.0f / (1.0f + __expf(-__bfloat162float(extras.gate[token * (size_t)extras.gate_stride + column])));
 }
-__device__ __forceinline__ bool scores_modified(const AttentionExtras& extras) {
+__host__ __device__ __forceinline__ bool scores_modified(const AttentionExtras& extras) {
   return extras.softcap > 0.0f || extras.rel_bias != nullptr || extras.slopes != nullptr;
 }
 // A score that is already scaled and in units of log2 e (the tile kernels' form), capped and biased in 32-bit.

@@ -174,16 +174,17 @@ MIR_EXPORT int mir_decode_attention_paged_scored_bf16(const void* q, long long q
                                                       int partition, int num_partitions, float* scratch,
                                                       long long scratch_floats, cudaStream_t stream, const float* sinks,
                                                       const void* gate, long long gate_stride, int gate_per_head,
-                                                      float softcap, const float* rel_bias, int rel_rows) {
-  if (g_decode_tensor_cores && cache_rows > 0 && mir_decode_attention_tc_takes(head_dim, page_size, partition))
+                                                      float softcap, const float* rel_bias, int rel_rows, const float* slopes, int value_dim) {
+  if (g_decode_tensor_cores && cache_rows > 0 && mir_decode_attention_tc_takes(head_dim, page_size, partition) &&
+      mir_decode_attention_tc_takes_values(value_dim > 0 ? value_dim : head_dim))
     return mir_decode_attention_tc_scored_bf16(q, q_stride, out, k_pages, v_pages, cache_rows, block_table, table_width,
                                                positions, rows, page_size, heads, kv_heads, head_dim, scale, window,
                                                partition, num_partitions, scratch, scratch_floats, stream, sinks, gate,
-                                               gate_stride, gate_per_head, softcap, rel_bias, rel_rows);
+                                               gate_stride, gate_per_head, softcap, rel_bias, rel_rows, slopes, value_dim);
   return mir_decode_attention_scored_bf16(q, q_stride, out, k_pages, v_pages, block_table, table_width, positions, rows,
                                           page_size, heads, kv_heads, head_dim, scale, window, partition, num_partitions,
                                           scratch, scratch_floats, stream, sinks, gate, gate_stride, gate_per_head, softcap,
-                                          rel_bias, rel_rows);
+                                          rel_bias, rel_rows, slopes, value_dim);
 }
 
 MIR_EXPORT int mir_decode_attention_paged_bf16(const void* q, long long q_stride, void* out, const void* k_pages,

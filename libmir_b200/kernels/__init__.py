@@ -125,19 +125,19 @@ _SIGNATURES = {
         "mir_decode_attention_scored_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                              c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p,
                                              c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float,
-                                             c_void_p, c_int],
+                                             c_void_p, c_int, c_void_p, c_int],
         "mir_prefill_attention_tc_scored_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
                                                  c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                  c_float, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float,
-                                                 c_void_p, c_int],
+                                                 c_void_p, c_int, c_void_p, c_int],
         "mir_decode_attention_paged_scored_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong,
                                                    c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                                    c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
-                                                   c_void_p, c_longlong, c_int, c_float, c_void_p, c_int],
+                                                   c_void_p, c_longlong, c_int, c_float, c_void_p, c_int, c_void_p, c_int],
         "mir_prefill_attention_scored_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                               c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                                               c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_void_p,
-                                              c_int],
+                                              c_int, c_void_p, c_int],
         "mir_decode_attention_paged_extra_bf16": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong,
                                                   c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                                   c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
@@ -152,6 +152,8 @@ _SIGNATURES = {
                                             c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
                                             c_int, c_void_p, c_longlong, c_void_p],
         "mir_decode_attention_tc_takes": [c_int, c_int, c_int],
+        "mir_decode_attention_tc_takes_values": [c_int],
+        "mir_prefill_attention_tc_takes_values": [c_int],
         "mir_head_logits_bf16": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                  c_int, c_void_p, c_size_t, c_void_p, c_void_p],
         "mir_gemm_tc_stream_head_candidates": [c_int],
@@ -1572,7 +1574,9 @@ def mixed_prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch
 
 
 def _check_extras(what: str, sinks, gate, out: torch.Tensor, heads: int, gate_per_head: bool = False,
-                  distance_bias=None) -> None:
+                  distance_bias=None, slopes=None) -> None:
+    _require(slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == heads and slopes.is_contiguous()),
+             f"{what}: slopes are float32 [heads]")
     _require(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads and sinks.is_contiguous()),
              f"{what}: sinks are float32 [heads]")
     _require(gate is None or (gate.dtype == out.dtype and gate.stride(1) == 1
@@ -1585,14 +1589,21 @@ def _check_extras(what: str, sinks, gate, out: torch.Tensor, heads: int, gate_pe
 
 
 FAST_HEAD_DIMS = (64, 128)      # what the tensor-core attention kernels take; other sizes use the reference kernel
+FAST_VALUE_DIMS = (32, 64, 128)  # widths of a value head that they take where it differs from the key's (no kept keys then)
 
 
-def decode_attention_plan(rows: int, heads: int, kv_heads: int, head_dim: int, page_size: int, max_context: int) -> tuple:
+def decode_attention_plan(rows: int, heads: int, kv_heads: int, head_dim: int, page_size: int, max_context: int,
+                          value_dim: Optional[int] = None) -> tuple:
     """(keys per partition, partitions, floats of scratch) for the attention of `rows` single tokens whose longest
     context (or block-table width) is max_context keys.  The plan is native (csrc/ops_bf16.cu:
     mir_decode_attention_plan), the same for the Python launcher and the layer executor: the tcgen05 kernel where
     it takes the sizes (partitions chosen by the cost of its waves, or decode_tc_partition_keys), else the mma.sync
-    kernel with partitions of decode_partition_keys."""
+    kernel with partitions of decode_partition_keys.  `value_dim`: width of a value head where it differs."""
+    if value_dim is not None and value_dim != head_dim:
+        if not library("bf16").mir_decode_attention_tc_takes_values(value_dim):
+            return decode_attention_kept_plan(rows, heads, value_dim, max_context)
+        partition, count, _ = decode_attention_plan(rows, heads, kv_heads, head_dim, page_size, max_context)
+        return partition, count, decode_attention_scratch_floats(rows, heads, value_dim, count)
     partition, count, floats = ctypes.c_int(), ctypes.c_int(), ctypes.c_longlong()
     lib = library("bf16")
     _check(lib, lib.mir_decode_attention_plan(rows, heads, kv_heads, head_dim, page_size, max_context,
@@ -1619,35 +1630,38 @@ def decode_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor
                      scratch: Optional[torch.Tensor], keep_first: int = 0,
                      numbering: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
                      gate: Optional[torch.Tensor] = None, gate_per_head: bool = False, softcap: Optional[float] = None,
-                     distance_bias: Optional[torch.Tensor] = None) -> None:
+                     distance_bias: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
+                     value_dim: Optional[int] = None) -> None:
     """bf16 split-KV attention for a batch of single tokens (row r of qkv belongs to request row r).  `keep_first`:
     with a window, the request's first keys that stay visible; the mma.sync kernel then walks over the kept keys and
     the window's as one run, and `numbering` (int32 [rows]) is scratch for the merge.  `sinks`, `gate`: as
     paged_attention_generic takes them (the kernel that writes a row's final result, the attention kernel or the
     merge of its partitions, adds the sink's term and applies the gate).  `gate_per_head`, `softcap`, `distance_bias`:
     as paged_attention_generic takes them: the scores are capped and biased in 32-bit before the softmax, by the
-    tcgen05 kernel where it takes the sizes and the partition (decode_attention_plan), else by the mma.sync kernel."""
-    _cuda(qkv, out, k_pages, v_pages, block_table, positions, scratch, sinks, gate, distance_bias)
+    tcgen05 kernel where it takes the sizes and the partition (decode_attention_plan), else by the mma.sync kernel.
+    `slopes` likewise; `value_dim`: width of a value head where it differs from a key head's."""
+    _cuda(qkv, out, k_pages, v_pages, block_table, positions, scratch, sinks, gate, distance_bias, slopes)
     rows = out.shape[0]
-    _check_extras("decode_attention", sinks, gate, out, heads, gate_per_head, distance_bias)
+    value_dim = head_dim if value_dim is None else value_dim
+    _check_extras("decode_attention", sinks, gate, out, heads, gate_per_head, distance_bias, slopes)
     gate_args = (_ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0)
     _require(qkv.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and k_pages.dtype == torch.bfloat16
-             and v_pages.dtype == torch.bfloat16 and out.is_contiguous() and out.shape[1] == heads * head_dim,
-             "decode_attention: bfloat16 tensors are needed")
+             and v_pages.dtype == torch.bfloat16 and out.is_contiguous() and out.shape[1] == heads * value_dim
+             and v_pages.shape[-1] == value_dim, "decode_attention: bfloat16 tensors are needed")
     _require(block_table.dtype == torch.int32 and block_table.is_contiguous() and positions.dtype == torch.int32
              and positions.numel() >= rows and block_table.shape[0] >= rows, "decode_attention: bad metadata")
     _require(scratch is None or scratch.dtype == torch.float32, "decode_attention: scratch must be float32")
     lib = library("bf16")
     _require(k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.shape[0] == v_pages.shape[0],
              "decode_attention: the cache tensors must be contiguous [token rows, kv_heads, head_dim]")
-    if gate_per_head or softcap or distance_bias is not None:
+    if gate_per_head or softcap or distance_bias is not None or slopes is not None or value_dim != head_dim:
         _require(not (keep_first and window), "decode_attention: capped or biased scores do not go with kept first keys")
         _check(lib, lib.mir_decode_attention_paged_scored_bf16(
             qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), k_pages.shape[0],
             block_table.data_ptr(), block_table.shape[1], positions.data_ptr(), rows, page_size, heads, kv_heads,
             head_dim, scale, int(window or 0), partition, num_partitions, _ptr(scratch),
             0 if scratch is None else scratch.numel(), _stream(), *gate_args, int(gate_per_head), float(softcap or 0.0),
-            _ptr(distance_bias), distance_bias.shape[1] if distance_bias is not None else 0))
+            _ptr(distance_bias), distance_bias.shape[1] if distance_bias is not None else 0, _ptr(slopes), value_dim))
         return
     if keep_first and window:
         _cuda(numbering)
@@ -1680,39 +1694,44 @@ def prefill_attention(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tenso
                       portion_tokens: Optional[int] = None, keep_first: int = 0,
                       sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                       gate_per_head: bool = False, softcap: Optional[float] = None,
-                      distance_bias: Optional[torch.Tensor] = None) -> None:
+                      distance_bias: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
+                      value_dim: Optional[int] = None) -> None:
     """bf16 tensor-core attention for any mix of portions (row r owns tokens query_starts[r]..query_starts[r+1]
     of the packed qkv and out; the rows may be a part of the batch, `portion_tokens` then says how many tokens
     they have together).  `tensor_cores`: True runs the tcgen05 kernel, False the mma.sync kernel, None chooses.
     `keep_first`: with a window, the first keys of a request that every later query still sees.  `sinks`, `gate`: as
     paged_attention_generic takes them, in the kernels' epilogues (the gate's rows are those of the whole batch, as
     out's are).  `gate_per_head`, `softcap`, `distance_bias`: as paged_attention_generic takes them; both tile kernels
-    cap and bias the scores in 32-bit before the softmax."""
-    _cuda(qkv, out, k_pages, v_pages, block_table, query_starts, context_lens, sinks, gate, distance_bias)
+    cap and bias the scores in 32-bit before the softmax.  `slopes` likewise; `value_dim`: width of a value head where it
+    differs from a key head's."""
+    _cuda(qkv, out, k_pages, v_pages, block_table, query_starts, context_lens, sinks, gate, distance_bias, slopes)
     tokens = out.shape[0]
-    _check_extras("prefill_attention", sinks, gate, out, heads, gate_per_head, distance_bias)
+    value_dim = head_dim if value_dim is None else value_dim
+    _check_extras("prefill_attention", sinks, gate, out, heads, gate_per_head, distance_bias, slopes)
     gate_args = (_ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0)
     rows = context_lens.numel()
     _require(qkv.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and k_pages.dtype == torch.bfloat16
-             and v_pages.dtype == torch.bfloat16 and out.is_contiguous() and out.shape[1] == heads * head_dim,
-             "prefill_attention: bfloat16 tensors are needed")
+             and v_pages.dtype == torch.bfloat16 and out.is_contiguous() and out.shape[1] == heads * value_dim
+             and v_pages.shape[-1] == value_dim, "prefill_attention: bfloat16 tensors are needed")
     _require(block_table.dtype == torch.int32 and block_table.is_contiguous() and query_starts.dtype == torch.int32
              and context_lens.dtype == torch.int32 and query_starts.numel() == rows + 1
              and block_table.shape[0] >= rows, "prefill_attention: bad metadata")
     lib = library("bf16")
     keep_first = int(keep_first or 0) if window else 0
-    if gate_per_head or softcap or distance_bias is not None:
+    if gate_per_head or softcap or distance_bias is not None or slopes is not None or value_dim != head_dim:
         _require(not keep_first, "prefill_attention: capped or biased scores do not go with kept first keys")
         scored_args = (*gate_args, int(gate_per_head), float(softcap or 0.0), _ptr(distance_bias),
-                       distance_bias.shape[1] if distance_bias is not None else 0)
+                       distance_bias.shape[1] if distance_bias is not None else 0, _ptr(slopes), value_dim)
         if tensor_cores is None:
             portion_tokens = tokens if portion_tokens is None else portion_tokens
             tensor_cores = (PREFILL_TENSOR_CORES and portion_tokens >= PREFILL_TENSOR_CORE_MIN_PORTION * rows
                             and bool(lib.mir_prefill_attention_tc_takes(head_dim, page_size))
+                            and bool(lib.mir_prefill_attention_tc_takes_values(value_dim))
+                            and (value_dim == head_dim or bool(softcap) or distance_bias is not None or slopes is not None)
                             and k_pages.is_contiguous() and v_pages.is_contiguous() and scale > 0
                             and (gate is None or gate_per_head or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0)))
         if tensor_cores:
-            _require(k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.shape == v_pages.shape,
+            _require(k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.shape[:-1] == v_pages.shape[:-1],
                      "prefill_attention: the tcgen05 kernel reads contiguous [rows, kv_heads, head_dim] pages")
             _check(lib, lib.mir_prefill_attention_tc_scored_bf16(
                 qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), k_pages.shape[0],

@@ -292,18 +292,20 @@ class SoftmaxAttention(Mixer):
         first = self.q_width + self.kv_columns
         gate = qkv[:, first:first + self.gate_width] if s.gate else None        # [tokens, heads * value_dim] or [tokens, heads]
         scored = s.softcap is not None or self.distance_bias is not None or s.gate_per_head or self.slopes is not None
-        fast = self.env.dtype == torch.bfloat16 and s.head_dim in kernels.FAST_HEAD_DIMS and s.value_dim == s.head_dim \
-            and s.chunk is None and self.slopes is None                  # (runs of positions without mixed heads: the reference kernel)
+        fast = self.env.dtype == torch.bfloat16 and s.head_dim in kernels.FAST_HEAD_DIMS \
+            and (s.value_dim == s.head_dim or (self.slopes is not None and s.value_dim in kernels.FAST_VALUE_DIMS)) \
+            and s.chunk is None                  # (runs of positions without mixed heads: the reference kernel)
         if fast and scored and not kept:
             # capped or biased scores, or a gate per head: single tokens split over the keys, portions as tiles of
             # queries, each on the tcgen05 or the mma.sync kernel by size
             extras = dict(sinks=self.sinks, gate_per_head=s.gate_per_head, softcap=s.softcap,
-                          distance_bias=self.distance_bias)
+                          distance_bias=self.distance_bias, slopes=self.slopes, value_dim=s.value_dim)
             singles = ctx.num_rows if ctx.decode_only else ctx.single_rows
             if singles:
                 longest = ctx.max_context if ctx.decode_only else ctx.single_context
                 partition, count, floats = kernels.decode_attention_plan(singles, s.heads, s.kv_heads, s.head_dim,
-                                                                         cache.page_size, longest)
+                                                                         cache.page_size, longest,
+                                                                         value_dim=s.value_dim)
                 scratch = ctx.alloc((floats,), torch.float32) if floats else None
                 kernels.decode_attention(qkv[:singles], out[:singles], cache.k_pages, cache.v_pages,
                                          group.block_table[:singles], ctx.positions, cache.page_size, s.heads,
