@@ -1,5 +1,5 @@
-"""`bench.py --design doderax | zufotar | dalesun | gumazen | pedotar`: prefill and decode throughput of a design at layer sizes that resemble a
-real model's (random weights), beside the dense SwiGLU decoder of equal width, depth and parameter count (and, for
+"""`bench.py --design doderax | zufotar | dalesun | gumazen | pedotar | biravik`: prefill and decode throughput of a design at
+layer sizes that resemble a real model's (random weights), beside the dense SwiGLU decoder of equal width, depth and parameter count (and, for
 Zufotar, beside Doderax, the closest model of the framework: recurrent mixers and attention in parallel layers), and
 every kernel the design adds alone, with the fraction of its roofline, beside the like kernel of the closest model.
 
@@ -705,6 +705,180 @@ def pedotar_kernel_table(s, tools) -> dict:
     return table
 
 
+# Biravik: a wkv layer, two layers of biased attention beside lightning attention, and a layer of windowed attention whose
+# values are its keys, in turn; every second feed-forward routed experts.
+BIRAVIK_SIZES = {
+    "w2048": dict(width=2048, ff=8192, layers=12, runs=12, heads=16, kv_heads=4, dim=128, vdim=64, window=1024, keep_first=4,
+                  right_heads=16, right_dim=128, wkv_heads=32, wkv_dim=64, decay_rank=64, experts=64, top=6, expert_ff=1024,
+                  vocab=65536),
+    "w4096": dict(width=4096, ff=14336, layers=8, runs=8, heads=32, kv_heads=8, dim=128, vdim=64, window=2048, keep_first=4,
+                  right_heads=32, right_dim=128, wkv_heads=64, wkv_dim=64, decay_rank=64, experts=64, top=6, expert_ff=2048,
+                  vocab=65536),
+}
+
+
+def biravik_config(s: dict, experts: bool = True) -> dict:
+    left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5,
+            "q_temp": {"coef": 0.1, "every": 4096}}
+    right = {"heads": s["right_heads"], "dim": s["right_dim"], "vdim": s["right_dim"],
+             "decay": [1.0 - 2.0 ** (-4.0 - 8.0 * h / s["right_heads"]) for h in range(s["right_heads"])]}
+    parallel = {"type": "parallel", "mixer": {"left": left, "left_scale": 0.7, "right": right, "right_scale": 0.7}}
+    attention = {"type": "attention", "mixer": {
+        "heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+        "mask": {"size": s["window"], "keep_first": s["keep_first"]},
+        "rot": {"dims": s["dim"], "base": 1000000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    wkv = {"type": "wkv", "mixer": {"heads": s["wkv_heads"], "dim": s["wkv_dim"], "decay_rank": s["decay_rank"]}}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "router": {"experts": s["experts"], "top": s["top"]}}
+    kinds = (wkv, parallel, parallel, attention)
+    return {"architecture": "Biravik", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "postln_alpha": 2.0,
+            "layers": [dict(kinds[i % 4], mlp=moe if experts and i % 2 else dense) for i in range(s["layers"])]}
+
+
+def biravik_kernel_table(s, tools) -> dict:
+    """Every kernel the design adds or extends, alone, at the sizes of a 2,048-token prompt and of a step of 8 decoded
+    tokens: [microseconds, fraction of its roofline], beside the like kernel of the closest models (Dalesun's addition of a
+    normed branch, q/k kernel, retention and gated norm; Gumazen's attention with a bias by distance over all keys; Doderax's
+    attention with kept first keys; Zufotar's router; the dense decoder's attention).  A prompt's attention and recurrence
+    against the matrix peak, everything else against the copy bandwidth."""
+    import torch
+    from libmir_b200 import kernels
+    timed, copies, rand, device, hbm, flops_peak = (tools[k] for k in ("timed", "copies", "rand", "device", "hbm", "flops_peak"))
+    bf16, f32, i32 = torch.bfloat16, torch.float32, torch.int32
+    width, heads, kv_heads, dim, vdim, window, keep = (s[k] for k in ("width", "heads", "kv_heads", "dim", "vdim", "window", "keep_first"))
+    rh, rd = s["right_heads"], s["right_dim"]
+    rwidth = rh * rd
+    table = {}
+    note = ["of the bf16 tensor peak; the kernel is 32-bit FMA, one token after the other"]
+    for label, rows, portion in ((f"prefill_{PROMPT}", 1, PROMPT), (f"decode_b{BATCH}", BATCH, 1)):
+        tokens, prompt = rows * portion, portion > 1
+        starts = torch.arange(0, tokens + 1, portion, dtype=i32, device=device)
+        slots = torch.arange(rows, dtype=i32, device=device)
+        context = PROMPT if prompt else PROMPT + 1
+        positions = (torch.arange(tokens, dtype=i32, device=device) % portion) + (context - portion)
+        # ---- the norm behind the sum, of one result and of two with factors; beside Dalesun's (16 bytes a number move: the
+        # residual in and out, one or two results in; 2 more for the rounded copy)
+        packs = copies(lambda: tuple(rand(tokens, width, dtype=f32) for _ in range(3)), tokens * width * 12)
+        w_a, w_b = rand(width, dtype=f32), rand(width, dtype=f32)
+        out_w = torch.empty(tokens, width, device=device, dtype=bf16)
+        for branches in (1, 2):
+            moved = tokens * width * (4 * (branches + 2) + 2)
+            calls = [lambda p=p: kernels.norm_scaled_sum(list(p[1:1 + branches]), [0.7, 0.9][:branches], p[0], w_a, 2.0, 1e-6,
+                                                         rounded=out_w) for p in packs]
+            table[f"{label}_norm_behind_the_sum_{branches}"] = timed(calls, moved, hbm)
+            calls = [lambda p=p: kernels.add_normed_branches(list(p[1:1 + branches]), [w_a, w_b][:branches], p[0], 1e-6, 0.6,
+                                                             rounded=out_w) for p in packs]
+            table[f"{label}_dalesun_add_normed_branches_{branches}"] = timed(calls, moved, hbm)
+        del packs
+        # ---- the recurrence with activated inputs, beside Dalesun's with the rotation inside; the norm over all heads
+        packs = copies(lambda: (torch.zeros(rows, rh, rd, rd, device=device, dtype=f32), rand(tokens, 4 * rwidth, scale=0.3)),
+                       rows * rh * rd * rd * 4)
+        decays = torch.rand(rh, device=device, dtype=f32) * 0.1 + 0.9
+        inv_freq = torch.rand(rd // 2, device=device, dtype=f32)
+        read = torch.empty(tokens, rwidth, device=device, dtype=f32)
+        scratch = torch.empty(kernels.retention_prepared_floats(tokens, rh, rd), device=device, dtype=f32) if prompt else None
+        state_bytes = rows * rh * rd * rd * 8 + tokens * rwidth * (3 * 2 + 4)
+        for name, freq, activated in (("lightning_scan", None, True), ("dalesun_retention_scan", inv_freq, False)):
+            calls = [lambda p=p, f=freq, a=activated: kernels.retention_scan(
+                p[1][:, :rwidth], p[1][:, rwidth:2 * rwidth], p[1][:, 2 * rwidth:3 * rwidth], f, decays, 1.0, p[0], starts, slots,
+                positions, read, rh, rd, rd, prepared=scratch, activated=a) for p in packs]
+            table[f"{label}_{name}"] = timed(calls, 4.0 * tokens * rh * rd * rd, flops_peak) + note if prompt else \
+                timed(calls, state_bytes, hbm)
+        del packs
+        packs = copies(lambda: (rand(tokens, rwidth, dtype=f32), rand(tokens, rwidth)), tokens * rwidth * 6)
+        gated = torch.empty(tokens, rwidth, device=device, dtype=bf16)
+        for name, units, span, sigmoid in (("norm_over_all_heads_sigmoid_gate", 1, rwidth, True), ("dalesun_gated_head_norm", rh, rd, False)):
+            weight = torch.ones(span, device=device, dtype=f32)
+            calls = [lambda p=p, w=weight, u=units, n=span, g=sigmoid: kernels.gated_head_norm(p[0], p[1], w, gated, u, n, 1e-6, g)
+                     for p in packs]
+            table[f"{label}_{name}"] = timed(calls, tokens * rwidth * 8, hbm)
+        # ---- q and k into place: the temperature without a rotation and values of their own width; keys that are the values
+        # with scaled interleaved rotation; beside Dalesun's and the dense decoder's
+        pages_per_row = -(-(context + PAGE) // PAGE)
+        cache_rows = rows * pages_per_row * PAGE
+        banks = max(2, min(24, -(-(300 << 20) // (cache_rows * kv_heads * dim * 4))))
+        k_cache = [rand(cache_rows, kv_heads, dim, scale=0.5) for _ in range(banks)]
+        v_cache = [rand(cache_rows, kv_heads, dim, scale=0.5) for _ in range(banks)]
+        narrow = [rand(cache_rows, kv_heads, vdim, scale=0.5) for _ in range(banks)]
+        block_table = torch.arange(rows * pages_per_row, dtype=i32, device=device).view(rows, pages_per_row).contiguous()
+        contexts = torch.full((rows,), context, dtype=i32, device=device)
+        slot_map = (torch.arange(tokens, dtype=i32, device=device) // portion) * (pages_per_row * PAGE) + positions
+        biased = rand(tokens, (heads + kv_heads) * dim + kv_heads * vdim + heads * vdim, scale=0.3)
+        shared = rand(tokens, (heads + kv_heads) * dim + heads * dim, scale=0.3)
+        gated_rows = rand(tokens, (heads + 2 * kv_heads) * dim + heads * dim, scale=0.3)
+        norm_q, norm_k = torch.ones(dim, device=device), torch.ones(dim, device=device)
+        freq = torch.rand(dim // 2, device=device, dtype=f32)
+        moved = tokens * (heads + kv_heads) * dim * 4
+        calls = [lambda k=k, v=v: kernels.qk_rope_store(biased, positions, slot_map, None, norm_q, norm_k, k, v, heads, kv_heads,
+                                                        dim, 0, 1e-6, value_dim=vdim, temperature=(0.1, 4096))
+                 for k, v in zip(k_cache, narrow)]
+        table[f"{label}_qk_temperature_values_of_64"] = timed(calls, moved + tokens * kv_heads * vdim * 4, hbm)
+        calls = [lambda k=k, v=v: kernels.qk_rope_store(shared, positions, slot_map, freq, norm_q, norm_k, k, v, heads, kv_heads,
+                                                        dim, dim, 1e-6, interleaved=True, magnitude=1.1, values_from_keys=True)
+                 for k, v in zip(k_cache, v_cache)]
+        table[f"{label}_qk_values_from_keys"] = timed(calls, moved + tokens * kv_heads * dim * 2, hbm)
+        calls = [lambda k=k, v=v: kernels.qk_rope_store(gated_rows, positions, slot_map, freq, norm_q, norm_k, k, v, heads,
+                                                        kv_heads, dim, dim, 1e-6, interleaved=True) for k, v in zip(k_cache, v_cache)]
+        table[f"{label}_dalesun_qk_rope_store_interleaved"] = timed(calls, moved + tokens * kv_heads * dim * 4, hbm)
+        # ---- attention over all keys: a linear bias, sinks and a gate, values of 64 and of 128; beside Gumazen's bias by
+        # distance and the dense decoder's; in a window with kept first keys, sinks and a gate, beside Doderax's without
+        slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], device=device, dtype=f32)
+        bias = rand(heads, 513, dtype=f32)
+        sinks = rand(heads, dtype=f32)
+        wide_out = torch.empty(tokens, heads * dim, device=device, dtype=bf16)
+        narrow_out = torch.empty(tokens, heads * vdim, device=device, dtype=bf16)
+        wide_gate, narrow_gate = gated_rows[:, (heads + 2 * kv_heads) * dim:], biased[:, (heads + kv_heads) * dim + kv_heads * vdim:]
+        scale = dim ** -0.5
+        visible = PROMPT * (PROMPT + 1) / 2
+        in_window = sum(min(p + 1, window) for p in range(PROMPT))
+        full = [("attention_linear_bias_values_of_64", biased, narrow_out, narrow, vdim,
+                 dict(slopes=slopes, sinks=sinks, gate=narrow_gate, value_dim=vdim)),
+                ("attention_linear_bias_values_of_128", gated_rows, wide_out, v_cache, dim, dict(slopes=slopes, sinks=sinks, gate=wide_gate)),
+                ("gumazen_attention_bias_by_distance", gated_rows, wide_out, v_cache, dim, dict(distance_bias=bias, gate=wide_gate)),
+                ("dense_attention", gated_rows, wide_out, v_cache, dim, {})]
+        for name, packed, result, values, wide, extras in full:
+            if prompt:
+                calls = [lambda k=k, v=v, q=packed, o=result, e=extras: kernels.prefill_attention(
+                    q, o, k, v, block_table, starts, contexts, PAGE, heads, kv_heads, dim, scale, None, **e)
+                    for k, v in zip(k_cache, values)]
+                table[f"{label}_{name}"] = timed(calls, 2.0 * visible * heads * (dim + wide), flops_peak)
+                continue
+            partition, parts, floats = kernels.decode_attention_plan(rows, heads, kv_heads, dim, PAGE, context, value_dim=wide)
+            space = torch.empty(max(floats, 1), device=device, dtype=f32)
+            calls = [lambda k=k, v=v, q=packed, o=result, e=extras: kernels.decode_attention(
+                q, o, k, v, block_table, positions, PAGE, heads, kv_heads, dim, scale, None, partition, parts,
+                space if floats else None, **e) for k, v in zip(k_cache, values)]
+            table[f"{label}_{name}"] = timed(calls, rows * context * kv_heads * (dim + wide) * 2, hbm)
+        for name, extras in (("attention_window_kept_sink_gate", dict(sinks=sinks, gate=wide_gate)), ("doderax_attention_window_kept", {})):
+            if prompt:
+                calls = [lambda k=k, v=v, e=extras: kernels.prefill_attention(
+                    gated_rows, wide_out, k, v, block_table, starts, contexts, PAGE, heads, kv_heads, dim, scale, window,
+                    keep_first=keep, **e) for k, v in zip(k_cache, v_cache)]
+                table[f"{label}_{name}"] = timed(calls, 4.0 * in_window * heads * dim, flops_peak)
+                continue
+            partition, parts, floats = kernels.decode_attention_kept_plan(rows, heads, dim, context)
+            space = torch.empty(max(floats, 1), device=device, dtype=f32)
+            numbering = torch.empty(rows, device=device, dtype=i32)
+            calls = [lambda k=k, v=v, e=extras: kernels.decode_attention(
+                gated_rows, wide_out, k, v, block_table, positions, PAGE, heads, kv_heads, dim, scale, window, partition, parts,
+                space if floats else None, keep_first=keep, numbering=numbering, **e) for k, v in zip(k_cache, v_cache)]
+            table[f"{label}_{name}"] = timed(calls, rows * (min(window, context) + keep) * kv_heads * dim * 4, hbm)
+        # ---- the router: a softmax over the chosen logits, beside Zufotar's with groups and a correction
+        total, top = s["experts"], s["top"]
+        logits = [rand(tokens, total, dtype=f32) for _ in range(4)]
+        correction = rand(total, dtype=f32, scale=0.05)
+        ids = torch.empty(tokens, top, device=device, dtype=i32)
+        weights = torch.empty(tokens, top, device=device, dtype=f32)
+        route_bytes = tokens * (total * 4 + top * 8)
+        calls = [lambda l=l: kernels.moe_route(l, None, False, ids, weights, None, total, top, 1, 1, 1.0, score="softmax",
+                                               group_score="max") for l in logits]
+        table[f"{label}_moe_route_softmax_of_the_chosen"] = timed(calls, route_bytes, hbm)
+        calls = [lambda l=l: kernels.moe_route(l, correction, False, ids, weights, None, total, top, 8, 4, 2.5) for l in logits]
+        table[f"{label}_zufotar_moe_route"] = timed(calls, route_bytes, hbm)
+    return table
+
+
 def doderax_config(s: dict) -> dict:
     delta = {"heads": s["heads"], "kv_heads": s["heads"], "dim": s["dim"], "vdim": s["dim"], "conv": 4,
              "decay_rank": 64, "gate_rank": 64}
@@ -994,6 +1168,23 @@ def run(args, peaks: dict) -> dict:
             entry["pedotar"] = model_numbers(pedotar_config(s), s["vocab"])
             entry["zufotar_dense_feed_forwards"] = model_numbers(pedotar_beside(s), s["vocab"])
             entry["dense_swiglu"] = model_numbers(dense_config(dict(s, layers=s["runs"])), s["vocab"])
+            report[name] = entry
+        return report
+    if args.design == "biravik":
+        rand = lambda *shape, dtype=bf16, scale=1.0: (torch.randn(*shape, device=device, dtype=f32) * scale).to(dtype)
+        tools = {"timed": timed, "copies": copies, "rand": rand, "device": device, "hbm": hbm, "flops_peak": flops_peak}
+        report = {}
+        for name in [n for n in BIRAVIK_SIZES if args.design_sizes in ("all", n)]:
+            s = BIRAVIK_SIZES[name]
+            entry = {"sizes": s}
+            if not args.skip_points:
+                entry["kernels_us_and_fraction_of_roofline"] = biravik_kernel_table(s, tools)
+                torch.cuda.empty_cache()
+            entry["biravik"] = model_numbers(biravik_config(s), s["vocab"])
+            entry["zufotar"] = model_numbers(zufotar_config(ZUFOTAR_SIZES[name]), s["vocab"])
+            entry["biravik_dense_feed_forwards"] = model_numbers(biravik_config(s, experts=False), s["vocab"])
+            entry["doderax"] = model_numbers(doderax_config(s), s["vocab"])
+            entry["dense_swiglu"] = model_numbers(dense_config(s), s["vocab"])
             report[name] = entry
         return report
     if args.design == "dalesun":

@@ -243,25 +243,27 @@ def mixture(h, weights, prefix, mlp):
 
 
 # ------------------------------------------------------------------------------ the model
-def layer(x, index, config, weights):
+def layer(x, index, config, weights, read=lambda h: h):
+    """`read`: what a sublayer makes of the residual as it reads it (a rounding, to see how much of one the model magnifies)."""
     spec = config["layers"][index]
     eps, alpha = float(config["norm"]["eps"]), float(config["postln_alpha"])
     prefix = f"l{index}."
-    mixed = MIXERS[spec["type"]](x, weights, prefix + "mix.", spec["mixer"], eps)
+    mixed = MIXERS[spec["type"]](read(x), weights, prefix + "mix.", spec["mixer"], eps)
     x = post_norm(x, mixed, weights[prefix + "norm1"], alpha, eps)
     mlp = spec.get("mlp")
     if mlp is None:
         return x
-    fed = dense_mlp(x, weights, prefix + "mlp.") if mlp["kind"] == "dense" else mixture(x, weights, prefix + "mlp.", mlp)
+    fed = dense_mlp(read(x), weights, prefix + "mlp.") if mlp["kind"] == "dense" \
+        else mixture(read(x), weights, prefix + "mlp.", mlp)
     return post_norm(x, fed, weights[prefix + "norm2"], alpha, eps)
 
 
-def forward(config, weights, ids, trace=None):
+def forward(config, weights, ids, trace=None, read=lambda h: h):
     """Logits [n, vocab] of one sequence; `trace`, a list, receives the residual stream after every layer."""
     ids = torch.as_tensor(ids, dtype=torch.long)
     x = weights["embed"][ids] * float((config.get("embedding") or {}).get("scale", 1.0))
     for index in range(len(config["layers"])):
-        x = layer(x, index, config, weights)
+        x = layer(x, index, config, weights, read)
         if trace is not None:
             trace.append(x.clone())
     return (unit_rms(x, float(config["norm"]["eps"])) * (1.0 + weights["final.norm"])) @ weights["head"].T

@@ -729,8 +729,9 @@ def test_generate_command_line(tmp_path):
 @pytest.mark.parametrize("seed", range(10))
 def test_configurations_drawn_at_random(tmp_path, seed):
     """Sizes nobody chose: a prompt whole, token by token, in portions and as a prompt followed by decoding, in both dtypes,
-    against the plain implementation (32-bit: the same bits under every cut; bfloat16: nine positions in ten within twice
-    the tolerance)."""
+    against the plain implementation (32-bit: the same bits under every cut; bfloat16: nine positions in ten within the
+    tolerance, or within four times what rounding the sublayers' inputs alone does to the 64-bit implementation where a
+    model drawn at random magnifies that)."""
     rng = np.random.default_rng(900 + seed)
     config = random_config(rng)
     page = int(rng.choice([4, 8, 16]))
@@ -738,6 +739,10 @@ def test_configurations_drawn_at_random(tmp_path, seed):
     for dtype in ("float32", "bfloat16"):
         folder = make_folder(tmp_path / dtype, config, seed=seed, dtype=dtype)
         want = reference(folder, ids)
+        bound = TOL["bfloat16"]
+        if dtype == "bfloat16":
+            rounded = plain.forward(*plain.read_model(folder), ids, read=lambda h: h.to(BF16).double()).numpy()
+            bound = max(bound, 4.0 * np.quantile(relative_error(rounded, want), 0.9))
         model = load(folder, dtype, page, 80)
         outputs = [feed(model, "whole", ids, [len(ids)]), feed(model, "single", ids, [1]),
                    feed(model, "portions", ids, [2, 5, 1, 33, 3, 16, 2, 7]), feed(model, "late", ids, [80, 1])]
@@ -747,7 +752,7 @@ def test_configurations_drawn_at_random(tmp_path, seed):
             if dtype == "float32":
                 assert relative.max() <= 2e-4, f"{relative.max():.3e} at {int(relative.argmax())}: {json.dumps(config)}"
             else:
-                assert np.quantile(relative, 0.9) <= 2 * TOL[dtype], f"{np.quantile(relative, 0.9):.3e}: {json.dumps(config)}"
+                assert np.quantile(relative, 0.9) <= bound, f"{bound:.3e} < {np.quantile(relative, 0.9):.3e}: {json.dumps(config)}"
         if dtype == "float32":
             assert all(np.array_equal(outputs[0], other) for other in outputs[1:]), json.dumps(config)
         model.unload()
