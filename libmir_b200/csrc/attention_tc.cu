@@ -130,6 +130,18 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// a * b + c of two numbers side by side.
+__device__ __forceinline__ float2 fma_pair(float2 a, float2 b, float2 c) {
+  unsigned long long x, y, z, d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(x) : "f"(a.x), "f"(a.y));
+  asm("mov.b64 %0, {%1, %2};" : "=l"(y) : "f"(b.x), "f"(b.y));
+  asm("mov.b64 %0, {%1, %2};" : "=l"(z) : "f"(c.x), "f"(c.y));
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(x), "l"(y), "l"(z));
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(d));
+  return r;
+}
+
 // 32 consecutive accumulator columns of this thread's lane, without waiting for them (tmem_load_wait()).
 __device__ __forceinline__ void tmem_load_32_nowait(uint32_t address, float* v) {
   uint32_t r[32];
@@ -194,10 +206,18 @@ __device__ __forceinline__ float softmax_tile(uint32_t scores, int first, int lo
     if (slope != 0.0f) {                                     // a bias that falls linearly: slope * (distance - c) off
       const float fall = slope * kLog2e;
       const float lift0 = fmaf(-fall, (float)distance, base);
+      if (capped) {
 #pragma unroll
-      for (int c = 0; c < kCols; ++c) {
-        const float lift = fmaf(fall, (float)c, lift0);
-        v[c] = capped ? fmaf(drop, fast_reciprocal(1.0f + fast_exp2(v[c] * k)), lift) : fmaf(v[c], k, lift);
+        for (int c = 0; c < kCols; ++c)
+          v[c] = fmaf(drop, fast_reciprocal(1.0f + fast_exp2(v[c] * k)), fmaf(fall, (float)c, lift0));
+      } else {
+#pragma unroll
+        for (int c = 0; c < kCols; c += 2) {                 // two columns an instruction
+          const float2 lift = fma_pair(make_float2(fall, fall), make_float2((float)c, (float)(c + 1)), make_float2(lift0, lift0));
+          const float2 both = fma_pair(make_float2(v[c], v[c + 1]), make_float2(k, k), lift);
+          v[c] = both.x;
+          v[c + 1] = both.y;
+        }
       }
     } else if (bias == nullptr || nearest >= bias_last) {
       const float lift = base + (bias != nullptr ? __ldg(bias + bias_last) * kLog2e : 0.0f);
@@ -281,11 +301,15 @@ struct Work {
   // kept_tiles tiles are the key tiles from key 0 on, in which exactly the keys below `kept` are seen (by every
   // query), and in the window's tiles that follow those keys are hidden, so that no key counts twice.  Else 0, 0.
   int kept, kept_tiles;
+  // Scores that fall with the distance are largest near the query: the tiles then run from the last to the first, so that
+  // a row's reference is at its height from the start and the output is hardly ever rescaled (no kept keys then).
+  bool backwards;
   const int* table;
 };
 
 // The first key of the item's tile t.
 __device__ __forceinline__ int tile_first_key(const Work& w, int t) {
+  if (w.backwards) return w.key_begin + (w.tiles - 1 - t) * kKeys;
   return t < w.kept_tiles ? t * kKeys : w.key_begin + (t - w.kept_tiles) * kKeys;
 }
 
@@ -295,9 +319,10 @@ __device__ __forceinline__ int tile_first_key(const Work& w, int t) {
 __device__ __forceinline__ Work work_item(int index, int items, int query_tiles, int heads, int kv_heads, int num_rows,
                                           const int* __restrict__ query_starts, const int* __restrict__ context_lens,
                                           const int* __restrict__ block_table, int table_width, int window,
-                                          int keep_first) {
+                                          int keep_first, bool backwards) {
   Work w;
   w.valid = false;
+  w.backwards = backwards;
   if (index < 0 || index >= items) return w;
   w.head = index % heads;
   w.kv_head = w.head / (heads / kv_heads);
@@ -374,7 +399,7 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
   const int items = heads * query_tiles;
   auto work = [&](int k) {
     return work_item(item_of(k, cta, ctas, items), items, query_tiles, heads, kv_heads, num_rows, query_starts,
-                     context_lens, block_table, table_width, window, keep_first);
+                     context_lens, block_table, table_width, window, keep_first, kScored && extras.slopes != nullptr);
   };
   auto more = [&](int k) { return (long long)k * ctas < items; };
 
@@ -757,7 +782,7 @@ tc_prefill_attention_kernel(const __grid_constant__ CUtensorMap q_map, const __g
               float g[8];
               load8(gate + i, g);
 #pragma unroll
-              for (int j = 0; j < 8; ++j) o[i + j] *= 1.0f / (1.0f + __expf(-g[j]));
+              for (int j = 0; j < 8; ++j) o[i + j] *= fast_reciprocal(1.0f + __expf(-g[j]));
             }
           }
           if (valid_row && alive) {
@@ -846,8 +871,8 @@ static int prefill_attention_tc_with(const void* q, long long q_stride, void* ou
   const int value_dim = extras.value_dim > 0 ? extras.value_dim : head_dim;
   const bool scored = scores_modified(extras);
   if (!mir_prefill_attention_tc_takes_values(value_dim) || (value_dim != kDim && !scored) ||
-      (extras.slopes != nullptr && extras.rel_bias != nullptr)) {
-    mir_set_error("prefill_attention_tc: value heads of %d (64 goes with modified scores), and one kind of bias at a time",
+      (extras.slopes != nullptr && (extras.rel_bias != nullptr || (keep_first > 0 && window > 0)))) {
+    mir_set_error("prefill_attention_tc: value heads of %d (64 goes with modified scores), one kind of bias at a time, no kept keys beside slopes",
                   value_dim);
     return MIR_BAD_ARGUMENT;
   }

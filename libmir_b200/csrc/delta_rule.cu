@@ -373,27 +373,109 @@ __global__ void gated_head_norm_kernel(const float* __restrict__ o, const TG* __
   }
 }
 
-// The same for wide rows (a norm over all heads at once): one CTA per (token, head), its sum by a fixed tree.
-template <typename T, typename TG>
-__global__ void gated_wide_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, long long ld_gate,
-                                       const float* __restrict__ weight, T* __restrict__ out, int heads, int value_dim,
-                                       float eps, int sigmoid_gate, int weight_per_head) {
-  __shared__ float scratch[32];
-  grid_launch_dependents();
-  grid_dependency_wait();
-  const int unit = blockIdx.x;                                  // token * heads + head
-  const float* src = o + (size_t)unit * value_dim;
-  float sum = 0.0f;
-  for (int d = threadIdx.x; d < value_dim; d += blockDim.x) sum = fmaf(src[d], src[d], sum);
-  const float inverse = rsqrtf(block_sum(sum, scratch) / (float)value_dim + eps);
-  const TG* gate_row = gate + (size_t)(unit / heads) * ld_gate + (size_t)(unit % heads) * value_dim;
-  const float* scale = weight + (weight_per_head ? (size_t)(unit % heads) * value_dim : 0);
-  for (int d = threadIdx.x; d < value_dim; d += blockDim.x) {
-    const float z = to_float(gate_row[d]);
-    out[(size_t)unit * value_dim + d] = from_float<T>(src[d] * inverse * scale[d] * (sigmoid_gate ? sigmoid(z) : silu(z)));
+// The same for wide rows (a norm over all heads at once): one CTA per (token, head), its sum by a fixed tree.  A thread keeps
+// its columns in registers, V at a time in PIECES places blockDim.x * V columns apart; the gate's loads are on their way
+// while the sum is formed.
+template <typename T, int V>
+__device__ __forceinline__ void load_columns(float (&v)[V], const T* __restrict__ from) {
+  if constexpr (V == 4 && sizeof(T) == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(from);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  } else if constexpr (V == 4) {
+    const uint2 a = *reinterpret_cast<const uint2*>(from);
+    const float2 low = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.x));
+    const float2 high = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.y));
+    v[0] = low.x; v[1] = low.y; v[2] = high.x; v[3] = high.y;
+  } else {
+    v[0] = to_float(from[0]);
   }
 }
-constexpr int kWideNormColumns = 512;                           // rows from this width on take a CTA each
+template <typename T, typename TG, int V, int PIECES>
+__global__ void __launch_bounds__(512) gated_wide_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate,
+                                                              long long ld_gate, const float* __restrict__ weight,
+                                                              T* __restrict__ out, int heads, int value_dim, float eps,
+                                                              int sigmoid_gate, int weight_per_head) {
+  __shared__ float scratch[32];
+  grid_launch_dependents();
+  const int unit = blockIdx.x;                                  // token * heads + head
+  const float* scale = weight + (weight_per_head ? (size_t)(unit % heads) * value_dim : 0);
+  float w[PIECES][V], x[PIECES][V], g[PIECES][V];
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int d = (p * blockDim.x + threadIdx.x) * V;
+    if (d < value_dim) load_columns(w[p], scale + d);           // (older than the kernel before this one)
+  }
+  grid_dependency_wait();
+  const float* src = o + (size_t)unit * value_dim;
+  const TG* gate_row = gate + (size_t)(unit / heads) * ld_gate + (size_t)(unit % heads) * value_dim;
+  float sum = 0.0f;
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int d = (p * blockDim.x + threadIdx.x) * V;
+    if (d >= value_dim) continue;
+    load_columns(x[p], src + d);
+    load_columns(g[p], gate_row + d);
+  }
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    if ((p * blockDim.x + threadIdx.x) * V >= value_dim) continue;
+#pragma unroll
+    for (int v = 0; v < V; ++v) sum = fmaf(x[p][v], x[p][v], sum);
+  }
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
+  sum = warp_sum(sum);
+  if (lane == 0) scratch[warp] = sum;
+  __syncthreads();
+  float total = 0.0f;
+  for (int i = 0; i < warps; ++i) total += scratch[i];
+  const float inverse = rsqrtf(total / (float)value_dim + eps);
+  T* dst = out + (size_t)unit * value_dim;
+#pragma unroll
+  for (int p = 0; p < PIECES; ++p) {
+    const int d = (p * blockDim.x + threadIdx.x) * V;
+    if (d >= value_dim) continue;
+#pragma unroll
+    for (int v = 0; v < V; ++v) x[p][v] *= inverse * w[p][v] * (sigmoid_gate ? sigmoid(g[p][v]) : silu(g[p][v]));
+    if constexpr (V == 4 && sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(dst + d) = make_float4(x[p][0], x[p][1], x[p][2], x[p][3]);
+    } else if constexpr (V == 4) {
+      uint2 packed;
+      *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(x[p][0], x[p][1]);
+      *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(x[p][2], x[p][3]);
+      *reinterpret_cast<uint2*>(dst + d) = packed;
+    } else {
+      dst[d] = from_float<T>(x[p][0]);
+    }
+  }
+}
+
+template <typename T, typename TG>
+int launch_gated_wide_norm(const float* o, const TG* gate, long long ld_gate, const float* weight, T* out, int units,
+                           int heads, int value_dim, float eps, int sigmoid_gate, int weight_per_head, cudaStream_t stream) {
+  const bool aligned = value_dim % 4 == 0 && ld_gate % 4 == 0 && ((uintptr_t)o & 15) == 0 && ((uintptr_t)weight & 15) == 0 &&
+                       ((uintptr_t)gate & (4 * sizeof(TG) - 1)) == 0 && ((uintptr_t)out & (4 * sizeof(T) - 1)) == 0;
+#define MIR_WIDE_NORM(V, P)                                                                                               \
+  return mir_launch("gated_head_norm", gated_wide_norm_kernel<T, TG, V, P>, dim3(units), dim3(threads), 0, stream, 0, o, \
+                    gate, ld_gate, weight, out, heads, value_dim, eps, sigmoid_gate, weight_per_head)
+  const int per_thread = aligned ? 4 : 1;
+  const int places = (value_dim + per_thread - 1) / per_thread;
+  const int threads = places >= 512 ? 512 : (places + 31) / 32 * 32;
+  const int pieces = (places + threads - 1) / threads;
+  if (per_thread == 4) {
+    if (pieces <= 1) MIR_WIDE_NORM(4, 1);
+    if (pieces <= 2) MIR_WIDE_NORM(4, 2);
+    if (pieces <= 4) MIR_WIDE_NORM(4, 4);
+    if (pieces <= 8) MIR_WIDE_NORM(4, 8);
+  } else {
+    if (pieces <= 2) MIR_WIDE_NORM(1, 2);
+    if (pieces <= 8) MIR_WIDE_NORM(1, 8);
+    if (pieces <= 32) MIR_WIDE_NORM(1, 32);
+  }
+#undef MIR_WIDE_NORM
+  mir_set_error("gated_head_norm: rows of %d numbers are wider than the kernel takes", value_dim);
+  return MIR_BAD_ARGUMENT;
+}
+constexpr int kWideNormColumns = 512, kWideNormLimit = 16384;   // rows of these widths take a CTA each
 
 // How many lanes share a column of the state: 0 lets the launcher choose, 8 / 16 / 32 fix it (for measurements).
 int g_scan_lanes = 0;
@@ -537,19 +619,15 @@ MIR_EXPORT int mir_gated_head_norm(int bf16, int gate_f32, const float* o, const
   if (tokens == 0) return MIR_OK;
   if (tokens < 0 || heads <= 0 || value_dim <= 0) { mir_set_error("gated_head_norm: bad sizes"); return MIR_BAD_ARGUMENT; }
   const int units = tokens * heads;
-  if (value_dim >= kWideNormColumns) {
-    const dim3 threads(256);
+  if (value_dim >= kWideNormColumns && value_dim <= kWideNormLimit) {
     if (bf16 && gate_f32)
-      return mir_launch("gated_head_norm", gated_wide_norm_kernel<__nv_bfloat16, float>, dim3(units), threads, 0, stream, 0,
-                        o, (const float*)gate, ld_gate, weight, (__nv_bfloat16*)out, heads, value_dim, eps, sigmoid_gate,
-                        weight_per_head);
+      return launch_gated_wide_norm(o, (const float*)gate, ld_gate, weight, (__nv_bfloat16*)out, units, heads, value_dim, eps,
+                                    sigmoid_gate, weight_per_head, stream);
     if (bf16)
-      return mir_launch("gated_head_norm", gated_wide_norm_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(units), threads, 0,
-                        stream, 0, o, (const __nv_bfloat16*)gate, ld_gate, weight, (__nv_bfloat16*)out, heads, value_dim,
-                        eps, sigmoid_gate, weight_per_head);
-    return mir_launch("gated_head_norm", gated_wide_norm_kernel<float, float>, dim3(units), threads, 0, stream, 0, o,
-                      (const float*)gate, ld_gate, weight, (float*)out, heads, value_dim, eps, sigmoid_gate,
-                      weight_per_head);
+      return launch_gated_wide_norm(o, (const __nv_bfloat16*)gate, ld_gate, weight, (__nv_bfloat16*)out, units, heads,
+                                    value_dim, eps, sigmoid_gate, weight_per_head, stream);
+    return launch_gated_wide_norm(o, (const float*)gate, ld_gate, weight, (float*)out, units, heads, value_dim, eps,
+                                  sigmoid_gate, weight_per_head, stream);
   }
   const dim3 grid((units + 3) / 4), block(32, 4);
   if (bf16 && gate_f32)
