@@ -156,12 +156,11 @@ __global__ void __launch_bounds__(512) norm_scaled_sum_kernel(ScaledBranches bra
       v[0] = *from;
     }
   };
-  float w[PIECES][V];                                // the weight is older than the kernel before this one
-#pragma unroll
-  for (int p = 0; p < PIECES; ++p) {
-    const int c = (p * blockDim.x + threadIdx.x) * V;
-    if (c < hidden) load(w[p], weight + c);
-  }
+  // one piece a thread (few rows' shortest chain): the weight, older than the kernel before this one, is asked for ahead;
+  // more pieces: the registers serve the rows in flight, and the weight comes behind the sum
+  constexpr bool kEarly = PIECES == 1;
+  float early[V];
+  if (kEarly && threadIdx.x * V < hidden) load(early, weight + threadIdx.x * V);
   grid_dependency_wait();
   float u[PIECES][V];
   float sum = 0.0f;
@@ -193,8 +192,15 @@ __global__ void __launch_bounds__(512) norm_scaled_sum_kernel(ScaledBranches bra
   for (int p = 0; p < PIECES; ++p) {
     const int c = (p * blockDim.x + threadIdx.x) * V;
     if (c >= hidden) continue;
+    float w[V];
+    if (kEarly) {
 #pragma unroll
-    for (int v = 0; v < V; ++v) u[p][v] *= inverse * w[p][v];
+      for (int v = 0; v < V; ++v) w[v] = early[v];
+    } else {
+      load(w, weight + c);
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) u[p][v] *= inverse * w[v];
     if constexpr (V == 4) {
       *reinterpret_cast<float4*>(residual + base + c) = make_float4(u[p][0], u[p][1], u[p][2], u[p][3]);
       if (rounded) {
@@ -473,7 +479,9 @@ MIR_EXPORT int mir_norm_scaled_sum(const float* const* branch_rows, const float*
                     residual, weight, (__nv_bfloat16*)rounded, hidden, alpha, eps)
   const int per_thread = aligned ? 4 : 1;
   const int places = (hidden + per_thread - 1) / per_thread;
-  const int threads = places >= 512 ? 512 : (places + 31) / 32 * 32;
+  // (a prompt's rows: two pieces a thread, twice the loads in flight; a few rows: the shortest chain)
+  const int wanted = rows >= 256 ? (places + 1) / 2 : places;
+  const int threads = wanted >= 512 ? 512 : (wanted + 31) / 32 * 32;
   const int pieces = (places + threads - 1) / threads;
   if (per_thread == 4) {
     if (pieces <= 1) MIR_NORM_SUM(4, 1);

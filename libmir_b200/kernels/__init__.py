@@ -29,8 +29,6 @@ _SIGNATURES = {
         "mir_silu_mul": [c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "mir_add_bias": [c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "mir_cast": [c_int, c_void_p, c_void_p, c_size_t, c_void_p],
-        "mir_qk_rope_store": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                              c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_longlong, c_int, c_void_p],
         "mir_qk_rope_store_forms": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                     c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_longlong, c_int,
                                     c_float, c_float, c_float, c_int, c_void_p],
