@@ -1,5 +1,6 @@
 """`bench.py --design doderax | zufotar | dalesun | gumazen | pedotar | biravik`: prefill and decode throughput of a design at
-layer sizes that resemble a real model's (random weights), beside the dense SwiGLU decoder of equal width, depth and parameter count (and, for
+layer sizes that resemble a real model's (random weights), beside the dense SwiGLU decoder of equal width, depth and
+parameter count (and, for
 Zufotar, beside Doderax, the closest model of the framework: recurrent mixers and attention in parallel layers), and
 every kernel the design adds alone, with the fraction of its roofline, beside the like kernel of the closest model.
 
