@@ -263,7 +263,7 @@ class SoftmaxAttentionSpec(PartSpec):
     # sum_g head_mix[h, g] weights_g of all heads' softmax weights to the values of its own kv head.
     chunk: Optional[int] = None
     head_mix: bool = False
-    # values_from_keys: there is no value tensor, a token's value is its key as projected, before norm and rotation.
+    # values_from_keys: there is no value tensor, a token's value is the key's raw projection (neither normed nor rotated).
     # slopes: one number per query head (or none): slopes[h] * (query position - key position) is taken off the score.
     # temperature: what the queries are multiplied by.
     values_from_keys: bool = False

@@ -19,7 +19,7 @@
 // another entry's keys and values).
 // QkForms, further forms: magnitude multiplies cos and sin; temperature: a query at position p is multiplied by
 // 1 + coef ln(floor((p + 1) / every) + 1), in 32-bit, before it is stored; values_from_keys: the row holds no values, a
-// token's value is its key as projected, before norm and rotation, and goes to the value pages as it is.
+// token's value is the key's raw projection, which goes to the value pages as it is.
 #include "common.cuh"
 #include "trace.cuh"
 

@@ -1310,7 +1310,7 @@ def qk_rope_store(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opti
     the rotation pairs dims 2i and 2i + 1.  The rows may be wider than q, k and v (what lies behind them is left
     alone); `queries_only`: they start with the query heads and hold no keys or values.  `magnitude` multiplies cos and
     sin; `temperature` (coef, every): a query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1);
-    `values_from_keys`: the rows hold no values, a token's value is its key as projected (before norm and rotation)."""
+    `values_from_keys`: the rows hold no values, a token's value is the key's raw projection (neither normed nor rotated)."""
     write_kv = write_kv and not keys_in_place and not queries_only
     _cuda(qkv, positions, slot_mapping, inv_freq, q_norm, k_norm, k_pages, v_pages)
     tokens = qkv.shape[0]

@@ -88,7 +88,7 @@ BIRAVIK_D = {   # heads of 128 channels: values of 64, of 128 and of 32 beside t
     "architecture": "Biravik", "vocab": 97, "width": 128, "norm": {"eps": 1e-6}, "embedding": {"scale": 0.5},
     "postln_alpha": 0.8,
     "layers": [
-        _layer(_parallel(_left(4, 2, 128, 64, 0.09, (0.3, 50)), _right(128, 64, (0.99, 0.9)), 0.8, 0.9), _moe(5, 2, 48)),
+        _layer(_parallel(_left(4, 2, 128, 64, 0.09, (0.35, 50)), _right(128, 64, (0.99, 0.9)), 0.85, 1.05), _moe(5, 2, 48)),
         _layer(_attention(4, 1, 128, 0.08, window=70, keep_first=9, rot=(32, 10000.0, (4.0, 128, 32.0, 1.0))), _dense(200)),
         _layer(_parallel(_left(2, 1, 128, 128, 0.1, (0.6, 33)), _right(64, 128, (0.98,)), 1.3, 0.4), _dense(48)),
         _layer(_parallel(_left(2, 2, 128, 32, 0.1), _right(100, 20, (0.7, 0.995)), 1.0, 1.0), None),

@@ -1,7 +1,7 @@
 """A plain, slow implementation of the Biravik design in float64: whole sequences, no cache, no batching, one function
 per mechanism.  It shares no code with the package and is what the engine is compared with.
 
-Notation: n tokens, width w.  Weights are stored [out, in] and applied as W x; a row vector x of a token is multiplied
+Notation: n tokens, width w.  A stored matrix W has shape [out, in]; the row vector x of a token is multiplied
 as x @ W.T.
 """
 
@@ -177,7 +177,7 @@ def side_by_side(h, weights, prefix, mixer, eps):
 
 
 def key_value_attention(h, weights, prefix, mixer, eps):
-    """Windowed attention whose values are its keys as projected, before norm and rotation."""
+    """Windowed attention whose values are the keys' raw projections (neither normed nor rotated)."""
     n = h.shape[0]
     heads, kv_heads, dim = (int(mixer[key]) for key in ("heads", "kv_heads", "dim"))
     w = lambda name: weights[prefix + name]

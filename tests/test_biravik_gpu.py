@@ -531,7 +531,7 @@ FAR_LAYERS = {
     # steep scores and a temperature that lifts late queries; the flat slopes of many heads reach far back
     "parallel": [{"type": "parallel", "mlp": None, "mixer": {
         "left_scale": 1.0, "right_scale": 0.3,
-        "left": {"heads": 8, "kv_heads": 2, "dim": 64, "vdim": 32, "scale": 0.13, "q_temp": {"coef": 0.3, "every": 100}},
+        "left": {"heads": 8, "kv_heads": 2, "dim": 64, "vdim": 32, "scale": 0.13, "q_temp": {"coef": 0.35, "every": 100}},
         "right": {"heads": 2, "dim": 16, "vdim": 24, "decay": [0.9995, 0.998]}}}],
     "attention": [{"type": "attention", "mlp": None, "mixer": {
         "heads": 4, "kv_heads": 2, "dim": 64, "vdim": 64, "scale": 0.13, "rot": {"dims": 16, "base": 10000.0}}}],
