@@ -533,6 +533,11 @@ FAR_LAYERS = {
         "left_scale": 1.0, "right_scale": 0.3,
         "left": {"heads": 8, "kv_heads": 2, "dim": 64, "vdim": 32, "scale": 0.13, "q_temp": {"coef": 0.35, "every": 100}},
         "right": {"heads": 2, "dim": 16, "vdim": 24, "decay": [0.9995, 0.998]}}}],
+    # heads of 128 channels: many key tiles of the tcgen05 kernels, from the query backwards
+    "wide": [{"type": "parallel", "mlp": None, "mixer": {
+        "left_scale": 1.0, "right_scale": 0.2,
+        "left": {"heads": 8, "kv_heads": 2, "dim": 128, "vdim": 64, "scale": 0.05, "q_temp": {"coef": 0.3, "every": 90}},
+        "right": {"heads": 1, "dim": 16, "vdim": 24, "decay": [0.99]}}}],
     "attention": [{"type": "attention", "mlp": None, "mixer": {
         "heads": 4, "kv_heads": 2, "dim": 64, "vdim": 64, "scale": 0.13, "rot": {"dims": 16, "base": 10000.0}}}],
     "kept": [{"type": "attention", "mlp": None, "mixer": {
@@ -559,9 +564,10 @@ def test_far_tokens_decide_the_logits_in_prompt_and_in_decoding(tmp_path, kind):
             write_file(folder / "model.safetensors", tensors)
             plain_config, weights = plain.read_model(folder)
         want = plain.forward(plain_config, weights, ids).numpy()
-        changed = [(t + 1) % 90 for t in ids[:60]] + ids[60:]
+        early = 250 if kind == "wide" else 60                    # (a bias takes weight off what lies far back)
+        changed = [(t + 1) % 90 for t in ids[:early]] + ids[early:]
         moved = relative_error(plain.forward(plain_config, weights, changed).numpy()[-20:], want[-20:])
-        assert np.median(moved) > 5e-3, f"{kind}: the first sixty tokens hardly matter ({np.median(moved):.1e})"
+        assert np.median(moved) > 5e-3, f"{kind}: the first tokens hardly matter ({np.median(moved):.1e})"
         model = load(folder, dtype, 16, 50)
         for label, cuts in (("whole", [700]), ("late", [650, 1]), ("cut", [15, 17, 300, 2, 31])):
             got = feed(model, label, ids, cuts)
